@@ -4,6 +4,7 @@ from .lomopel_config import GatedDeltaConfig, LomopelConfig, LomopelLayer, Softm
 from .bufulorn_config import BufulornConfig, BufulornLayer, ChunkAttentionConfig, FeedForwardConfig, HeadDecayDeltaConfig
 from .pironex_config import (ClampedExpertsConfig, PironexConfig, PironexLayer, PooledAttentionConfig, StateSpaceConfig,
                              WindowLatentConfig)
+from .fanopel_config import FanopelConfig, FanopelLayer, KeyValueAttentionConfig, PlainExpertsConfig
 from .engine_config import EngineConfig, parse_dtype
 from .registry import (Architecture, register_architecture, unregister_architecture,
                        known_architectures, architecture_for)
@@ -11,6 +12,7 @@ from .registry import (Architecture, register_architecture, unregister_architect
 __all__ = ["LlamaConfig", "RopeScaling", "RotepelConfig", "RotepelLayer", "LomopelConfig", "LomopelLayer", "SoftmaxMixerConfig",
            "GatedDeltaConfig", "BufulornConfig", "BufulornLayer", "ChunkAttentionConfig", "FeedForwardConfig",
            "HeadDecayDeltaConfig", "PironexConfig", "PironexLayer", "PooledAttentionConfig", "StateSpaceConfig",
-           "WindowLatentConfig", "ClampedExpertsConfig", "read_config_json", "write_config_json", "EngineConfig",
+           "WindowLatentConfig", "ClampedExpertsConfig", "FanopelConfig", "FanopelLayer", "KeyValueAttentionConfig", "PlainExpertsConfig",
+           "read_config_json", "write_config_json", "EngineConfig",
            "parse_dtype", "Architecture", "register_architecture", "unregister_architecture",
            "known_architectures", "architecture_for"]

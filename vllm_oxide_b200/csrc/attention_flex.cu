@@ -4,6 +4,9 @@
 // earlier layer made of the same token, a window, blocks of positions, a cap on the scores, a bias that grows with the
 // distance, a sink in the softmax, a sigmoid gate on the result.
 //
+// The values may be the keys as projected (before their norm): the cache then holds only those, and one number per token
+// that brings its keys to unit root mean square; the norm's weights are taken into the query (vob_whole_norm_prep).
+//
 // Two steps per call of a layer:
 //   vob_flex_prep      per token: q, k, v (columns of one projection output) -> q' to a buffer, k' and
 //                      v' to their cache slots;
@@ -12,9 +15,12 @@
 //                                                `chunk` not before p - p % chunk (the query's own block of positions)
 //       with `pool` (and a window): every block of `pool` positions that ends at or before p - window is one more key and
 //                                                value, the means of the block's keys and values, in the same softmax
-//       s_j <- cap * tanh(s_j / cap)  (cap > 0);   s_j <- s_j - r1_a * ln(1 + r2_a * (p - j))  (r1, r2 given)
+//       with `keep` (and a window): the keys j < keep are seen too, at their true distances
+//       with `kscale` (one float per cached token): q . K is multiplied by key j's before anything else
+//       s_j <- cap * tanh(s_j / cap)  (cap > 0);   s_j <- s_j - r1_a * ln(1 + r2_a * (p - j))  (r1, r2 given), or
+//                                                s_j <- s_j - r1_a * (p - j)  (r1 alone)
 //       den = sum_j exp(s_j) (+ exp(sink_a): a key with no value, counted once)
-//       out_a = sum_j exp(s_j) V[j, g] / den    (* sigmoid(gate) * out_scale)
+//       out_a = sum_j exp(s_j) V[j, g] / den    (* sigmoid(gate) * out_scale; the gate per feature or one number per head)
 // The step's own keys are in the cache before they are read. Scores, softmax, angles, norms and the
 // query factor are float32. Cache layout per layer: K [pages][G][page_size][D], V [pages][G][page_size][DV].
 #include "common.cuh"
@@ -232,6 +238,135 @@ template <> struct Vec16<__nv_bfloat16> {
     }
 };
 
+// ---------------------------------------------------------------------------------------------
+// Preparation where q and k are each normed as a whole (all heads at once, a weight per feature), nothing is rotated and the
+// values are the keys as projected. One block of 256 threads per token; q and k lie side by side in `proj` from column q_off:
+//   q_out = q / sqrt(mean(q^2) + eps) * qw,   qw [H * D] = the query norm's weights times the key norm's (of the kv head a
+//                                             query head reads), so that q_out . k is the normed q times the weighted k;
+//   K     = k as it is;   kscale[slot] = 1 / sqrt(mean(k^2) + eps).
+// VN features a thread and turn (16 bytes where the rows allow, else one), NV turns held in registers (0: read twice).
+// Padding rows (position < 0) are left alone; a negative slot skips the cache write.
+// ---------------------------------------------------------------------------------------------
+template <typename T, int VN> struct PrepVec;
+template <typename T> struct PrepVec<T, 1> {
+    __device__ static inline void load(const T* p, float* o) { o[0] = ld_f(p); }
+    __device__ static inline void store(T* p, const float* v) { st_f(p, v[0]); }
+};
+template <> struct PrepVec<float, 4> {
+    __device__ static inline void load(const float* p, float* o) { Vec16<float>::load(p, o); }
+    __device__ static inline void store(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+};
+template <> struct PrepVec<__nv_bfloat16, 8> {
+    __device__ static inline void load(const __nv_bfloat16* p, float* o) { Vec16<__nv_bfloat16>::load(p, o); }
+    __device__ static inline void store(__nv_bfloat16* p, const float* v) {
+        uint4 u;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        *reinterpret_cast<uint4*>(p) = u;
+    }
+};
+
+template <typename T, int VN, int NV>
+__global__ void __launch_bounds__(256)
+whole_norm_prep_kernel(const T* __restrict__ proj, long ld, int q_off, const int* __restrict__ positions, const int* __restrict__ slots,
+                       const float* __restrict__ qw, float eps, T* __restrict__ q_out, long ld_q, T* __restrict__ kcache,
+                       float* __restrict__ kscale, int H, int G, int D, int page_size) {
+    pdl_launch_dependents();
+    pdl_wait(64);
+    __shared__ float red[2][8];
+    const int t = blockIdx.x, tid = threadIdx.x;
+    const int nq = H * D, n = (H + G) * D;
+    const T* src = proj + (size_t)t * ld + q_off;
+    float v[NV > 0 ? NV : 1][VN];
+    float sq = 0.f, sk = 0.f;
+    auto sum = [&](int c, const float* x) {
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < VN; ++i) s = fmaf(x[i], x[i], s);
+        if (c * VN < nq) sq += s; else sk += s;
+    };
+    if (NV > 0) {
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int c = tid + 256 * j;
+            if (c * VN < n) PrepVec<T, VN>::load(src + (size_t)c * VN, v[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int c = tid + 256 * j;
+            if (c * VN < n) sum(c, v[j]);
+        }
+    } else {
+        for (int c = tid; c * VN < n; c += 256) {
+            PrepVec<T, VN>::load(src + (size_t)c * VN, v[0]);
+            sum(c, v[0]);
+        }
+    }
+    const int pos = positions[t], slot = slots[t];
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
+    __syncthreads();
+    if (pos < 0) return;                             // the whole block
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) { sq += red[0][i]; sk += red[1][i]; }
+    const float inv_q = 1.0f / sqrtf(sq / (float)nq + eps);
+    auto write = [&](int c, float* x) {
+        const int f = c * VN;
+        if (f < nq) {
+#pragma unroll
+            for (int i = 0; i < VN; ++i) x[i] = x[i] * inv_q * qw[f + i];
+            PrepVec<T, VN>::store(q_out + (size_t)t * ld_q + f, x);
+        } else if (slot >= 0) {
+            const int g = (f - nq) / D, d = (f - nq) - g * D;
+            PrepVec<T, VN>::store(kcache + ((size_t)((slot / page_size) * G + g) * page_size + slot % page_size) * D + d, x);
+        }
+    };
+    if (NV > 0) {
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int c = tid + 256 * j;
+            if (c * VN < n) write(c, v[j]);
+        }
+    } else {
+        for (int c = tid; c * VN < n; c += 256) {
+            PrepVec<T, VN>::load(src + (size_t)c * VN, v[0]);
+            write(c, v[0]);
+        }
+    }
+    if (tid == 0 && slot >= 0) kscale[slot] = 1.0f / sqrtf(sk / (float)(G * D) + eps);
+}
+
+VOB_EXPORT int vob_whole_norm_prep(const void* proj, int code, long ld, int q_off, const int* positions, const int* slots, const float* qw,
+                                   float eps, void* q_out, long ld_q, void* kcache, float* kscale, int T_rows, int H, int G, int D,
+                                   int page_size, cudaStream_t stream) {
+    if (T_rows <= 0) return 0;
+    if (H <= 0 || G <= 0 || D <= 0 || page_size <= 0 || q_off < 0 || !positions || !slots || !qw || !kcache || !kscale) return VOB_ERR_BAD_ARG;
+    const long long n = (long long)(H + G) * D;
+    if (n > 0x3fffffffLL) return VOB_ERR_UNSUPPORTED;
+#define VOB_WNP(T_, VN_, NV_)                                                                                                              \
+    return vob_launch(whole_norm_prep_kernel<T_, VN_, NV_>, dim3(T_rows), dim3(256), 0, stream, (const T_*)proj, ld, q_off, positions, slots, qw, \
+                      eps, (T_*)q_out, ld_q, (T_*)kcache, kscale, H, G, D, page_size)
+    const int vn = code == VOB_BF16 ? 8 : 4;
+    const bool vec = D % vn == 0 && q_off % vn == 0 && ld % vn == 0 && ld_q % vn == 0 &&
+                     ((((uintptr_t)proj) | ((uintptr_t)q_out) | ((uintptr_t)kcache)) & 15) == 0;
+    const long long turns = (n / vn + 255) / 256;
+    if (code == VOB_BF16) {
+        if (!vec) VOB_WNP(__nv_bfloat16, 1, 0);
+        if (turns <= 1) VOB_WNP(__nv_bfloat16, 8, 1);
+        if (turns <= 2) VOB_WNP(__nv_bfloat16, 8, 2);
+        if (turns <= 4) VOB_WNP(__nv_bfloat16, 8, 4);
+        VOB_WNP(__nv_bfloat16, 8, 0);
+    }
+    if (code != VOB_F32) return VOB_ERR_BAD_ARG;
+    if (!vec) VOB_WNP(float, 1, 0);
+    if (turns <= 4) VOB_WNP(float, 4, 4);
+    VOB_WNP(float, 4, 0);
+#undef VOB_WNP
+}
+
 __device__ __forceinline__ float flex_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 template <typename T>
@@ -241,7 +376,8 @@ flex_attention_warp_kernel(const T* __restrict__ q, long q_stride, T* __restrict
                            int max_pages, const int* __restrict__ row_seq, const int* __restrict__ positions, int T_rows, int H,
                            int G, int D, int DV, int page_size, int window, float scale, const float* __restrict__ sink,
                            const T* __restrict__ gate, long gate_stride, float out_scale, int chunk, float softcap,
-                           const float* __restrict__ dist_r1, const float* __restrict__ dist_r2, int pool) {
+                           const float* __restrict__ dist_r1, const float* __restrict__ dist_r2, int pool, int keep,
+                           const float* __restrict__ kscale, int gate_heads) {
     pdl_launch_dependents();
     pdl_wait(62);
     extern __shared__ float qs_all[];
@@ -264,7 +400,7 @@ flex_attention_warp_kernel(const T* __restrict__ q, long q_stride, T* __restrict
     const int* bt = block_tables + (size_t)seq * max_pages;
     int first = window > 0 ? max(0, pos + 1 - window) : 0;
     if (chunk > 0) first = max(first, pos - pos % chunk);
-    const float r1 = dist_r1 ? dist_r1[head] : 0.f, r2 = dist_r1 ? dist_r2[head] : 0.f;
+    const float r1 = dist_r1 ? dist_r1[head] : 0.f, r2 = dist_r2 ? dist_r2[head] : 0.f;
 
     constexpr int VN = Vec16<T>::N;
     const bool vec = D % VN == 0;                    // a key row then starts on a 16-byte boundary
@@ -324,9 +460,13 @@ flex_attention_warp_kernel(const T* __restrict__ q, long q_stride, T* __restrict
             }
         }
     }
-    for (int c0 = first; c0 <= pos; c0 += 32) {
+    // kept first tokens that the window does not reach, then the window's
+    const int n_kept = min(keep, first), kept_chunks = (n_kept + 31) / 32, chunks = kept_chunks + (pos - first) / 32 + 1;
+    for (int ci = 0; ci < chunks; ++ci) {
+        const bool kept = ci < kept_chunks;
+        const int c0 = kept ? ci * 32 : first + (ci - kept_chunks) * 32, last = kept ? n_kept - 1 : pos;
         const int j = c0 + lane;
-        const bool valid = j <= pos;
+        const bool valid = j <= last;
         int slot_row = 0;                            // row of key j in the [.., D] / [.., DV] view of the layer's cache
         float s = -INFINITY;
         if (valid) {
@@ -344,9 +484,11 @@ flex_attention_warp_kernel(const T* __restrict__ q, long q_stride, T* __restrict
             } else {
                 for (int d = 0; d < D; ++d) dot = fmaf(qs[d], ld_f(kp + d), dot);
             }
+            if (kscale) dot *= kscale[(size_t)page * page_size + j % page_size];
             s = dot * scale;
             if (softcap > 0.f) s = softcap * tanhf(s / softcap);
-            if (dist_r1) s -= r1 * log1pf(r2 * (float)(pos - j));
+            if (dist_r2) s -= r1 * log1pf(r2 * (float)(pos - j));
+            else if (dist_r1) s -= r1 * (float)(pos - j);
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float p = valid ? expf(s - m_new) : 0.f;
@@ -355,7 +497,7 @@ flex_attention_warp_kernel(const T* __restrict__ q, long q_stride, T* __restrict
 #pragma unroll
         for (int i = 0; i < 8; ++i) acc[i] *= alpha;
         m = m_new;
-        const int nk = min(32, pos - c0 + 1);
+        const int nk = min(32, last - c0 + 1);
         for (int jj = 0; jj < nk; ++jj) {
             const float pj = __shfl_sync(0xffffffffu, p, jj);
             const int sr = __shfl_sync(0xffffffffu, slot_row, jj);
@@ -376,13 +518,13 @@ flex_attention_warp_kernel(const T* __restrict__ q, long q_stride, T* __restrict
         for (int i = 0; i < 8; ++i) acc[i] *= alpha;
     }
     const float inv_l = out_scale / l;
-    const T* gp = gate ? gate + (size_t)row * gate_stride + (size_t)head * DV : nullptr;
+    const T* gp = gate ? gate + (size_t)row * gate_stride + (gate_heads ? (size_t)head : (size_t)head * DV) : nullptr;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int d = lane + 32 * i;
         if (d < DV) {
             float v = acc[i] * inv_l;
-            if (gp) v *= flex_sigmoid(ld_f(gp + d));
+            if (gp) v *= flex_sigmoid(ld_f(gp + (gate_heads ? 0 : d)));
             st_f(op + d, v);
         }
     }
@@ -392,12 +534,13 @@ VOB_EXPORT int vob_flex_attention(const void* q, long q_stride, void* out, long 
                                   int code, const int* block_tables, int max_pages, const int* row_seq, const int* positions,
                                   int T_rows, int H, int G, int D, int DV, int page_size, int window, float scale,
                                   const float* sink, const void* gate, long gate_stride, float out_scale, int chunk, float softcap,
-                                  const float* dist_r1, const float* dist_r2, int pool, cudaStream_t stream) {
+                                  const float* dist_r1, const float* dist_r2, int pool, int keep, const float* kscale, int gate_heads,
+                                  cudaStream_t stream) {
     if (T_rows <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G != 0 || page_size <= 0 || max_pages <= 0 || D <= 0 || DV <= 0) return VOB_ERR_BAD_ARG;
     if (D > 256 || DV > 256) return VOB_ERR_UNSUPPORTED;
-    if (chunk < 0 || softcap < 0.f || (dist_r1 != nullptr) != (dist_r2 != nullptr) || pool < 0 || (pool > 0 && (window <= 0 || chunk > 0)))
-        return VOB_ERR_BAD_ARG;
+    if (chunk < 0 || softcap < 0.f || (dist_r2 && !dist_r1) || pool < 0 || (pool > 0 && (window <= 0 || chunk > 0))) return VOB_ERR_BAD_ARG;
+    if (keep < 0 || (keep > 0 && (window <= 0 || chunk > 0 || pool > 0)) || (pool > 0 && (dist_r1 || kscale))) return VOB_ERR_BAD_ARG;
     const long long warps = (long long)T_rows * H;
     const long long blocks = (warps + 3) / 4;
     if (blocks > 0x7fffffffLL) return VOB_ERR_UNSUPPORTED;
@@ -406,6 +549,6 @@ VOB_EXPORT int vob_flex_attention(const void* q, long q_stride, void* out, long 
                                               (const ElemT*)q, q_stride, (ElemT*)out, out_stride, (const ElemT*)kcache,
                                               (const ElemT*)vcache, block_tables, max_pages, row_seq, positions, T_rows, H, G, D, DV,
                                               page_size, window, scale, sink, (const ElemT*)gate, gate_stride, out_scale, chunk, softcap,
-                                              dist_r1, dist_r2, pool));
+                                              dist_r1, dist_r2, pool, keep, kscale, gate_heads));
     return 0;
 }

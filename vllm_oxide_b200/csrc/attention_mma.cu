@@ -21,7 +21,7 @@
 //
 // What may follow the weighted sum (`AttnTail`, all optional): a sink per head (exp(sink) joins the
 // softmax's denominator once, a key with no value), a gate (the result times sigmoid(gate[row,
-// head * hd + d])) and a constant factor.
+// head * hd + d]), or sigmoid(gate[row, head]) with one number per head) and a constant factor.
 #include "common.cuh"
 VOB_PDL_SWITCH(attention_mma)
 
@@ -63,21 +63,28 @@ struct AttnTail {
     const __nv_bfloat16* gate;        // [rows, gate_stride], or null
     long long gate_stride;
     float out_scale;
+    int gate_heads;                   // the gate has one column per head
 };
 // The denominator of a row of `head` whose sum `L` is relative to the maximum `Ms` (base-2 scale).
 __device__ __forceinline__ float tail_den(const AttnTail& t, int head, float L, float Ms) {
     return t.sink ? L + exp2f(t.sink[head] * 1.4426950408889634f - Ms) : L;
 }
-__device__ __forceinline__ float tail_val(const AttnTail& t, long long row, int col, float v) {
+__device__ __forceinline__ float tail_val(const AttnTail& t, long long row, int head, int col, float v) {
     v *= t.out_scale;
-    if (t.gate) v *= 1.0f / (1.0f + expf(-__bfloat162float(t.gate[row * t.gate_stride + col])));
+    if (t.gate) v *= 1.0f / (1.0f + expf(-__bfloat162float(t.gate[row * t.gate_stride + (t.gate_heads ? head : col)])));
     return v;
 }
 
 // What may lie between q . k and the softmax (all optional; the kernels built with SHAPED take it):
 //   chunk > 0    a query reads only the keys of its own block of `chunk` positions, blocks counted from position 0;
 //   a cap        score <- softcap * tanh(score / softcap);
-//   r1, r2       [H] each: r1 * ln(1 + r2 * (i - j)) is taken off the score of key j for the query at i.
+//   r1, r2       [H] each: r1 * ln(1 + r2 * (i - j)) is taken off the score of key j for the query at i; with `linear`
+//                r1 * (i - j) is (r2 is not used);
+//   keep         (with a window) the keys of the first `keep` positions are seen by every query behind them (the portion kernel
+//                takes it where the values are the keys, KV1);
+//   kscale       one float per cached token (laid out [pages][page_size]): q . k is multiplied by key j's before anything else
+//                (kernels built with KV1, where the cache holds the keys as projected: those are the values, and their norm,
+//                one number per token and a weight per feature, is this number and a factor on q).
 // Scores leave in base-2 units (times log2 e), and the launchers' scale_log2 is not used by a shaped kernel. The struct
 // is a kernel parameter: what the inner loop reads of it comes from the constant bank and holds no register.
 //   pooled keys  (with a window, portion kernel only) beside the window's tokens a query at position p sees the first
@@ -92,14 +99,18 @@ struct ScoreShape {
     const __nv_bfloat16* kp;      // pooled keys and values (null: none), laid out like the caches
     const __nv_bfloat16* vp;
     int pool;
+    int keep;
+    int linear;
+    const float* kscale;
 };
 inline ScoreShape make_shape(int chunk, float softcap, const float* r1, const float* r2, float scale, const void* kp = nullptr,
-                             const void* vp = nullptr, int pool = 0) {
+                             const void* vp = nullptr, int pool = 0, int keep = 0, int linear = 0, const float* kscale = nullptr) {
     const float log2e = 1.4426950408889634f;
     return ScoreShape{chunk, softcap > 0.f ? scale / softcap : scale * log2e, softcap > 0.f ? softcap * log2e : 0.f, r1, r2,
-                      (const __nv_bfloat16*)kp, (const __nv_bfloat16*)vp, pool};
+                      (const __nv_bfloat16*)kp, (const __nv_bfloat16*)vp, pool, keep, linear, kscale};
 }
-// The distance bias of a thread's two rows: r1 and r2 of their heads (zero for a row that is no row of the request).
+// The distance bias of a thread's two rows: r1 and r2 of their heads (zero for a row that is no row of the request); a linear
+// bias has its slope in base-2 units here.
 struct RowShape {
     float r1[2], r2[2];
 };
@@ -108,8 +119,12 @@ __device__ __forceinline__ RowShape row_shape(const ScoreShape& sh, int head0, i
     const bool bias = sh.r1 != nullptr;
     rs.r1[0] = bias && head0 >= 0 ? sh.r1[head0] : 0.f;
     rs.r1[1] = bias && head1 >= 0 ? sh.r1[head1] : 0.f;
-    rs.r2[0] = bias && head0 >= 0 ? sh.r2[head0] : 0.f;
-    rs.r2[1] = bias && head1 >= 0 ? sh.r2[head1] : 0.f;
+    if (sh.linear) {
+        rs.r1[0] *= 1.4426950408889634f;
+        rs.r1[1] *= 1.4426950408889634f;
+    }
+    rs.r2[0] = bias && !sh.linear && head0 >= 0 ? sh.r2[head0] : 0.f;
+    rs.r2[1] = bias && !sh.linear && head1 >= 0 ? sh.r2[head1] : 0.f;
     return rs;
 }
 // The first key a query at `pos` reads (0 for a row of position -1, which is no row of a request).
@@ -132,14 +147,15 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 // Gather one tile of 64 keys (K and V of one kv head) into shared memory. Keys outside
-// [lo, hi) are zero-filled and never touched in global memory. Page numbers come from `s_pages`,
+// [lo, hi) and [0, keep) are zero-filled and never touched in global memory.
+// VALUES false: only K. Page numbers come from `s_pages`,
 // this block's copy of its request's block-table entries starting at logical page `page0` (a
 // global lookup per key would put a dependent L2 round trip in front of every copy); page sizes
 // are powers of two (they divide 64), so positions split into page and offset by shift and mask.
-template <int HD>
+template <int HD, bool VALUES = true>
 __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* sK, __nv_bfloat16* sV, const __nv_bfloat16* __restrict__ kc,
                                              const __nv_bfloat16* __restrict__ vc, const int* s_pages, int page0, int kvh,
-                                             int KV, int page_shift, int tile_start, int lo, int hi) {
+                                             int KV, int page_shift, int tile_start, int lo, int hi, int keep = 0) {
     constexpr int LD = HD + 8;
     constexpr int CH = HD / 8;                 // 16-byte pieces per key
     constexpr int KEYS_PER_PASS = NTHREADS / CH;
@@ -151,15 +167,29 @@ __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* sK, __nv_bfloat16* s
         int j = tile_start + key;
         __nv_bfloat16* dk = sK + key * LD + ch * 8;
         __nv_bfloat16* dv = sV + key * LD + ch * 8;
-        if (j >= lo && j < hi) {
+        if ((j >= lo || j < keep) && j < hi) {
             int page = s_pages[(j >> page_shift) - page0];
             size_t off = ((((size_t)page * KV + kvh) << page_shift) + (j & (page_size - 1))) * HD + ch * 8;
             cp_async16(dk, kc + off);
-            cp_async16(dv, vc + off);
+            if (VALUES) cp_async16(dv, vc + off);
         } else {
             *reinterpret_cast<uint4*>(dk) = make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint4*>(dv) = make_uint4(0, 0, 0, 0);
+            if (VALUES) *reinterpret_cast<uint4*>(dv) = make_uint4(0, 0, 0, 0);
         }
+    }
+}
+
+// The tile's 64 numbers per cached token (ones without `kscale`) into shared memory, for the same keys.
+__device__ __forceinline__ void load_key_scales(float* sR, const float* __restrict__ kscale, const int* s_pages, int page0, int page_shift,
+                                                int tile_start, int lo, int hi, int keep) {
+    if (threadIdx.x >= BN) return;
+    const int j = tile_start + threadIdx.x;
+    float* d = sR + threadIdx.x;
+    if (kscale && (j >= lo || j < keep) && j < hi) {
+        const float* s = kscale + ((size_t)s_pages[(j >> page_shift) - page0] << page_shift) + (j & ((1 << page_shift) - 1));
+        asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(smem_u32(d)), "l"(s));
+    } else {
+        *d = 1.f;
     }
 }
 
@@ -203,11 +233,12 @@ __device__ __forceinline__ void pv_tile(float (&o)[HD / 8][4], const uint32_t (&
 // starting at key index key0; this thread's rows are r and r+8 with limits [lo, pos]. With MASK
 // false the caller knows that every key of the tile is visible to every row of the warp. SHAPED: the scores
 // first become what `rs` makes of them (cap, distance bias), in base-2 units, and `scale_log2` is not used.
-template <int NB, int HDN, bool MASK, bool SHAPED = false>
+// KSC: q . k is first multiplied by key j's number, ksc[j - key0].
+template <int NB, int HDN, bool MASK, bool SHAPED = false, bool KSC = false, bool KEPT = KSC>
 __device__ __forceinline__ void softmax_step(float (&s)[NB][4], uint32_t (&pa)[NB / 2][4], float (&o)[HDN][4],
                                              float (&m)[2], float (&l)[2], int key0, const int (&lo)[2],
                                              const int (&pos)[2], float scale_log2, const ScoreShape* sh = nullptr,
-                                             const RowShape* rs = nullptr) {
+                                             const RowShape* rs = nullptr, const float* ksc = nullptr) {
     int lane = threadIdx.x & 31;
     float mx[2] = {-INFINITY, -INFINITY};
     if (SHAPED) scale_log2 = 1.f;
@@ -219,13 +250,15 @@ __device__ __forceinline__ void softmax_step(float (&s)[NB][4], uint32_t (&pa)[N
             if (SHAPED) {
                 int j = key0 + nb * 8 + (lane & 3) * 2 + (i & 1);
                 float t = s[nb][i] * sh->pre;
+                if (KSC) t *= ksc[nb * 8 + (lane & 3) * 2 + (i & 1)];
                 if (sh->cap_log2 > 0.f) t = sh->cap_log2 * fast_tanh(t);
-                if (sh->r1) t -= rs->r1[h] * __log2f(fmaf(rs->r2[h], (float)max(pos[h] - j, 0), 1.f));
+                if (sh->linear) t = fmaf(-rs->r1[h], (float)(pos[h] - j), t);
+                else if (sh->r1) t -= rs->r1[h] * __log2f(fmaf(rs->r2[h], (float)max(pos[h] - j, 0), 1.f));
                 s[nb][i] = t;
             }
             if (MASK) {
                 int j = key0 + nb * 8 + (lane & 3) * 2 + (i & 1);
-                if (!(j >= lo[h] && j <= pos[h])) s[nb][i] = -INFINITY;
+                if (!((j >= lo[h] || (KEPT && j < sh->keep)) && j <= pos[h])) s[nb][i] = -INFINITY;
             }
             mx[h] = fmaxf(mx[h], s[nb][i]);
         }
@@ -395,8 +428,8 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride,
         const int col = head * HD + (lane & 3) * 2;
 #pragma unroll
         for (int n = 0; n < HD / 8; ++n)
-            *reinterpret_cast<uint32_t*>(op + n * 8) = pack_bf16(tail_val(tail, row0 + tok, col + n * 8, o[n][2 * h] * inv),
-                                                                 tail_val(tail, row0 + tok, col + n * 8 + 1, o[n][2 * h + 1] * inv));
+            *reinterpret_cast<uint32_t*>(op + n * 8) = pack_bf16(tail_val(tail, row0 + tok, head, col + n * 8, o[n][2 * h] * inv),
+                                                                 tail_val(tail, row0 + tok, head, col + n * 8 + 1, o[n][2 * h + 1] * inv));
     }
 }
 
@@ -404,18 +437,19 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride,
 // The same for keys of D and values of DV features (multiples of 8 up to 128, different or not): the tiles in
 // shared memory are HD = D rounded up to a multiple of 32 and HDV = DV rounded up to 32, 64 or 128 wide, the
 // columns beyond the real sizes zero (a zero column of Q and K adds nothing to a score, a zero column of V
-// gives an output column that is not stored). Same grid, same walk over the key tiles, same tail.
+// gives an output column that is not stored). Same grid, same walk over the key tiles, same tail. KV1: the values are the
+// cached keys (HDV == HD): a tile is fetched once and serves both products, with a number per key beside it (`ScoreShape`).
 // ---------------------------------------------------------------------------------------------
 template <int W>
 __device__ __forceinline__ void load_rows_padded(__nv_bfloat16* dst, const __nv_bfloat16* __restrict__ cache, int real, const int* s_pages,
-                                                 int page0, int kvh, int KV, int page_shift, int tile_start, int lo, int hi) {
+                                                 int page0, int kvh, int KV, int page_shift, int tile_start, int lo, int hi, int keep = 0) {
     constexpr int LD = W + 8, CH = W / 8;
     const int page_size = 1 << page_shift, real_ch = real >> 3;
     for (int idx = threadIdx.x; idx < BN * CH; idx += NTHREADS) {
         const int key = idx / CH, ch = idx - key * CH;
         const int j = tile_start + key;
         __nv_bfloat16* d = dst + key * LD + ch * 8;
-        if (ch < real_ch && j >= lo && j < hi) {
+        if (ch < real_ch && (j >= lo || j < keep) && j < hi) {
             const int page = s_pages[(j >> page_shift) - page0];
             cp_async16(d, cache + ((((size_t)page * KV + kvh) << page_shift) + (j & (page_size - 1))) * real + ch * 8);
         } else {
@@ -424,8 +458,12 @@ __device__ __forceinline__ void load_rows_padded(__nv_bfloat16* dst, const __nv_
     }
 }
 
-template <int HD, int HDV, bool SHAPED>
-__global__ void __launch_bounds__(NTHREADS)
+// Blocks per SM the compiler is told to aim at, where its own choice of registers would spill a few bytes.
+constexpr int any_min_blocks(int hd, int hdv, bool shaped, bool kv1) {
+    return shaped && !kv1 && hd == 96 && hdv == 64 ? 2 : kv1 && hd == 32 ? 3 : 1;
+}
+template <int HD, int HDV, bool SHAPED, bool KV1>
+__global__ void __launch_bounds__(NTHREADS, any_min_blocks(HD, HDV, SHAPED, KV1))
 attn_prefill_mma_any_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, __nv_bfloat16* __restrict__ out,
                             long long out_stride, const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc,
                             const int* __restrict__ block_tables, int max_pages, const int* __restrict__ seq_starts,
@@ -438,8 +476,11 @@ attn_prefill_mma_any_kernel(const __nv_bfloat16* __restrict__ q, long long q_str
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem_raw);
     __nv_bfloat16* sK0 = sQ + BM * LD;
-    __nv_bfloat16* sV0 = sK0 + 2 * BN * LD;
-    int* s_pages = reinterpret_cast<int*>(sV0 + 2 * BN * LDV);            // [2 * max_pages]: the tokens' pages, then the pooled entries'
+    static_assert(!KV1 || (SHAPED && HD == HDV), "one tile serves both products");
+    __nv_bfloat16* sV0 = KV1 ? sK0 : sK0 + 2 * BN * LD;
+    float* sR0 = reinterpret_cast<float*>(sK0 + 2 * BN * LD);            // KV1: [2][BN] a number per key
+    // [2 * max_pages]: the tokens' pages, then the kept first tokens' or the pooled entries'
+    int* s_pages = KV1 ? reinterpret_cast<int*>(sR0 + 2 * BN) : reinterpret_cast<int*>(sV0 + 2 * BN * LDV);
 
     const int G = H / KV;
     const int kvh = blockIdx.x, seq = blockIdx.y;
@@ -468,34 +509,31 @@ attn_prefill_mma_any_kernel(const __nv_bfloat16* __restrict__ q, long long q_str
     const int first_tok_pos = ctx + tile_row0 / G;
     const int chunk = SHAPED ? shape.chunk : 0;
     const int lo_blk = first_key(first_tok_pos, window, chunk);      // the block's first row reads furthest back
-    const int pool = SHAPED && shape.kp ? shape.pool : 0;
+    const int pool = SHAPED && !KV1 && shape.kp ? shape.pool : 0;
     // pooled entries the block's last row sees (the most of all its rows)
     const int hi_pool = pool > 0 && window > 0 && hi - window >= pool ? (hi - window) / pool : 0;
 
-    int pos[2], lo[2], hd[2], pos_p[2];
+    // the last pooled entry a query at position p sees (-1: none); it grows with p
+    auto last_pooled = [&](int p) { return p >= 0 && p + 1 - window >= pool ? (p + 1 - window) / pool - 1 : -1; };
+    int pos[2], lo[2], hd[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         int rr = tile_row0 + warp * 16 + (lane >> 2) + h * 8;
         pos[h] = rr < total_rows ? ctx + rr / G : -1;
         hd[h] = rr < total_rows ? kvh * G + rr % G : -1;
         lo[h] = first_key(pos[h], window, chunk);
-        // the last pooled entry this row sees (-1: none)
-        pos_p[h] = pool > 0 && pos[h] >= 0 && pos[h] + 1 - window >= pool ? (pos[h] + 1 - window) / pool - 1 : -1;
     }
     RowShape rs;
     if (SHAPED) rs = row_shape(shape, hd[0], hd[1]);
     int warp_last_pos = max(pos[0], pos[1]), warp_first_pos = min(pos[0], pos[1]), warp_max_lo = max(lo[0], lo[1]);
     int warp_min_lo = 0;                             // blocks of positions: the first key any row of the warp reads
     if (SHAPED) warp_min_lo = min(pos[0] < 0 ? 0x7fffffff : lo[0], pos[1] < 0 ? 0x7fffffff : lo[1]);
-    int warp_last_p = max(pos_p[0], pos_p[1]), warp_first_p = min(pos_p[0], pos_p[1]);
 #pragma unroll
     for (int x = 4; x < 32; x <<= 1) {
         warp_last_pos = max(warp_last_pos, __shfl_xor_sync(0xffffffffu, warp_last_pos, x));
         warp_first_pos = min(warp_first_pos, __shfl_xor_sync(0xffffffffu, warp_first_pos, x));
         warp_max_lo = max(warp_max_lo, __shfl_xor_sync(0xffffffffu, warp_max_lo, x));
         if (SHAPED) warp_min_lo = min(warp_min_lo, __shfl_xor_sync(0xffffffffu, warp_min_lo, x));
-        if (SHAPED) warp_last_p = max(warp_last_p, __shfl_xor_sync(0xffffffffu, warp_last_p, x));
-        if (SHAPED) warp_first_p = min(warp_first_p, __shfl_xor_sync(0xffffffffu, warp_first_p, x));
     }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     float o[HDV / 8][4];
@@ -504,18 +542,26 @@ attn_prefill_mma_any_kernel(const __nv_bfloat16* __restrict__ q, long long q_str
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
     uint32_t qf[HD / 16][4];
-    // One walk over key tiles with one running softmax: first the tiles of pooled entries (where there are any), then the
-    // tiles of tokens. Both page lists sit in shared memory, the tokens' first.
-    const int tp_end = (hi_pool + BN - 1) / BN;
+    // One walk over key tiles with one running softmax: first the tiles of pooled entries or of kept first tokens (where
+    // there are any, and not the tiles the window reaches itself), then the tiles of tokens. Both page lists sit in shared
+    // memory, the tokens' first.
     const int t_begin = lo_blk / BN, t_end = (hi + BN - 1) / BN;
-    const int page0 = lo_blk >> page_shift, page_end = ((hi - 1) >> page_shift) + 1;
+    const int keep = KV1 ? shape.keep : 0;
+    const int tp_end = KV1 ? min((keep + BN - 1) / BN, t_begin) : (hi_pool + BN - 1) / BN;
+    const int page0 = (t_begin * BN) >> page_shift, page_end = ((hi - 1) >> page_shift) + 1;
     int* s_pages_p = s_pages + (page_end - page0);
-    const int pages_p = hi_pool > 0 ? ((hi_pool - 1) >> page_shift) + 1 : 0;
+    const int pages_p = KV1 ? (tp_end * BN) >> page_shift : hi_pool > 0 ? ((hi_pool - 1) >> page_shift) + 1 : 0;
     for (int i = threadIdx.x; i < page_end - page0 + pages_p; i += NTHREADS) s_pages[i] = i < page_end - page0 ? bt[page0 + i] : bt[i - (page_end - page0)];
     __syncthreads();
     const int n_it = tp_end + (t_end - t_begin);
     auto load_tile = [&](int it, int buf) {
-        if (SHAPED && it < tp_end) {
+        if (KV1) {
+            const bool kept = it < tp_end;
+            const int t = kept ? it : t_begin + it - tp_end, lo_t = kept ? 0 : lo_blk, hi_t = kept ? keep : hi, p0 = kept ? 0 : page0;
+            const int* pages = kept ? s_pages_p : s_pages;
+            load_rows_padded<HD>(sK0 + buf * BN * LD, kc, D, pages, p0, kvh, KV, page_shift, t * BN, lo_t, hi_t, keep);
+            load_key_scales(sR0 + buf * BN, shape.kscale, pages, p0, page_shift, t * BN, lo_t, hi_t, keep);
+        } else if (SHAPED && it < tp_end) {
             load_rows_padded<HD>(sK0 + buf * BN * LD, shape.kp, D, s_pages_p, 0, kvh, KV, page_shift, it * BN, 0, hi_pool);
             load_rows_padded<HDV>(sV0 + buf * BN * LDV, shape.vp, DV, s_pages_p, 0, kvh, KV, page_shift, it * BN, 0, hi_pool);
         } else {
@@ -538,20 +584,22 @@ attn_prefill_mma_any_kernel(const __nv_bfloat16* __restrict__ q, long long q_str
             for (int kk = 0; kk < HD / 16; ++kk)
                 ldmatrix_x4(qf[kk], sQ + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LD + kk * 16 + (lane >> 4) * 8);
         }
-        const bool pooled = SHAPED && it < tp_end;
-        const int t = pooled ? it : t_begin + it - tp_end;
-        const int w_last = pooled ? warp_last_p : warp_last_pos, w_first = pooled ? warp_first_p : warp_first_pos;
+        const bool pooled = SHAPED && !KV1 && it < tp_end;
+        const int t = SHAPED && it < tp_end ? it : t_begin + it - tp_end;
+        const int w_last = pooled ? last_pooled(warp_last_pos) : warp_last_pos, w_first = pooled ? last_pooled(warp_first_pos) : warp_first_pos;
         const int w_max_lo = pooled ? 0 : warp_max_lo, w_min_lo = pooled ? 0 : warp_min_lo;
-        const int lo_r[2] = {pooled ? 0 : lo[0], pooled ? 0 : lo[1]}, pos_r[2] = {pooled ? pos_p[0] : pos[0], pooled ? pos_p[1] : pos[1]};
+        const int lo_r[2] = {pooled ? 0 : lo[0], pooled ? 0 : lo[1]}, pos_r[2] = {pooled ? last_pooled(pos[0]) : pos[0], pooled ? last_pooled(pos[1]) : pos[1]};
         // a tile behind the warp's last key needs no work, nor has one whose rows all begin to read behind this tile's last key
-        if (t * BN <= w_last && (!SHAPED || (t + 1) * BN > w_min_lo)) {
+        // (unless it holds kept first tokens)
+        if (t * BN <= w_last && (!SHAPED || (t + 1) * BN > w_min_lo || (KV1 && t * BN < keep))) {
             float s[8][4];
             qk_tile<HD, 8>(s, qf, sK, 0);
             uint32_t pa[4][4];
-            if ((t + 1) * BN - 1 <= w_first && t * BN >= w_max_lo)
-                softmax_step<8, HDV / 8, false, SHAPED>(s, pa, o, m, l, t * BN, lo_r, pos_r, scale_log2, &shape, &rs);
+            const float* ksc = sR0 + buf * BN;
+            if ((t + 1) * BN - 1 <= w_first && (t * BN >= w_max_lo || (KV1 && (t + 1) * BN <= keep)))
+                softmax_step<8, HDV / 8, false, SHAPED, KV1>(s, pa, o, m, l, t * BN, lo_r, pos_r, scale_log2, &shape, &rs, ksc);
             else
-                softmax_step<8, HDV / 8, true, SHAPED>(s, pa, o, m, l, t * BN, lo_r, pos_r, scale_log2, &shape, &rs);
+                softmax_step<8, HDV / 8, true, SHAPED, KV1>(s, pa, o, m, l, t * BN, lo_r, pos_r, scale_log2, &shape, &rs, ksc);
             pv_tile<HDV, 4>(o, pa, sV, 0);
         }
     }
@@ -571,8 +619,8 @@ attn_prefill_mma_any_kernel(const __nv_bfloat16* __restrict__ q, long long q_str
 #pragma unroll
         for (int n = 0; n < HDV / 8; ++n)
             if (n * 8 + (lane & 3) * 2 < DV)
-                *reinterpret_cast<uint32_t*>(op + n * 8) = pack_bf16(tail_val(tail, row0 + tok, col + n * 8, o[n][2 * h] * inv),
-                                                                     tail_val(tail, row0 + tok, col + n * 8 + 1, o[n][2 * h + 1] * inv));
+                *reinterpret_cast<uint32_t*>(op + n * 8) = pack_bf16(tail_val(tail, row0 + tok, head, col + n * 8, o[n][2 * h] * inv),
+                                                                     tail_val(tail, row0 + tok, head, col + n * 8 + 1, o[n][2 * h + 1] * inv));
     }
 }
 
@@ -626,7 +674,7 @@ __device__ __noinline__ void merge_partials(const float* __restrict__ all, int s
     __syncthreads();
     for (int e = threadIdx.x; e < G * HD; e += NTHREADS) {
         const float L = Lrow[e / HD];
-        out[e] = __float2bfloat16_rn(L > 0.f ? tail_val(tail, row, head0 * HD + e, (hs[e] + hs[16 * HD + e]) / L) : 0.f);
+        out[e] = __float2bfloat16_rn(L > 0.f ? tail_val(tail, row, head0 + e / HD, head0 * HD + e, (hs[e] + hs[16 * HD + e]) / L) : 0.f);
     }
 }
 
@@ -653,14 +701,16 @@ __device__ __noinline__ void merge_partials(const float* __restrict__ all, int s
 
 // Shared memory of a decode block: the K/V ring (used again for the combine of the four warps),
 // then what the cluster's peers send, then the block's page list.
-template <int HD, int DEC_STAGES> __host__ __device__ constexpr size_t decode_ring_bytes() {
-    size_t ring = (size_t)(16 + 2 * DEC_STAGES * BN) * (HD + 8) * sizeof(__nv_bfloat16);
+template <int HD, int DEC_STAGES, bool KV1> __host__ __device__ constexpr size_t decode_ring_bytes() {
+    size_t ring = (size_t)(16 + (KV1 ? 1 : 2) * DEC_STAGES * BN) * (HD + 8) * sizeof(__nv_bfloat16) + (KV1 ? DEC_STAGES * BN * sizeof(float) : 0);
     size_t combine = 16 * (HD + 8) * sizeof(__nv_bfloat16) + (size_t)(128 + 4 * 16 * HD + 16 * HD + 32) * sizeof(float);
     return ((ring > combine ? ring : combine) + 15) / 16 * 16;
 }
 __host__ __device__ constexpr size_t decode_recv_bytes(int G, int HD) { return (size_t)(G * HD + 8 + 256) * sizeof(float); }
 
-template <int HD, int DEC_STAGES, bool SHAPED>
+// KV1: the values are the cached keys; the ring holds one tile a stage, which serves both products, and a number per key.
+// Kept first tokens (ScoreShape::keep): their tiles come first in a request's list of tiles, in front of the window's.
+template <int HD, int DEC_STAGES, bool SHAPED, bool KV1>
 __global__ void __launch_bounds__(NTHREADS)
 attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, __nv_bfloat16* __restrict__ out,
                        long long out_stride, const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc,
@@ -674,9 +724,10 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
     __shared__ int s_last;
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem_raw);            // 16 x LD
     __nv_bfloat16* sK0 = sQ + 16 * LD;                                          // DEC_STAGES x BN x LD
-    __nv_bfloat16* sV0 = sK0 + DEC_STAGES * BN * LD;
+    __nv_bfloat16* sV0 = KV1 ? sK0 : sK0 + DEC_STAGES * BN * LD;
+    float* sR0 = reinterpret_cast<float*>(sK0 + DEC_STAGES * BN * LD);          // KV1: DEC_STAGES x BN numbers
     // what the peers of a cluster send this block: [splits][chunk] values, [8][16] maxima, [8][16] sums
-    float* recv_val = reinterpret_cast<float*>(smem_raw + decode_ring_bytes<HD, DEC_STAGES>());
+    float* recv_val = reinterpret_cast<float*>(smem_raw + decode_ring_bytes<HD, DEC_STAGES, KV1>());
     float* recv_m = recv_val + (H / KV) * HD + 8;
     float* recv_l = recv_m + 128;
     // this block's pages (a launch without a cluster has no region for what peers send)
@@ -697,7 +748,11 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
     const int hi = p + 1;
     const int lo_key = first_key(p, window, SHAPED ? shape.chunk : 0);
     const int t_first = lo_key / BN;
-    const int n_tiles = p >= 0 ? (hi + BN - 1) / BN - t_first : 0;
+    const int keep = SHAPED ? shape.keep : 0;
+    const int kt = SHAPED ? min((keep + BN - 1) / BN, t_first) : 0;      // tiles of kept first tokens in front of the window's
+    const int n_tiles = p >= 0 ? (hi + BN - 1) / BN - t_first + kt : 0;
+    // the request's tile number n (0 .. n_tiles - 1) holds the keys from BN * tile_of(n) on
+    auto tile_of = [&](int n) { return SHAPED && n < kt ? n : t_first + n - kt; };
     if (partials) {
         splits = max(1, min(splits, n_tiles / DEC_MIN_TILES));
         const int share = max(1, (n_tiles + splits - 1) / splits);
@@ -705,23 +760,30 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
         if (split >= splits) return;                  // the whole block: this request has no tiles for it
     }
     const int per = (n_tiles + splits - 1) / splits;
-    const int t_begin = t_first + split * per;
-    const int t_end = min(t_first + n_tiles, t_begin + per);
-    // this block's pages: those of its tiles, one coalesced read of the block table
-    const int page0 = (t_begin * BN) >> page_shift;
-    const int page_end = t_begin < t_end ? ((min(hi, t_end * BN) - 1) >> page_shift) + 1 : page0;
-    for (int i = threadIdx.x; i < page_end - page0; i += NTHREADS) s_pages[i] = bt[page0 + i];
+    const int n_begin = split * per;
+    const int n_end = min(n_tiles, n_begin + per);
+    // this block's pages: those of its tiles, BN / page_size of them each, one coalesced read of the block table
+    const int ppt_shift = 6 - page_shift;
+    for (int i = threadIdx.x; i < (max(n_end - n_begin, 0) << ppt_shift); i += NTHREADS) {
+        const int lp = (tile_of(n_begin + (i >> ppt_shift)) << ppt_shift) + (i & ((1 << ppt_shift) - 1));
+        s_pages[i] = lp <= (hi - 1) >> page_shift ? bt[lp] : 0;
+    }
     __syncthreads();
+    auto load_tile = [&](int n, int buf) {
+        const int t = tile_of(n);
+        const int* pages = s_pages + ((n - n_begin) << ppt_shift);
+        load_kv_tile<HD, !KV1>(sK0 + buf * BN * LD, sV0 + buf * BN * LD, kc, vc, pages, t << ppt_shift, kvh, KV, page_shift, t * BN, lo_key, hi, keep);
+        if (KV1) load_key_scales(sR0 + buf * BN, shape.kscale, pages, t << ppt_shift, page_shift, t * BN, lo_key, hi, keep);
+    };
 
     // prologue: the first DEC_STAGES - 1 tiles, one commit group each (empty groups keep the
     // count); tiles that end before the newest key go out before the wait, the rest after it
     int s_done = 0;
 #pragma unroll
     for (int s = 0; s < DEC_STAGES - 1; ++s) {
-        int t = t_begin + s;
-        if (s_done == s && (t >= t_end || (t + 1) * BN <= p)) {
-            if (t < t_end)
-                load_kv_tile<HD>(sK0 + s * BN * LD, sV0 + s * BN * LD, kc, vc, s_pages, page0, kvh, KV, page_shift, t * BN, lo_key, hi);
+        int n = n_begin + s;
+        if (s_done == s && (n >= n_end || (tile_of(n) + 1) * BN <= p)) {
+            if (n < n_end) load_tile(n, s);
             cp_async_commit();
             s_done = s + 1;
         }
@@ -738,9 +800,8 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
 #pragma unroll
     for (int s = 0; s < DEC_STAGES - 1; ++s) {
         if (s >= s_done) {
-            int t = t_begin + s;
-            if (t < t_end)
-                load_kv_tile<HD>(sK0 + s * BN * LD, sV0 + s * BN * LD, kc, vc, s_pages, page0, kvh, KV, page_shift, t * BN, lo_key, hi);
+            int n = n_begin + s;
+            if (n < n_end) load_tile(n, s);
             cp_async_commit();
         }
     }
@@ -765,20 +826,19 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
         for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
     uint32_t qf[HD / 16][4];
 
-    for (int t = t_begin; t < t_end; ++t) {
-        int buf = (t - t_begin) % DEC_STAGES;
+    for (int n = n_begin; n < n_end; ++n) {
+        const int t = tile_of(n);
+        int buf = (n - n_begin) % DEC_STAGES;
         __nv_bfloat16* sK = sK0 + buf * BN * LD;
         __nv_bfloat16* sV = sV0 + buf * BN * LD;
-        cp_async_wait<DEC_STAGES - 2>();        // tile t has landed (one newer group may be in flight)
-        __syncthreads();                        // ... for every thread; and everyone is done with tile t-1
+        cp_async_wait<DEC_STAGES - 2>();        // tile n has landed (one newer group may be in flight)
+        __syncthreads();                        // ... for every thread; and everyone is done with tile n-1
         {
-            int tn = t + DEC_STAGES - 1;        // refill the buffer tile t-1 used
-            int nb = (tn - t_begin) % DEC_STAGES;
-            if (tn < t_end)
-                load_kv_tile<HD>(sK0 + nb * BN * LD, sV0 + nb * BN * LD, kc, vc, s_pages, page0, kvh, KV, page_shift, tn * BN, lo_key, hi);
+            int nn = n + DEC_STAGES - 1;        // refill the buffer tile n-1 used
+            if (nn < n_end) load_tile(nn, (nn - n_begin) % DEC_STAGES);
             cp_async_commit();
         }
-        if (t == t_begin) {
+        if (n == n_begin) {
 #pragma unroll
             for (int kk = 0; kk < HD / 16; ++kk)
                 ldmatrix_x4(qf[kk], sQ + ((lane & 7) + ((lane >> 3) & 1) * 8) * LD + kk * 16 + (lane >> 4) * 8);
@@ -786,7 +846,8 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
         float s[2][4];
         qk_tile<HD, 2>(s, qf, sK, warp * 2);                    // this warp's 16 keys of the tile
         uint32_t pa[1][4];
-        softmax_step<2, HD / 8, true, SHAPED>(s, pa, o, m, l, t * BN + warp * 16, lo, pos, scale_log2, &shape, &rs);
+        softmax_step<2, HD / 8, true, SHAPED, KV1, SHAPED>(s, pa, o, m, l, t * BN + warp * 16, lo, pos, scale_log2, &shape, &rs,
+                                                   sR0 + buf * BN + warp * 16);
         pv_tile<HD, 1>(o, pa, sV, warp);
     }
     cp_async_wait<0>();
@@ -828,7 +889,7 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
         if (splits == 1) {
             L = tail_den(tail, kvh * G + r, L, Ms);
             out[(size_t)seq * out_stride + (size_t)(kvh * G + r) * HD + d] =
-                __float2bfloat16_rn(L > 0.f ? tail_val(tail, seq, (kvh * G + r) * HD + d, acc / L) : 0.f);
+                __float2bfloat16_rn(L > 0.f ? tail_val(tail, seq, kvh * G + r, (kvh * G + r) * HD + d, acc / L) : 0.f);
         } else if (push) {
             // to the block that finishes this output; the row's maximum and sum to every block
             const int owner = e / chunk;
@@ -887,15 +948,15 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
             }
             L = tail_den(tail, kvh * G + r, L, Ms);
             out[(size_t)seq * out_stride + (size_t)(kvh * G + r) * HD + d] =
-                __float2bfloat16_rn(L > 0.f ? tail_val(tail, seq, (kvh * G + r) * HD + d, acc / L) : 0.f);
+                __float2bfloat16_rn(L > 0.f ? tail_val(tail, seq, kvh * G + r, (kvh * G + r) * HD + d, acc / L) : 0.f);
         }
         // nothing of this block is read by a peer: it may leave at once
     }
 }
 
 template <int HD> constexpr size_t prefill_smem() { return (size_t)(64 + 4 * BN) * (HD + 8) * sizeof(__nv_bfloat16); }
-template <int HD, int DEC_STAGES> size_t decode_smem(int G, bool cluster) {
-    return decode_ring_bytes<HD, DEC_STAGES>() + (cluster ? decode_recv_bytes(G, HD) : 0);
+template <int HD, int DEC_STAGES, bool KV1> size_t decode_smem(int G, bool cluster) {
+    return decode_ring_bytes<HD, DEC_STAGES, KV1>() + (cluster ? decode_recv_bytes(G, HD) : 0);
 }
 
 inline int log2_exact(int v) {
@@ -934,7 +995,7 @@ int launch_prefill(const void* q, long long q_stride, void* out, long long out_s
         scale * 1.4426950408889634f, tail);
 }
 
-template <int HD, int ST, bool SHAPED>
+template <int HD, int ST, bool SHAPED, bool KV1>
 int launch_decode_st(const void* q, long long q_stride, void* out, long long out_stride, const void* kc, const void* vc,
                      const int* bt, int max_pages, const int* positions, int S, int H, int KV, int page_size, int window,
                      float scale, int splits, float* partials, int* arrived, AttnTail tail, ScoreShape shape, cudaStream_t stream) {
@@ -945,8 +1006,8 @@ int launch_decode_st(const void* q, long long q_stride, void* out, long long out
     long long per_max = (tiles_max + splits - 1) / splits;
     if (partials && per_max < 2 * DEC_MIN_TILES) per_max = 2 * DEC_MIN_TILES;
     long long pages_cta = per_max * (BN / page_size) + 1;
-    size_t smem = decode_smem<HD, ST>(H / KV, splits > 1 && !partials) + (size_t)pages_cta * sizeof(int);
-    int e = ensure_smem(attn_decode_mma_kernel<HD, ST, SHAPED>, smem, &configured);
+    size_t smem = decode_smem<HD, ST, KV1>(H / KV, splits > 1 && !partials) + (size_t)pages_cta * sizeof(int);
+    int e = ensure_smem(attn_decode_mma_kernel<HD, ST, SHAPED, KV1>, smem, &configured);
     if (e) return e;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(S, KV, splits);
@@ -962,13 +1023,13 @@ int launch_decode_st(const void* q, long long q_stride, void* out, long long out
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = g_vob_pdl ? 2 : 1;
-    cudaError_t ce = cudaLaunchKernelEx(&cfg, attn_decode_mma_kernel<HD, ST, SHAPED>, (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out,
+    cudaError_t ce = cudaLaunchKernelEx(&cfg, attn_decode_mma_kernel<HD, ST, SHAPED, KV1>, (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out,
                                         out_stride, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, bt, max_pages, positions,
                                         H, KV, log2_exact(page_size), window, scale * 1.4426950408889634f, partials, arrived, tail, shape);
     return ce != cudaSuccess ? (int)ce : vob_launch_status();
 }
 
-template <int HD, bool SHAPED>
+template <int HD, bool SHAPED, bool KV1 = false>
 int launch_decode(const void* q, long long q_stride, void* out, long long out_stride, const void* kc, const void* vc,
                   const int* bt, int max_pages, const int* positions, int S, int H, int KV, int page_size, int window,
                   float scale, int splits, float* partials, int* arrived, AttnTail tail, ScoreShape shape, cudaStream_t stream) {
@@ -981,27 +1042,28 @@ int launch_decode(const void* q, long long q_stride, void* out, long long out_st
     }
     // three stages while every block of the grid can be resident at once with them; else two
     long long blocks = (long long)S * KV * splits;
-    long long fit3 = (long long)num_sms * ((227 * 1024) / (long long)(decode_smem<HD, 3>(H / KV, splits > 1 && !partials) + 2048));
+    long long fit3 = (long long)num_sms * ((227 * 1024) / (long long)(decode_smem<HD, 3, KV1>(H / KV, splits > 1 && !partials) + 2048));
     if (blocks <= fit3)
-        return launch_decode_st<HD, 3, SHAPED>(q, q_stride, out, out_stride, kc, vc, bt, max_pages, positions, S, H, KV, page_size,
+        return launch_decode_st<HD, 3, SHAPED, KV1>(q, q_stride, out, out_stride, kc, vc, bt, max_pages, positions, S, H, KV, page_size,
                                                window, scale, splits, partials, arrived, tail, shape, stream);
-    return launch_decode_st<HD, 2, SHAPED>(q, q_stride, out, out_stride, kc, vc, bt, max_pages, positions, S, H, KV, page_size,
+    return launch_decode_st<HD, 2, SHAPED, KV1>(q, q_stride, out, out_stride, kc, vc, bt, max_pages, positions, S, H, KV, page_size,
                                            window, scale, splits, partials, arrived, tail, shape, stream);
 }
 
-template <int HD, int HDV, bool SHAPED>
+template <int HD, int HDV, bool SHAPED, bool KV1>
 int launch_prefill_any(const void* q, long long q_stride, void* out, long long out_stride, const void* kc, const void* vc,
                        const int* bt, int max_pages, const int* seq_starts, const int* context_lens, int S, int max_new,
                        int H, int KV, int D, int DV, int page_size, int window, float scale, AttnTail tail, ScoreShape shape,
                        cudaStream_t stream) {
     static size_t configured = 0;
-    size_t smem = ((size_t)(64 + 2 * BN) * (HD + 8) + (size_t)2 * BN * (HDV + 8)) * sizeof(__nv_bfloat16) + (size_t)2 * max_pages * sizeof(int);
-    int e = ensure_smem(attn_prefill_mma_any_kernel<HD, HDV, SHAPED>, smem, &configured);
+    size_t smem = ((size_t)(64 + 2 * BN) * (HD + 8) + (KV1 ? (size_t)0 : (size_t)2 * BN * (HDV + 8))) * sizeof(__nv_bfloat16) +
+                  (KV1 ? 2 * BN * sizeof(float) : 0) + (size_t)2 * max_pages * sizeof(int);
+    int e = ensure_smem(attn_prefill_mma_any_kernel<HD, HDV, SHAPED, KV1>, smem, &configured);
     if (e) return e;
     const long long row_tiles = ((long long)max_new * (H / KV) + 63) / 64;
     if (row_tiles > 65535) return VOB_ERR_UNSUPPORTED;
     dim3 grid(KV, S, (unsigned)row_tiles);
-    return vob_launch(attn_prefill_mma_any_kernel<HD, HDV, SHAPED>, grid, dim3(NTHREADS), smem, stream,
+    return vob_launch(attn_prefill_mma_any_kernel<HD, HDV, SHAPED, KV1>, grid, dim3(NTHREADS), smem, stream,
         (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)kc,
         (const __nv_bfloat16*)vc, bt, max_pages, seq_starts, context_lens, H, KV, D, DV, log2_exact(page_size), window,
         scale * 1.4426950408889634f, tail, shape);
@@ -1020,8 +1082,21 @@ int prefill_any(const void* q, long long q_stride, void* out, long long out_stri
     if (KV <= 0 || H % KV != 0 || page_size <= 0 || BN % page_size != 0) return VOB_ERR_UNSUPPORTED;
     if (D <= 0 || DV <= 0 || D % 8 != 0 || DV % 8 != 0 || D > 128 || DV > 128) return VOB_ERR_UNSUPPORTED;
     if (q_stride % 8 != 0 || out_stride % 2 != 0 || S > 65535 || KV > 65535) return VOB_ERR_BAD_ARG;
+    if (shape.keep > 0 && kcache != vcache) return VOB_ERR_UNSUPPORTED;
+    if (SHAPED && kcache == vcache) {          // the values are the cached keys
+        if (D != DV || shape.pool > 0) return VOB_ERR_BAD_ARG;
+#define VOB_KV1(HD_)                                                                                                                \
+    return launch_prefill_any<HD_, HD_, true, true>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages,           \
+                                                    seq_starts, context_lens, S, max_new, H, KV, D, DV, page_size, window, scale,    \
+                                                    tail, shape, stream)
+        if (D <= 32) VOB_KV1(32);
+        if (D <= 64) VOB_KV1(64);
+        if (D <= 96) VOB_KV1(96);
+        VOB_KV1(128);
+#undef VOB_KV1
+    }
 #define VOB_ANY(HD_, HDV_)                                                                                                          \
-    return launch_prefill_any<HD_, HDV_, SHAPED>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, seq_starts,  \
+    return launch_prefill_any<HD_, HDV_, SHAPED, false>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, seq_starts,  \
                                                  context_lens, S, max_new, H, KV, D, DV, page_size, window, scale, tail, shape, stream)
 #define VOB_ANY_V(HD_)                                                                                                              \
     do {                                                                                                                            \
@@ -1051,7 +1126,7 @@ VOB_EXPORT int vob_attn_prefill_mma(const void* q, long long q_stride, void* out
                                     const int* context_lens, int S, int max_new, int H, int KV, int hd, int page_size,
                                     int window, float scale, const float* sink, const void* gate, long long gate_stride,
                                     float out_scale, cudaStream_t stream) {
-    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale};
+    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale, 0};
     if (S <= 0 || max_new <= 0) return 0;
     if (!sizes_ok(H, KV, hd, page_size)) return VOB_ERR_UNSUPPORTED;
     if (q_stride % 8 != 0 || out_stride % 2 != 0 || S > 65535 || KV > 65535) return VOB_ERR_BAD_ARG;
@@ -1068,27 +1143,40 @@ VOB_EXPORT int vob_attn_prefill_mma_any(const void* q, long long q_stride, void*
                                         const int* context_lens, int S, int max_new, int H, int KV, int D, int DV, int page_size,
                                         int window, float scale, const float* sink, const void* gate, long long gate_stride,
                                         float out_scale, cudaStream_t stream) {
-    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale};
+    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale, 0};
     return prefill_any<false>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, seq_starts, context_lens, S, max_new,
                               H, KV, D, DV, page_size, window, scale, tail, make_shape(0, 0.f, nullptr, nullptr, scale), stream);
 }
 
+// The checked arguments of the shaped forms. r1 without r2: a linear bias. `keep` goes with a window; `kscale` with values
+// that are the cached keys (kcache == vcache).
+static int shape_args_ok(int chunk, float softcap, const float* r1, const float* r2, int keep, int window, const float* kscale,
+                         const void* kcache, const void* vcache) {
+    if (chunk < 0 || softcap < 0.f || (r2 && !r1)) return 0;
+    if (keep < 0 || (keep > 0 && (window <= 0 || chunk > 0))) return 0;
+    if (kscale && kcache != vcache) return 0;
+    return 1;
+}
+
 // The same with scores that are shaped before the softmax: a query reads the keys of its own block of `chunk` positions
 // (0: no blocks), score <- softcap * tanh(score / softcap) (0: no cap), r1[head] * ln(1 + r2[head] * distance) is taken
-// off (r1, r2 float32 [H], or both null). Any sign of `scale`.
+// off (r1, r2 float32 [H], or both null), or r1[head] * distance (r2 null). Any sign of `scale`. `keep`: the first so many keys are
+// seen whatever the window. kcache == vcache: the values are the cached keys, q . k is multiplied by kscale [pages][page_size]
+// (null: by nothing). `gate_heads`: the gate has one column per head.
 VOB_EXPORT int vob_attn_prefill_shaped(const void* q, long long q_stride, void* out, long long out_stride, const void* kcache,
                                        const void* vcache, const int* block_tables, int max_pages, const int* seq_starts,
                                        const int* context_lens, int S, int max_new, int H, int KV, int D, int DV, int page_size,
                                        int window, float scale, const float* sink, const void* gate, long long gate_stride,
                                        float out_scale, int chunk, float softcap, const float* r1, const float* r2,
-                                       const void* kpool, const void* vpool, int pool, cudaStream_t stream) {
-    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale};
-    if (chunk < 0 || softcap < 0.f || (r1 != nullptr) != (r2 != nullptr)) return VOB_ERR_BAD_ARG;
+                                       const void* kpool, const void* vpool, int pool, int keep, const float* kscale, int gate_heads,
+                                       cudaStream_t stream) {
+    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale, gate_heads};
+    if (!shape_args_ok(chunk, softcap, r1, r2, keep, window, kscale, kcache, vcache)) return VOB_ERR_BAD_ARG;
     // pooled entries (kpool, vpool laid out like the caches, `pool` tokens an entry) go with a window, without blocks of
     // positions and without a distance bias
     if (pool < 0 || (pool > 0) != (kpool != nullptr) || (kpool != nullptr) != (vpool != nullptr)) return VOB_ERR_BAD_ARG;
-    if (pool > 0 && (window <= 0 || chunk > 0 || r1)) return VOB_ERR_BAD_ARG;
-    const ScoreShape shape = make_shape(chunk, softcap, r1, r2, scale, kpool, vpool, pool);
+    if (pool > 0 && (window <= 0 || chunk > 0 || r1 || keep > 0)) return VOB_ERR_BAD_ARG;
+    const ScoreShape shape = make_shape(chunk, softcap, r1, r2, scale, kpool, vpool, pool, keep, r1 && !r2, kscale);
     return prefill_any<true>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, seq_starts, context_lens, S, max_new,
                              H, KV, D, DV, page_size, window, scale, tail, shape, stream);
 }
@@ -1101,7 +1189,7 @@ VOB_EXPORT int vob_attn_decode_mma(const void* q, long long q_stride, void* out,
                                    int H, int KV, int hd, int page_size, int window, float scale, int splits,
                                    void* partials, int* arrived, const float* sink, const void* gate, long long gate_stride,
                                    float out_scale, cudaStream_t stream) {
-    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale};
+    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale, 0};
     const ScoreShape none = make_shape(0, 0.f, nullptr, nullptr, scale);
     if (S <= 0) return 0;
     if (!sizes_ok(H, KV, hd, page_size) || H / KV > 16) return VOB_ERR_UNSUPPORTED;
@@ -1119,14 +1207,20 @@ VOB_EXPORT int vob_attn_decode_shaped(const void* q, long long q_stride, void* o
                                       int H, int KV, int hd, int page_size, int window, float scale, int splits,
                                       void* partials, int* arrived, const float* sink, const void* gate, long long gate_stride,
                                       float out_scale, int chunk, float softcap, const float* r1, const float* r2,
-                                      cudaStream_t stream) {
-    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale};
+                                      int keep, const float* kscale, int gate_heads, cudaStream_t stream) {
+    const AttnTail tail{sink, (const __nv_bfloat16*)gate, gate_stride, out_scale, gate_heads};
     if (S <= 0) return 0;
-    if (chunk < 0 || softcap < 0.f || (r1 != nullptr) != (r2 != nullptr)) return VOB_ERR_BAD_ARG;
-    const ScoreShape shape = make_shape(chunk, softcap, r1, r2, scale);
+    if (!shape_args_ok(chunk, softcap, r1, r2, keep, window, kscale, kcache, vcache)) return VOB_ERR_BAD_ARG;
+    const ScoreShape shape = make_shape(chunk, softcap, r1, r2, scale, nullptr, nullptr, 0, keep, r1 && !r2, kscale);
     if (!sizes_ok(H, KV, hd, page_size) || H / KV > 16) return VOB_ERR_UNSUPPORTED;
     if ((partials == nullptr) != (arrived == nullptr)) return VOB_ERR_BAD_ARG;
     if (q_stride % 8 != 0 || splits < 1 || splits > (partials ? DEC_MAX_SPLITS_WIDE : 8) || KV > 65535) return VOB_ERR_BAD_ARG;
+    if (kcache == vcache) {                    // the values are the cached keys
+        if (hd == 64) return launch_decode<64, true, true>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, positions, S,
+                                                          H, KV, page_size, window, scale, splits, (float*)partials, arrived, tail, shape, stream);
+        return launch_decode<128, true, true>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, positions, S, H, KV,
+                                              page_size, window, scale, splits, (float*)partials, arrived, tail, shape, stream);
+    }
     if (hd == 64) return launch_decode<64, true>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, positions, S,
                                                 H, KV, page_size, window, scale, splits, (float*)partials, arrived, tail, shape, stream);
     return launch_decode<128, true>(q, q_stride, out, out_stride, kcache, vcache, block_tables, max_pages, positions, S, H, KV,

@@ -900,6 +900,133 @@ VOB_EXPORT int vob_layernorm_tail(float* resid, const void* delta, int delta_cod
 }
 
 // ---------------------------------------------------------------------------------------------
+// Residual add + layer norm, for blocks whose norms sit in front of their sub-layers:
+//   x = resid[src] (+ delta[src] * mult);   without a row list: resid[src] = x  (the residual sum, float32)
+//   out[r] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w (+ b)
+// The mean first, then the mean of the squared deviations. Launch: one block of 256 threads per output row. NV > 0: rows
+// whose width is a multiple of 4 and fits NV float4 per thread stay in registers (every load is issued before anything
+// depends on one); NV == 0: h floats of shared memory, any width. Partial sums per thread over its features in order, then
+// a fixed tree, so a row's value is the same in every batch. Bound: memory.
+// ---------------------------------------------------------------------------------------------
+template <typename TD, typename TO, int NV>
+__global__ void __launch_bounds__(256)
+add_layernorm_kernel(float* __restrict__ resid, const TD* __restrict__ delta, const float* __restrict__ weight,
+                     const float* __restrict__ bias, const int* __restrict__ rows, TO* __restrict__ out, int h, float eps, float mult) {
+    pdl_launch_dependents();
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[8];
+    const int r = blockIdx.x;
+    constexpr int N = NV > 0 ? NV : 1;
+    float4 w[N];
+    if (NV > 0) {                                  // weights are written by no kernel
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+            const int i = (threadIdx.x + 256 * k) * 4;
+            w[k] = i < h ? *reinterpret_cast<const float4*>(weight + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
+    pdl_wait(5);
+    const int src = rows ? rows[r] : r;
+    float* x = resid + (size_t)src * h;
+    const TD* d = delta ? delta + (size_t)src * h : nullptr;
+    TO* o = out + (size_t)r * h;
+    if (NV > 0) {
+        float4 v[N];
+        float s = 0.f;
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+            const int i = (threadIdx.x + 256 * k) * 4;
+            v[k] = i < h ? *reinterpret_cast<const float4*>(x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        if (d) {
+#pragma unroll
+            for (int k = 0; k < N; ++k) {
+                const int i = (threadIdx.x + 256 * k) * 4;
+                if (i < h) {
+                    float e[4];
+                    ld4_f<TD>(d + i, e);
+                    v[k].x = fmaf(e[0], mult, v[k].x); v[k].y = fmaf(e[1], mult, v[k].y);
+                    v[k].z = fmaf(e[2], mult, v[k].z); v[k].w = fmaf(e[3], mult, v[k].w);
+                    if (!rows) *reinterpret_cast<float4*>(x + i) = v[k];
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < N; ++k) { s += v[k].x; s += v[k].y; s += v[k].z; s += v[k].w; }     // absent features are zeros
+        const float mean = block_sum_256(s, red) / (float)h;
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+            if ((threadIdx.x + 256 * k) * 4 < h) {
+                v[k].x -= mean; v[k].y -= mean; v[k].z -= mean; v[k].w -= mean;
+                ss = fmaf(v[k].x, v[k].x, ss); ss = fmaf(v[k].y, v[k].y, ss);
+                ss = fmaf(v[k].z, v[k].z, ss); ss = fmaf(v[k].w, v[k].w, ss);
+            }
+        }
+        const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)h + eps);
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+            const int i = (threadIdx.x + 256 * k) * 4;
+            if (i < h) {
+                float y[4] = {v[k].x * inv * w[k].x, v[k].y * inv * w[k].y, v[k].z * inv * w[k].z, v[k].w * inv * w[k].w};
+                if (bias) {
+                    const float4 b = *reinterpret_cast<const float4*>(bias + i);
+                    y[0] += b.x; y[1] += b.y; y[2] += b.z; y[3] += b.w;
+                }
+                st4_f<TO>(o + i, y);
+            }
+        }
+    } else {
+        float s = 0.f;
+        for (int i = threadIdx.x; i < h; i += 256) {
+            float v = x[i];
+            if (d) {
+                v = fmaf(ld_f(d + i), mult, v);
+                if (!rows) x[i] = v;
+            }
+            row[i] = v;
+            s += v;
+        }
+        const float mean = block_sum_256(s, red) / (float)h;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < h; i += 256) {
+            const float c = row[i] - mean;
+            ss = fmaf(c, c, ss);
+        }
+        const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)h + eps);
+        for (int i = threadIdx.x; i < h; i += 256) st_f(o + i, (row[i] - mean) * inv * weight[i] + (bias ? bias[i] : 0.f));
+    }
+}
+
+template <typename TD, typename TO>
+static int launch_add_layernorm(float* resid, const void* delta, const float* weight, const float* bias, const int* rows, void* out, int R,
+                                int h, float eps, float mult, cudaStream_t stream) {
+    const bool by4 = h % 4 == 0 && ((((uintptr_t)resid) | ((uintptr_t)weight) | ((uintptr_t)bias) | ((uintptr_t)delta) | ((uintptr_t)out)) & 15) == 0;
+    const int nv = (h / 4 + 255) / 256;
+#define VOB_ALN(NV_) return vob_launch(add_layernorm_kernel<TD, TO, NV_>, dim3(R), dim3(256), NV_ ? 0 : (size_t)h * sizeof(float), stream, resid, \
+                                       (const TD*)delta, weight, bias, rows, (TO*)out, h, eps, mult)
+    if (by4 && nv <= 8) {
+        if (nv <= 1) VOB_ALN(1); else if (nv <= 2) VOB_ALN(2); else if (nv <= 4) VOB_ALN(4); else VOB_ALN(8);
+    }
+    if ((size_t)h * sizeof(float) > 48 * 1024) return VOB_ERR_UNSUPPORTED;
+    VOB_ALN(0);
+#undef VOB_ALN
+}
+
+VOB_EXPORT int vob_add_layernorm(float* resid, const void* delta, int delta_code, const float* weight, const float* bias, const int* rows,
+                                 void* out, int out_code, int R, int h, float eps, float mult, cudaStream_t stream) {
+    if (R <= 0) return 0;
+    if (h <= 0 || !weight || !out) return VOB_ERR_BAD_ARG;
+    if (!delta) delta_code = out_code;
+    if (delta_code == VOB_F32 && out_code == VOB_F32) return launch_add_layernorm<float, float>(resid, delta, weight, bias, rows, out, R, h, eps, mult, stream);
+    if (delta_code == VOB_BF16 && out_code == VOB_BF16)
+        return launch_add_layernorm<__nv_bfloat16, __nv_bfloat16>(resid, delta, weight, bias, rows, out, R, h, eps, mult, stream);
+    if (delta_code == VOB_F32 && out_code == VOB_BF16) return launch_add_layernorm<float, __nv_bfloat16>(resid, delta, weight, bias, rows, out, R, h, eps, mult, stream);
+    if (delta_code == VOB_BF16 && out_code == VOB_F32) return launch_add_layernorm<__nv_bfloat16, float>(resid, delta, weight, bias, rows, out, R, h, eps, mult, stream);
+    return VOB_ERR_BAD_ARG;
+}
+
+// ---------------------------------------------------------------------------------------------
 // The float32 residual in the activations' type: out[i] = in[i] (rounded to nearest even for bfloat16). What a
 // sub-layer that reads the residual itself is given where nothing before it has left such a copy.
 // ---------------------------------------------------------------------------------------------

@@ -4,10 +4,13 @@
 //                    all experts; the experts form `n_groups` runs of neighbours, a run scores as its best expert, only
 //                    experts of the `keep` best runs stand for election (n_groups <= 1: all do); the `top` experts with
 //                    the largest scores are chosen (a tie goes to the lower index), their weights are their own scores
-//                    (times 1 / their sum where `renorm` is set).
+//                    (divided by their sum + `eps` where `renorm` is set, times `out_scale`). Options (`RouteRule`): scores
+//                    s = sigmoid(z); the election (groups and experts) goes by s + correction[e] while the weights are
+//                    made of s; a run scores as the sum of its two best experts.
 //   vob_moe_align    the (token, choice) pairs put in order of their expert, every expert's run padded to whole tiles
 //                    of VOB_MOE_BM rows, with the expert of every tile.
 //   vob_moe_gate_up  per tile: h = act(W_gate[e] x) * (W_up[e] x) for the tile's pairs (x gathered by token).
+//   vob_moe_up       per tile: h = act(W_up[e] x), experts without a gate.
 //   vob_moe_down     per tile: y[pair] = weight[pair] * (W_down[e] h[pair]), float32.
 //   vob_moe_combine  out[token] = sum over the token's choices, in the order they were chosen, of y.
 //
@@ -49,10 +52,18 @@ template <> __device__ __forceinline__ void moe_ld4<__nv_bfloat16>(const __nv_bf
 // The block's four warps first share out the experts: a warp reads an expert's router row once and multiplies it with
 // the rows of all four tokens (a lane's chain runs over its own features in order, whoever the other tokens are; rows
 // whose width and addresses allow are read four features at a time). Then warp w holds the election of token w.
+struct RouteRule {
+    int sigmoid;               // scores: 0 softmax over all experts, 1 sigmoid of each logit
+    int group_best;            // a group's score: the sum of its best 1 or 2 choice scores
+    int renorm;                // weights divided by their sum + eps
+    const float* correction;   // [E] added to a score for the election only, or null
+    float eps, out_scale;
+};
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w_router, const int* __restrict__ positions,
-                 int T_rows, int width, int E, int top, int n_groups, int keep, int renorm, int* __restrict__ idx_out,
+                 int T_rows, int width, int E, int top, int n_groups, int keep, RouteRule rule, int* __restrict__ idx_out,
                  float* __restrict__ w_out) {
     pdl_launch_dependents();
     pdl_wait(71);
@@ -98,19 +109,23 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
         for (int k = lane; k < top; k += 32) { idx_out[(size_t)t * top + k] = -1; w_out[(size_t)t * top + k] = 0.f; }
         return;
     }
-    float* sc = sc_all + (size_t)warp * 2 * E;       // scores, then the working copy the election strikes names from
+    // the scores, then the choice scores the election strikes names from (-inf: does not stand)
+    float* sc = sc_all + (size_t)warp * 2 * E;
     float* cand = sc + E;
     __syncwarp();
-    float m = -INFINITY;
-    for (int e = lane; e < E; e += 32) m = fmaxf(m, sc[e]);
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) sum += expf(sc[e] - m);
-    sum = warp_sum(sum);
+    float m = 0.f, sum = 1.f;
+    if (!rule.sigmoid) {
+        m = -INFINITY;
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, sc[e]);
+        m = warp_max(m);
+        sum = 0.f;
+        for (int e = lane; e < E; e += 32) sum += expf(sc[e] - m);
+        sum = warp_sum(sum);
+    }
+    auto choice = [&](int e) { return rule.correction ? sc[e] + rule.correction[e] : sc[e]; };
     for (int e = lane; e < E; e += 32) {
-        const float s = expf(sc[e] - m) / sum;
-        sc[e] = s;
-        cand[e] = (n_groups > 1) ? -1.f : s;         // with groups: nobody stands until the group is kept
+        sc[e] = rule.sigmoid ? 1.0f / (1.0f + expf(-sc[e])) : expf(sc[e] - m) / sum;
+        cand[e] = (n_groups > 1) ? -INFINITY : choice(e);         // with groups: nobody stands until the group is kept
     }
     __syncwarp();
     if (n_groups > 1) {
@@ -120,15 +135,20 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
             float bv = -INFINITY;
             int bi = 0x7fffffff;
             for (int g = lane; g < n_groups; g += 32) {
-                if (cand[g * per] >= 0.f) continue;                 // group already kept (its experts stand)
-                float gv = -INFINITY;
-                for (int j = 0; j < per; ++j) gv = fmaxf(gv, sc[g * per + j]);
+                if (cand[g * per] > -INFINITY) continue;            // group already kept (its experts stand)
+                float best = -INFINITY, second = -INFINITY;
+                for (int j = 0; j < per; ++j) {
+                    const float c = choice(g * per + j);
+                    second = fmaxf(second, fminf(best, c));
+                    best = fmaxf(best, c);
+                }
+                const float gv = rule.group_best > 1 && per > 1 ? best + second : best;
                 if (gv > bv) { bv = gv; bi = g; }
             }
             warp_argmax(bv, bi);
             __syncwarp();
             if (bi != 0x7fffffff)
-                for (int j = lane; j < per; j += 32) cand[bi * per + j] = sc[bi * per + j];
+                for (int j = lane; j < per; j += 32) cand[bi * per + j] = choice(bi * per + j);
             __syncwarp();
         }
     }
@@ -138,31 +158,38 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
         int bi = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
             const float c = cand[e];
-            if (c >= 0.f && c > bv) { bv = c; bi = e; }
+            if (c > bv) { bv = c; bi = e; }
         }
         warp_argmax(bv, bi);
         __syncwarp();
+        const float s = bi != 0x7fffffff ? sc[bi] : 0.f;
         if (lane == 0) {
             idx_out[(size_t)t * top + k] = bi != 0x7fffffff ? bi : -1;
-            w_out[(size_t)t * top + k] = bi != 0x7fffffff ? bv : 0.f;
-            if (bi != 0x7fffffff) cand[bi] = -2.f;
+            w_out[(size_t)t * top + k] = s;
+            if (bi != 0x7fffffff) cand[bi] = -INFINITY;
         }
-        if (bi != 0x7fffffff) total += bv;
+        total += s;
         __syncwarp();
     }
-    if (renorm && lane == 0 && total > 0.f)
-        for (int k = 0; k < top; ++k) w_out[(size_t)t * top + k] /= total;
+    if (lane == 0 && (rule.renorm || rule.out_scale != 1.f)) {
+        const float den = rule.renorm ? total + rule.eps : 1.f;
+        if (den > 0.f)
+            for (int k = 0; k < top; ++k) w_out[(size_t)t * top + k] = w_out[(size_t)t * top + k] / den * rule.out_scale;
+    }
 }
 
 VOB_EXPORT int vob_moe_route(const void* x, int code, long ld_x, const float* w_router, const int* positions, int T, int width, int E,
-                             int top, int n_groups, int keep, int renorm, int* idx_out, float* w_out, cudaStream_t stream) {
+                             int top, int n_groups, int keep, int renorm, int sigmoid, int group_best, const float* correction, float eps,
+                             float out_scale, int* idx_out, float* w_out, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (group_best != 1 && group_best != 2) return VOB_ERR_BAD_ARG;
+    const RouteRule rule{sigmoid, group_best, renorm, correction, eps, out_scale};
     if (width <= 0 || E <= 0 || top <= 0 || top > E) return VOB_ERR_BAD_ARG;
     if (n_groups > 1 && (E % n_groups != 0 || keep <= 0 || keep > n_groups || top > keep * (E / n_groups))) return VOB_ERR_BAD_ARG;
     const size_t smem = (size_t)4 * 2 * E * sizeof(float);
     if (smem > 48 * 1024) return VOB_ERR_UNSUPPORTED;
     VOB_DISPATCH_ELEM(code, return vob_launch(moe_route_kernel<ElemT>, dim3((T + 3) / 4), dim3(128), smem, stream, (const ElemT*)x, ld_x, w_router,
-                                              positions, T, width, E, top, n_groups, keep, renorm, idx_out, w_out));
+                                              positions, T, width, E, top, n_groups, keep, rule, idx_out, w_out));
     return 0;
 }
 
@@ -237,6 +264,12 @@ __device__ __forceinline__ float moe_gate(float g, float u, int act, float limit
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
+// The activation of an expert without a gate, on the float32 sum. act 2: relu(u)^2.
+__device__ __forceinline__ float moe_act(float u, int act) {
+    (void)act;
+    u = fmaxf(u, 0.f);
+    return u * u;
+}
 // a float32 sum as the activations' type holds it
 template <typename T> __device__ __forceinline__ float moe_rounded(float v);
 template <> __device__ __forceinline__ float moe_rounded<float>(float v) { return v; }
@@ -297,15 +330,16 @@ moe_gate_up_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ w_g
 }
 
 // ---------------------------------------------------------------------------------------------
-// The experts' second product, plain multiply-adds. Grid (tiles, ceil(width / 64)); thread (ty, tx) owns rows ty, ty + 16
-// and columns tx, tx + 16, tx + 32, tx + 48. w_down [E, width, ff]. y float32 [P, width] = weight[pair] * sum.
+// One product per pair, plain multiply-adds: the experts' second product, or (UP) the first one of experts without a gate.
+// Grid (tiles, ceil(N / 64)); thread (ty, tx) owns rows ty, ty + 16 and columns tx, tx + 16, tx + 32, tx + 48. w [E, N, K].
+//   UP false: a [P, K] by pair, out float32 [P, N] = weight[pair] * sum;   UP true: a gathered by token, out [P, N] = act(sum).
 // ---------------------------------------------------------------------------------------------
-template <typename T>
+template <typename T, bool UP>
 __global__ void __launch_bounds__(256, 2)
-moe_down_kernel(const T* __restrict__ h, const T* __restrict__ w_down, const int* __restrict__ sorted,
-                const int* __restrict__ tile_expert, const float* __restrict__ pair_w, int width, int ff, float* __restrict__ y) {
+moe_single_kernel(const T* __restrict__ a, long ld_a, int a_div, const T* __restrict__ w, const int* __restrict__ sorted,
+                  const int* __restrict__ tile_expert, const float* __restrict__ pair_w, int N, int K, void* __restrict__ out, int act) {
     pdl_launch_dependents();
-    pdl_wait(74);
+    pdl_wait(UP ? 73 : 74);
     const int tile = blockIdx.x;
     const int e = tile_expert[tile];
     if (e < 0) return;
@@ -315,23 +349,23 @@ moe_down_kernel(const T* __restrict__ h, const T* __restrict__ w_down, const int
     if (tid < VOB_MOE_BM) pair_of[tid] = sorted[tile * VOB_MOE_BM + tid];
     __syncthreads();
     const int col0 = blockIdx.y * 64;
-    const T* wd = w_down + (size_t)e * width * ff;
+    const T* wd = w + (size_t)e * N * K;
     float acc[2][4];
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-    for (int k0 = 0; k0 < ff; k0 += 32) {
+    for (int k0 = 0; k0 < K; k0 += 32) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const int el = tid + 256 * i, r = el >> 5, c = el & 31;
             const int p = pair_of[r];
-            As[r][c] = (p >= 0 && k0 + c < ff) ? ld_f(h + (size_t)p * ff + k0 + c) : 0.f;
+            As[r][c] = (p >= 0 && k0 + c < K) ? ld_f(a + (size_t)(p / a_div) * ld_a + k0 + c) : 0.f;
         }
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             const int el = tid + 256 * i, r = el >> 5, c = el & 31;
-            Bs[r][c] = (col0 + r < width && k0 + c < ff) ? ld_f(wd + (size_t)(col0 + r) * ff + k0 + c) : 0.f;
+            Bs[r][c] = (col0 + r < N && k0 + c < K) ? ld_f(wd + (size_t)(col0 + r) * K + k0 + c) : 0.f;
         }
         __syncthreads();
 #pragma unroll 8
@@ -350,11 +384,13 @@ moe_down_kernel(const T* __restrict__ h, const T* __restrict__ w_down, const int
     for (int i = 0; i < 2; ++i) {
         const int p = pair_of[ty + 16 * i];
         if (p < 0) continue;
-        const float wgt = pair_w[p];
+        const float wgt = UP ? 1.f : pair_w[p];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int c = col0 + tx + 16 * j;
-            if (c < width) y[(size_t)p * width + c] = wgt * acc[i][j];
+            if (c >= N) continue;
+            if (UP) st_f(reinterpret_cast<T*>(out) + (size_t)p * N + c, moe_act(acc[i][j], act));
+            else reinterpret_cast<float*>(out)[(size_t)p * N + c] = wgt * acc[i][j];
         }
     }
 }
@@ -461,11 +497,14 @@ moe_gate_up_tc_kernel(const __nv_bfloat16* __restrict__ x, long ld_x, const __nv
     }
 }
 
+// The tensor-core form of moe_single_kernel (same arguments).
+template <bool UP>
 __global__ void __launch_bounds__(128)
-moe_down_tc_kernel(const __nv_bfloat16* __restrict__ h, const __nv_bfloat16* __restrict__ w_down, const int* __restrict__ sorted,
-                   const int* __restrict__ tile_expert, const float* __restrict__ pair_w, int width, int ff, float* __restrict__ y) {
+moe_single_tc_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const __nv_bfloat16* __restrict__ w,
+                     const int* __restrict__ sorted, const int* __restrict__ tile_expert, const float* __restrict__ pair_w, int N, int K,
+                     void* __restrict__ out, int act) {
     pdl_launch_dependents();
-    pdl_wait(76);
+    pdl_wait(UP ? 75 : 76);
     const int tile = blockIdx.x;
     const int e = tile_expert[tile];
     if (e < 0) return;
@@ -476,20 +515,20 @@ moe_down_tc_kernel(const __nv_bfloat16* __restrict__ h, const __nv_bfloat16* __r
     __shared__ const __nv_bfloat16* b_rows[64];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int col0 = blockIdx.y * 64;
-    const __nv_bfloat16* wd = w_down + (size_t)e * width * ff;
+    const __nv_bfloat16* wd = w + (size_t)e * N * K;
     if (tid < VOB_MOE_BM) {
         const int p = sorted[tile * VOB_MOE_BM + tid];
         pair_of[tid] = p;
-        a_rows[tid] = p >= 0 ? h + (size_t)p * ff : nullptr;
+        a_rows[tid] = p >= 0 ? a + (size_t)(p / a_div) * ld_a : nullptr;
     }
-    if (tid < 64) b_rows[tid] = col0 + tid < width ? wd + (size_t)(col0 + tid) * ff : nullptr;
+    if (tid < 64) b_rows[tid] = col0 + tid < N ? wd + (size_t)(col0 + tid) * K : nullptr;
     __syncthreads();
     wmma::fragment<wmma::accumulator, 16, 16, 16, float> cc[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) wmma::fill_fragment(cc[i], 0.f);
-    for (int k0 = 0; k0 < ff; k0 += VOB_MOE_TK) {
-        moe_stage_rows(As, VOB_MOE_BM, a_rows, k0, ff);
-        moe_stage_rows(Bs, 64, b_rows, k0, ff);
+    for (int k0 = 0; k0 < K; k0 += VOB_MOE_TK) {
+        moe_stage_rows(As, VOB_MOE_BM, a_rows, k0, K);
+        moe_stage_rows(Bs, 64, b_rows, k0, K);
         __syncthreads();
 #pragma unroll
         for (int kk = 0; kk < VOB_MOE_TK; kk += 16) {
@@ -497,9 +536,9 @@ moe_down_tc_kernel(const __nv_bfloat16* __restrict__ h, const __nv_bfloat16* __r
             wmma::load_matrix_sync(b, &Bs[warp * 16][kk], VOB_MOE_LDS);
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
-                wmma::fragment<wmma::matrix_a, 16, 16, 16, __nv_bfloat16, wmma::row_major> a;
-                wmma::load_matrix_sync(a, &As[16 * i][kk], VOB_MOE_LDS);
-                wmma::mma_sync(cc[i], a, b, cc[i]);
+                wmma::fragment<wmma::matrix_a, 16, 16, 16, __nv_bfloat16, wmma::row_major> fa;
+                wmma::load_matrix_sync(fa, &As[16 * i][kk], VOB_MOE_LDS);
+                wmma::mma_sync(cc[i], fa, b, cc[i]);
             }
         }
         __syncthreads();
@@ -511,7 +550,10 @@ moe_down_tc_kernel(const __nv_bfloat16* __restrict__ h, const __nv_bfloat16* __r
         for (int el = lane; el < 256; el += 32) {
             const int r = el >> 4, c = el & 15;
             const int p = pair_of[16 * i + r], col = col0 + warp * 16 + c;
-            if (p >= 0 && col < width) y[(size_t)p * width + col] = pair_w[p] * Cs[warp][el];
+            if (p >= 0 && col < N) {
+                if (UP) reinterpret_cast<__nv_bfloat16*>(out)[(size_t)p * N + col] = __float2bfloat16_rn(moe_act(Cs[warp][el], act));
+                else reinterpret_cast<float*>(out)[(size_t)p * N + col] = pair_w[p] * Cs[warp][el];
+            }
         }
         __syncwarp();
     }
@@ -520,7 +562,7 @@ moe_down_tc_kernel(const __nv_bfloat16* __restrict__ h, const __nv_bfloat16* __r
 // ---------------------------------------------------------------------------------------------
 // The same two products for rows that 16-byte copies can fetch (K a multiple of 8, 16-byte aligned rows): tiles of BM
 // pairs (32: four warps; 128: eight warps, two along the rows) and 128 weight rows (gate_up: 64 gate and the 64 up rows
-// of the same hidden columns; down: 128 output columns), 32 features a stage, STAGES stages in flight through cp.async
+// of the same hidden columns; down, and up of experts without a gate: 128 output columns), 32 features a stage, STAGES stages in flight through cp.async
 // (absent rows and features behind K arrive as zeros). The order of a sum is the one of the kernels above: 16
 // features a step, in order.
 // ---------------------------------------------------------------------------------------------
@@ -534,13 +576,15 @@ __device__ __forceinline__ void moe_cp16(void* dst, const void* src, int bytes) 
 __device__ __forceinline__ void moe_cp_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 template <int N> __device__ __forceinline__ void moe_cp_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
 
-template <int BM, int STAGES, bool DOWN>
+enum MoeProduct { MOE_GATE_UP = 0, MOE_DOWN = 1, MOE_UP = 2 };
+
+template <int BM, int STAGES, int KIND>
 __global__ void __launch_bounds__(BM == 128 ? 256 : 128)
 moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const __nv_bfloat16* __restrict__ w,
                 const int* __restrict__ sorted, const int* __restrict__ tile_expert, const float* __restrict__ pair_w,
                 int K, int N, void* __restrict__ out, int act, float limit) {
     pdl_launch_dependents();
-    pdl_wait(DOWN ? 76 : 75);
+    pdl_wait(KIND == MOE_DOWN ? 76 : 75);
     constexpr int WR = BM == 128 ? 2 : 1;             // warps along the rows
     constexpr int NT = 128 * WR;
     constexpr int RF = BM / WR / 16;                   // 16-row fragments a warp owns
@@ -553,7 +597,7 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
     __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(moe_smem);
     __shared__ int pair_of[BM];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wc = warp & 3, wr = warp >> 2;
-    const int col0 = blockIdx.y * (DOWN ? 128 : 64);
+    const int col0 = blockIdx.y * (KIND != MOE_GATE_UP ? 128 : 64);
     // the rows this thread fetches, the same in every stage
     const __nv_bfloat16* src[CHUNKS];
     int dst_off[CHUNKS], feat[CHUNKS];
@@ -572,7 +616,7 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
             if (p >= 0) src[i] = a + (size_t)(p / a_div) * ld_a;
         } else {
             const int j = r - BM;
-            if (DOWN) {
+            if (KIND != MOE_GATE_UP) {
                 if (col0 + j < N) src[i] = w + ((size_t)e * N + col0 + j) * K;
             } else {
                 const int col = col0 + (j & 63);
@@ -632,7 +676,12 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
             const int r = el >> 4, c = el & 15;
             const int p = pair_of[wr * (BM / WR) + 16 * i + r];
             if (p < 0) continue;
-            if (DOWN) {
+            if (KIND == MOE_UP) {
+                __nv_bfloat16* ho = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)p * N;
+                const int ca = col0 + wc * 16 + c, cb = ca + 64;
+                if (ca < N) ho[ca] = __float2bfloat16_rn(moe_act(Cs[el], act));
+                if (cb < N) ho[cb] = __float2bfloat16_rn(moe_act(Cs[256 + el], act));
+            } else if (KIND == MOE_DOWN) {
                 float* y = reinterpret_cast<float*>(out);
                 const float wgt = pair_w[p];
                 const int ca = col0 + wc * 16 + c, cb = ca + 64;
@@ -651,17 +700,17 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
     }
 }
 
-template <int BM, int STAGES, bool DOWN>
+template <int BM, int STAGES, int KIND>
 static int moe_pipe_launch(dim3 grid, cudaStream_t stream, const __nv_bfloat16* a, long ld_a, int a_div, const __nv_bfloat16* w,
                            const int* sorted, const int* tile_expert, const float* pair_w, int K, int N, void* out, int act = 0, float limit = 0.f) {
     const size_t smem = (size_t)STAGES * (BM + 128) * VOB_MOE_PLD * sizeof(__nv_bfloat16);
     static bool raised = false;
     if (!raised) {
-        cudaError_t err = cudaFuncSetAttribute(moe_pipe_kernel<BM, STAGES, DOWN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t err = cudaFuncSetAttribute(moe_pipe_kernel<BM, STAGES, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (err != cudaSuccess) return (int)err;
         raised = true;
     }
-    return vob_launch(moe_pipe_kernel<BM, STAGES, DOWN>, grid, dim3(BM == 128 ? 256 : 128), smem, stream, a, ld_a, a_div, w, sorted,
+    return vob_launch(moe_pipe_kernel<BM, STAGES, KIND>, grid, dim3(BM == 128 ? 256 : 128), smem, stream, a, ld_a, a_div, w, sorted,
                       tile_expert, pair_w, K, N, out, act, limit);
 }
 
@@ -682,8 +731,8 @@ VOB_EXPORT int vob_moe_gate_up(const void* x, int code, long ld_x, const void* w
         const dim3 grid(max_tiles, (ff + 63) / 64);
         const __nv_bfloat16 *xa = (const __nv_bfloat16*)x, *wa = (const __nv_bfloat16*)w_gu;
         if (moe_rows_by16(x, ld_x, width) && moe_rows_by16(w_gu, width, width)) {
-            if (tile_rows == 128) return moe_pipe_launch<128, 3, false>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act, limit);
-            return moe_pipe_launch<32, 4, false>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act, limit);
+            if (tile_rows == 128) return moe_pipe_launch<128, 3, MOE_GATE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act, limit);
+            return moe_pipe_launch<32, 4, MOE_GATE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act, limit);
         }
         if (tile_rows != VOB_MOE_BM) return VOB_ERR_UNSUPPORTED;
         return vob_launch(moe_gate_up_tc_kernel, grid, dim3(128), 0, stream, xa, ld_x, wa, sorted, tile_expert, top, width, ff,
@@ -706,15 +755,40 @@ VOB_EXPORT int vob_moe_down(const void* h, int code, const void* w_down, const i
         const __nv_bfloat16 *ha = (const __nv_bfloat16*)h, *wa = (const __nv_bfloat16*)w_down;
         if (moe_rows_by16(h, ff, ff) && moe_rows_by16(w_down, ff, ff)) {
             const dim3 grid(max_tiles, (width + 127) / 128);
-            if (tile_rows == 128) return moe_pipe_launch<128, 3, true>(grid, stream, ha, ff, 1, wa, sorted, tile_expert, pair_w, ff, width, y);
-            return moe_pipe_launch<32, 4, true>(grid, stream, ha, ff, 1, wa, sorted, tile_expert, pair_w, ff, width, y);
+            if (tile_rows == 128) return moe_pipe_launch<128, 3, MOE_DOWN>(grid, stream, ha, ff, 1, wa, sorted, tile_expert, pair_w, ff, width, y);
+            return moe_pipe_launch<32, 4, MOE_DOWN>(grid, stream, ha, ff, 1, wa, sorted, tile_expert, pair_w, ff, width, y);
         }
         if (tile_rows != VOB_MOE_BM) return VOB_ERR_UNSUPPORTED;
-        return vob_launch(moe_down_tc_kernel, dim3(max_tiles, (width + 63) / 64), dim3(128), 0, stream, ha, wa, sorted, tile_expert, pair_w,
-                          width, ff, y);
+        return vob_launch(moe_single_tc_kernel<false>, dim3(max_tiles, (width + 63) / 64), dim3(128), 0, stream, ha, (long)ff, 1, wa, sorted,
+                          tile_expert, pair_w, width, ff, y, 0);
     }
-    VOB_DISPATCH_ELEM(code, return vob_launch(moe_down_kernel<ElemT>, dim3(max_tiles, (width + 63) / 64), dim3(256), 0, stream, (const ElemT*)h,
-                                              (const ElemT*)w_down, sorted, tile_expert, pair_w, width, ff, y));
+    VOB_DISPATCH_ELEM(code, return vob_launch(moe_single_kernel<ElemT, false>, dim3(max_tiles, (width + 63) / 64), dim3(256), 0, stream,
+                                              (const ElemT*)h, (long)ff, 1, (const ElemT*)w_down, sorted, tile_expert, pair_w, width, ff, y, 0));
+    return 0;
+}
+
+// The first product of experts without a gate: h_out [T * top, ff] = act(W_up[e] x[token]), act 2: relu squared. w_up
+// [E, ff, width]. Everything else as vob_moe_gate_up.
+VOB_EXPORT int vob_moe_up(const void* x, int code, long ld_x, const void* w_up, const int* sorted, const int* tile_expert, int max_tiles,
+                          int tile_rows, int top, int width, int ff, void* h_out, int tensor_cores, int act, cudaStream_t stream) {
+    if (max_tiles <= 0) return 0;
+    if (top <= 0 || width <= 0 || ff <= 0 || act != 2) return VOB_ERR_BAD_ARG;
+    if (tile_rows != VOB_MOE_BM && !(tile_rows == 128 && tensor_cores)) return VOB_ERR_BAD_ARG;
+    if ((ff + 63) / 64 > 65535) return VOB_ERR_UNSUPPORTED;
+    if (tensor_cores) {
+        if (code != VOB_BF16) return VOB_ERR_BAD_ARG;
+        const __nv_bfloat16 *xa = (const __nv_bfloat16*)x, *wa = (const __nv_bfloat16*)w_up;
+        if (moe_rows_by16(x, ld_x, width) && moe_rows_by16(w_up, width, width)) {
+            const dim3 grid(max_tiles, (ff + 127) / 128);
+            if (tile_rows == 128) return moe_pipe_launch<128, 3, MOE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act);
+            return moe_pipe_launch<32, 4, MOE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act);
+        }
+        if (tile_rows != VOB_MOE_BM) return VOB_ERR_UNSUPPORTED;
+        return vob_launch(moe_single_tc_kernel<true>, dim3(max_tiles, (ff + 63) / 64), dim3(128), 0, stream, xa, ld_x, top, wa, sorted, tile_expert,
+                          (const float*)nullptr, ff, width, h_out, act);
+    }
+    VOB_DISPATCH_ELEM(code, return vob_launch(moe_single_kernel<ElemT, true>, dim3(max_tiles, (ff + 63) / 64), dim3(256), 0, stream, (const ElemT*)x,
+                                              ld_x, top, (const ElemT*)w_up, sorted, tile_expert, (const float*)nullptr, ff, width, h_out, act));
     return 0;
 }
 

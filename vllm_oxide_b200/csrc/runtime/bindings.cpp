@@ -24,11 +24,13 @@ PYBIND11_MODULE(VOB_MODULE_NAME, m) {
     py::register_exception<CacheError>(m, "RuntimeFault");
 
     py::class_<GroupSpec>(m, "GroupSpec")
-        .def(py::init([](int kind, int window, int num_pages) { GroupSpec g; g.kind = kind; g.window = window; g.num_pages = num_pages; return g; }),
-             py::arg("kind"), py::arg("window"), py::arg("num_pages"))
+        .def(py::init([](int kind, int window, int num_pages, int keep_first) {
+                 GroupSpec g; g.kind = kind; g.window = window; g.num_pages = num_pages; g.keep_first = keep_first; return g; }),
+             py::arg("kind"), py::arg("window"), py::arg("num_pages"), py::arg("keep_first") = 0)
         .def_readwrite("kind", &GroupSpec::kind)
         .def_readwrite("window", &GroupSpec::window)
-        .def_readwrite("num_pages", &GroupSpec::num_pages);
+        .def_readwrite("num_pages", &GroupSpec::num_pages)
+        .def_readwrite("keep_first", &GroupSpec::keep_first);
     m.attr("FULL") = (int)kFull;
     m.attr("WINDOW") = (int)kWindow;
     m.attr("CHUNK") = (int)kChunk;

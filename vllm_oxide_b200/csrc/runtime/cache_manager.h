@@ -12,7 +12,8 @@
 // and every request has one block table per group:
 //   Full   - every key is kept while the request lives;
 //   Window - only the last `window` keys are read, so a page is given back as soon as every
-//            position in it has fallen out of the window of the next query;
+//            position in it has fallen out of the window of the next query; with `keep_first` the
+//            keys of the first so many positions are read as well, and their pages stay;
 //   Chunk  - positions are cut into blocks of `window` counted from 0 and a query reads the keys
 //            of its own block only, so a page is given back once the next query's block starts
 //            behind it.
@@ -39,18 +40,24 @@ struct GroupSpec {
     int kind = kFull;
     int window = 0;      // keys visible to a query, itself included (Window groups); the block length (Chunk groups)
     int num_pages = 0;
+    int keep_first = 0;  // Window groups: so many first positions stay visible to every query behind them
 
-    // First position whose key a query at position `pos` still reads.
+    // Pages at the start of a request that are never given back while it lives.
+    int64_t kept_pages(int page_size) const {
+        return kind == kWindow ? ((int64_t)keep_first + page_size - 1) / page_size : 0;
+    }
+    // First position whose key a query at position `pos` still reads (kept first positions aside).
     int64_t first_visible(int64_t pos) const {
         if (kind == kWindow) return std::max<int64_t>(0, pos + 1 - window);
         if (kind == kChunk) return pos - pos % window;
         return 0;
     }
     // Most tokens whose pages a request of `total` tokens holds at any one time: a window group
-    // holds the window plus the page being filled, a chunk group one block plus the page it
-    // starts in the middle of, a full group everything.
+    // holds the window plus the page being filled plus the kept first pages, a chunk group one block plus
+    // the page it starts in the middle of, a full group everything.
     int64_t max_live_tokens(int64_t total, int page_size) const {
-        if (kind == kWindow || kind == kChunk) return std::min<int64_t>(total, (int64_t)window + page_size);
+        if (kind == kWindow || kind == kChunk)
+            return std::min<int64_t>(total, (int64_t)window + page_size + kept_pages(page_size) * page_size);
         return total;
     }
 };
@@ -106,6 +113,7 @@ public:
         for (const auto& g : groups_) {
             if (g.num_pages <= 0) throw CacheError("a cache group needs at least one page");
             if (g.kind == kWindow && g.window <= 0) throw CacheError("a window group needs a positive window");
+            if (g.keep_first < 0 || (g.keep_first > 0 && g.kind != kWindow)) throw CacheError("kept first positions go with a window group");
             if (g.kind == kChunk && g.window <= 0) throw CacheError("a chunk group needs a positive block length");
             if (g.kind != kFull && g.kind != kWindow && g.kind != kChunk) throw CacheError("unknown cache group kind");
             pools_.emplace_back(g.num_pages);
@@ -193,7 +201,7 @@ public:
     }
 
     // The step that wrote n_new tokens is done: they count, and window groups give back every
-    // page that the next query (at position len) can no longer see.
+    // page that the next query (at position len) can no longer see (pages of kept first positions stay).
     std::vector<std::pair<int, int>> commit(int64_t id, int64_t n_new) {
         auto it = reqs_.find(id);
         if (it == reqs_.end()) throw CacheError("request " + std::to_string(id) + " is not admitted");
@@ -206,7 +214,7 @@ public:
             int64_t first = first_visible((int)g, r.len);        // next query sits at position len
             int64_t dead_pages = first / page_size_;             // pages wholly below `first` (none in a full group)
             auto& t = r.tables[g];
-            for (int64_t i = 0; i < dead_pages && i < (int64_t)t.size(); ++i) {
+            for (int64_t i = groups_[g].kept_pages(page_size_); i < dead_pages && i < (int64_t)t.size(); ++i) {
                 if (t[i] >= 0) {
                     pools_[g].give_back(t[i]);
                     released.emplace_back((int)g, t[i]);

@@ -340,6 +340,31 @@ def layernorm_rows(resid: torch.Tensor, weight: torch.Tensor, bias: Optional[tor
 
 
 @_timed
+def add_layernorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                  out: torch.Tensor, rows: Optional[torch.Tensor] = None, mult: float = 1.0) -> None:
+    """resid += mult * delta in place, then out = LN(resid); with `rows` only those rows are normalised (delta is still added
+    to what they read) and the residual is left as it is."""
+    op = "add_layernorm"
+    _cuda(op, resid, delta, weight, bias, out, rows)
+    if resid.dtype != torch.float32 or resid.dim() != 2 or not resid.is_contiguous():
+        raise ShapeError(op, f"the residual must be contiguous float32 [T, h], got {resid.dtype} {list(resid.shape)}")
+    T, h = resid.shape
+    _f32_vec(weight, h, op, "weight")
+    _f32_vec(bias, h, op, "bias")
+    if delta is not None and (delta.shape != resid.shape or not delta.is_contiguous()):
+        raise ShapeError(op, f"delta must be contiguous {list(resid.shape)}, got {list(delta.shape)}")
+    R = T
+    if rows is not None:
+        R = rows.numel()
+        _int32_vec(rows, R, op, "rows")
+    if out.dim() != 2 or out.shape[0] < R or out.shape[1] != h or not out.is_contiguous():
+        raise ShapeError(op, f"out must be contiguous [>={R}, {h}], got {list(out.shape)}")
+    f = _fn("elementwise", "vob_add_layernorm", [_P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _F, _F, _P])
+    _check(f(_ptr(resid), _ptr(delta), _code(delta, op) if delta is not None else 0, _ptr(weight), _ptr(bias), _ptr(rows), _ptr(out),
+             _code(out, op), R, h, float(eps), float(mult), _stream()), op)
+
+
+@_timed
 def cast_rows(src: torch.Tensor, out: torch.Tensor) -> None:
     """out = src (float32, contiguous) in out's type, element by element."""
     op = "cast_rows"
@@ -1224,6 +1249,8 @@ def depth_average(stack: torch.Tensor, x: torch.Tensor, weights: Optional[torch.
 MOE_TILE_ROWS = 32           # rows of a tile of (token, expert) pairs (VOB_MOE_BM of csrc/moe.cu)
 MOE_LARGE_TILE_ROWS = 128    # the pipelined tensor-core products also take tiles of this many
 MOE_ACTIVATIONS = {"silu": 0, "clamped_swish": 1}    # how an expert's gate acts on its hidden values
+MOE_UNGATED = {"relu2": 2}                           # activations of experts without a gate
+MOE_SCORES = {"softmax": 0, "sigmoid": 1}            # how router logits become scores
 MOE_LARGE_TILE_FROM = 64     # pairs an expert gets on average from which the large tiles are taken
 
 
@@ -1242,17 +1269,23 @@ def moe_sorted_rows(pairs: int, experts: int, tile_rows: int = MOE_TILE_ROWS) ->
 
 @_timed
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, positions: Optional[torch.Tensor], top: int, groups: int, keep: int,
-              renorm: bool, idx_out: torch.Tensor, w_out: torch.Tensor) -> None:
+              renorm: bool, idx_out: torch.Tensor, w_out: torch.Tensor, score: str = "softmax", correction: Optional[torch.Tensor] = None,
+              group_best: int = 1, eps: float = 0.0, out_scale: float = 1.0) -> None:
     """Per row of x [T, width]: softmax over the E router logits (w_router float32 [E, width], float32 sums), election of
     `top` experts among those of the `keep` best of `groups` runs of neighbours (groups <= 1: among all), weights = their
-    scores (renorm: divided by their sum). idx_out int32 [T, top] (-1 for rows of negative position), w_out float32 [T, top]."""
+    scores (renorm: divided by their sum + `eps`) times `out_scale`. idx_out int32 [T, top] (-1 for rows of negative position),
+    w_out float32 [T, top]. `score` "sigmoid": scores are the sigmoids of the logits. `correction` (float32 [E]): the election
+    goes by score + correction, the weights by the score. `group_best` 2: a run scores as the sum of its two best experts."""
     op = "moe_route"
-    _cuda(op, x, w_router, positions, idx_out, w_out)
+    _cuda(op, x, w_router, positions, idx_out, w_out, correction)
+    if score not in MOE_SCORES or group_best not in (1, 2):
+        raise ShapeError(op, f"score {score!r} ({', '.join(MOE_SCORES)}) or group_best {group_best} (1 or 2) is not known")
     _rows_2d(x, op, "x")
     T, width = x.shape
     if w_router.dtype != torch.float32 or w_router.dim() != 2 or w_router.shape[1] != width or not w_router.is_contiguous():
         raise ShapeError(op, f"w_router must be contiguous float32 [experts, {width}], got {w_router.dtype} {list(w_router.shape)}")
     E = w_router.shape[0]
+    _f32_vec(correction, E, op, "correction")
     if not 0 < top <= E:
         raise ShapeError(op, f"{top} choices among {E} experts")
     if groups > 1 and (E % groups or not 0 < keep <= groups or top > keep * (E // groups)):
@@ -1263,9 +1296,10 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, positions: Optional[torch
         raise ShapeError(op, f"w_out must be contiguous float32 [{T}, {top}], got {w_out.dtype} {list(w_out.shape)}")
     if positions is not None:
         _int32_vec(positions, T, op, "positions")
-    f = _fn("moe", "vob_moe_route", [_P, _I, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P])
+    f = _fn("moe", "vob_moe_route", [_P, _I, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _F, _F, _P, _P, _P])
     _check(f(_ptr(x), _code(x, op), x.stride(0), _ptr(w_router), _ptr(positions), T, width, E, int(top), int(groups), int(keep),
-             1 if renorm else 0, _ptr(idx_out), _ptr(w_out), _stream()), op)
+             1 if renorm else 0, MOE_SCORES[score], int(group_best), _ptr(correction), float(eps), float(out_scale), _ptr(idx_out),
+             _ptr(w_out), _stream()), op)
 
 
 @_timed
@@ -1329,6 +1363,32 @@ def moe_gate_up(x: torch.Tensor, w_gu: torch.Tensor, sorted_pairs: torch.Tensor,
     f = _fn("moe", "vob_moe_gate_up", [_P, _I, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P])
     _check(f(_ptr(x), _code(x, op), x.stride(0), _ptr(w_gu), _ptr(sorted_pairs), _ptr(tile_expert), tiles, int(tile_rows), int(top), width, ff,
              _ptr(h_out), 1 if tensor_cores else 0, MOE_ACTIVATIONS[activation], float(limit), _stream()), op)
+
+
+@_timed
+def moe_up(x: torch.Tensor, w_up: torch.Tensor, sorted_pairs: torch.Tensor, tile_expert: torch.Tensor, top: int, h_out: torch.Tensor,
+           activation: str, tensor_cores: bool = False, tile_rows: int = MOE_TILE_ROWS) -> None:
+    """The first product of experts without a gate: h_out[pair] = act(W_up[e] x[token]); w_up [E, ff, width]. `activation`
+    "relu2": relu squared. Everything else as `moe_gate_up`."""
+    op = "moe_up"
+    if activation not in MOE_UNGATED:
+        raise ShapeError(op, f"activation {activation!r} is not known ({', '.join(MOE_UNGATED)})")
+    _cuda(op, x, w_up, sorted_pairs, tile_expert, h_out)
+    _rows_2d(x, op, "x")
+    T, width = x.shape
+    if w_up.dim() != 3 or w_up.shape[2] != width or w_up.dtype != x.dtype or not w_up.is_contiguous():
+        raise ShapeError(op, f"w_up must be contiguous {x.dtype} [experts, ff, {width}], got {w_up.dtype} {list(w_up.shape)}")
+    ff = w_up.shape[1]
+    if h_out.shape != (T * top, ff) or h_out.dtype != x.dtype or not h_out.is_contiguous():
+        raise ShapeError(op, f"h_out must be contiguous {x.dtype} [{T * top}, {ff}], got {h_out.dtype} {list(h_out.shape)}")
+    if tensor_cores and x.dtype != torch.bfloat16:
+        raise ShapeError(op, "the tensor-core form takes bfloat16")
+    tiles = _moe_tiles(op, sorted_pairs, tile_expert, tile_rows, tensor_cores, width, ff)
+    if tile_rows != MOE_TILE_ROWS and (x.stride(0) % 8 or x.data_ptr() % 16):
+        raise ShapeError(op, f"tiles of {tile_rows} rows need rows of x that start on 16-byte boundaries")
+    f = _fn("moe", "vob_moe_up", [_P, _I, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _P])
+    _check(f(_ptr(x), _code(x, op), x.stride(0), _ptr(w_up), _ptr(sorted_pairs), _ptr(tile_expert), tiles, int(tile_rows), int(top), width, ff,
+             _ptr(h_out), 1 if tensor_cores else 0, MOE_UNGATED[activation], _stream()), op)
 
 
 @_timed
@@ -1499,6 +1559,22 @@ def _kv_caches(op, kcache, vcache, kv_heads, dim, vdim, dtype):
         raise ShapeError(op, "one layer's cache has 2^31 rows or more")
 
 
+def _key_scales(op, kscale, kcache):
+    want = (kcache.shape[0], 1, kcache.shape[2], 1)
+    if kscale is not None and (kscale.dtype != torch.float32 or tuple(kscale.shape) != want or not kscale.is_contiguous()):
+        raise ShapeError(op, f"one float32 per cached token, contiguous {list(want)}, is needed, got {kscale.dtype} {list(kscale.shape)}")
+
+
+def _gate_cols(op, gate, rows, heads, vdim, dtype) -> int:
+    """1 where the gate has one column per head, 0 where it has one per feature; anything else is refused."""
+    if gate is None:
+        return 0
+    _rows_2d(gate, op, "gate")
+    if gate.dtype != dtype or gate.shape not in ((rows, heads * vdim), (rows, heads)):
+        raise ShapeError(op, f"gate must be {dtype} [{rows}, {heads * vdim}] or [{rows}, {heads}], got {gate.dtype} {list(gate.shape)}")
+    return 1 if gate.shape[1] != heads * vdim else 0
+
+
 @_timed
 def flex_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, positions: torch.Tensor, slots: Optional[torch.Tensor],
               inv_freq: Optional[torch.Tensor], rot: int, unit_rms: bool, eps: float, q_temp, vmix: Optional[torch.Tensor],
@@ -1557,6 +1633,31 @@ def flex_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, positions:
 
 
 @_timed
+def whole_norm_prep(proj: torch.Tensor, q_off: int, positions: torch.Tensor, slots: torch.Tensor, q_weight: torch.Tensor, eps: float,
+                    q_out: torch.Tensor, kcache: torch.Tensor, kscale: torch.Tensor, heads: int, kv_heads: int, dim: int) -> None:
+    """Per token, from the columns [q | k] of `proj` that start at q_off, q and k each normed as a whole (all heads at once):
+    q_out [T, heads * dim] = q / sqrt(mean(q^2) + eps) * q_weight (float32 [heads * dim]); the keys go to their cache slots as
+    they are and kscale (float32 [pages, 1, page_size, 1]) gets 1 / sqrt(mean(k^2) + eps) of the token."""
+    op = "whole_norm_prep"
+    _cuda(op, proj, positions, slots, q_weight, q_out, kcache, kscale)
+    _rows_2d(proj, op, "proj")
+    _rows_2d(q_out, op, "q_out")
+    T = proj.shape[0]
+    if q_off < 0 or q_off + (heads + kv_heads) * dim > proj.shape[1]:
+        raise ShapeError(op, f"columns {q_off}..{q_off + (heads + kv_heads) * dim} lie outside proj's {proj.shape[1]}")
+    if q_out.shape != (T, heads * dim) or q_out.dtype != proj.dtype:
+        raise ShapeError(op, f"q_out must be {proj.dtype} [{T}, {heads * dim}], got {q_out.dtype} {list(q_out.shape)}")
+    _f32_vec(q_weight, heads * dim, op, "q_weight")
+    _kv_caches(op, kcache, kcache, kv_heads, dim, dim, proj.dtype)
+    _key_scales(op, kscale, kcache)
+    _int32_vec(positions, T, op, "positions")
+    _int32_vec(slots, T, op, "slots")
+    f = _fn("attention_flex", "vob_whole_norm_prep", [_P, _I, _L, _I, _P, _P, _P, _F, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P])
+    _check(f(_ptr(proj), _code(proj, op), proj.stride(0), int(q_off), _ptr(positions), _ptr(slots), _ptr(q_weight), float(eps), _ptr(q_out),
+             q_out.stride(0), _ptr(kcache), _ptr(kscale), T, heads, kv_heads, dim, kcache.shape[2], _stream()), op)
+
+
+@_timed
 def pool_blocks(kcache: torch.Tensor, vcache: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, block_tables: torch.Tensor,
                 row_seq: torch.Tensor, positions: torch.Tensor, pool: int) -> None:
     """For every row whose position p ends a block of `pool` tokens ((p + 1) % pool == 0): the mean of the block's cached keys
@@ -1586,7 +1687,8 @@ def pool_blocks(kcache: torch.Tensor, vcache: torch.Tensor, kpool: torch.Tensor,
 def flex_attention(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_tables: torch.Tensor,
                    row_seq: torch.Tensor, positions: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, scale: float,
                    window: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                   out_scale: float = 1.0, chunk: int = 0, softcap: float = 0.0, dist_bias=None, pool: int = 0) -> None:
+                   out_scale: float = 1.0, chunk: int = 0, softcap: float = 0.0, dist_bias=None, pool: int = 0, keep_first: int = 0,
+                   dist_slopes: Optional[torch.Tensor] = None, key_scale: Optional[torch.Tensor] = None) -> None:
     """Causal attention of every row of q [T, heads * dim] over its request's pages, keys of `dim` and values of `vdim`
     features: out [T, heads * vdim] (any row stride) = softmax(q . K * scale) V, over the last `window` keys (0: all), the
     denominator also holding exp(sink[head]) if `sink` (float32 [heads]) is given; times sigmoid(gate) ([T, heads * vdim],
@@ -1594,12 +1696,19 @@ def flex_attention(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vca
     counted from position 0). `softcap` > 0: score <- softcap * tanh(score / softcap). `dist_bias` = (r1, r2), float32 [heads]
     each: r1 * ln(1 + r2 * distance) is taken off the score. `pool` > 0 (with a window): every block of `pool` positions that
     ends at or before position - window is seen as one key and one value, the means of the block's cached keys and values, in
-    the same softmax as the window's tokens."""
+    the same softmax as the window's tokens. `keep_first`, `dist_slopes`, `key_scale`: see `_score_shape`. `gate` may have one
+    column per head."""
     op = "flex_attention"
+    if keep_first and (keep_first < 0 or window <= 0 or chunk or pool):
+        raise ShapeError(op, f"{keep_first} kept first tokens go with a window, without blocks of positions and pooled blocks")
+    if dist_slopes is not None and dist_bias is not None:
+        raise ShapeError(op, "a bias on the logarithm of the distance or on the distance, not both")
+    if pool and (dist_slopes is not None or key_scale is not None):
+        raise ShapeError(op, "pooled blocks go without a bias on the distance and without numbers per key")
     if pool < 0 or (pool and (window <= 0 or chunk)):
         raise ShapeError(op, f"pooled blocks of {pool} go with a window and without blocks of positions")
-    r1, r2 = dist_bias if dist_bias is not None else (None, None)
-    _cuda(op, q, out, kcache, vcache, block_tables, row_seq, positions, sink, gate, r1, r2)
+    r1, r2 = dist_bias if dist_bias is not None else (dist_slopes, None)
+    _cuda(op, q, out, kcache, vcache, block_tables, row_seq, positions, sink, gate, r1, r2, key_scale)
     _f32_vec(r1, heads, op, "dist_bias[0]")
     _f32_vec(r2, heads, op, "dist_bias[1]")
     if chunk < 0 or softcap < 0:
@@ -1620,16 +1729,14 @@ def flex_attention(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vca
     _int32_vec(row_seq, T, op, "row_seq")
     _int32_vec(positions, T, op, "positions")
     _f32_vec(sink, heads, op, "sink")
-    if gate is not None:
-        _rows_2d(gate, op, "gate")
-        if gate.shape != (T, heads * vdim) or gate.dtype != q.dtype:
-            raise ShapeError(op, f"gate must be {q.dtype} [{T}, {heads * vdim}], got {gate.dtype} {list(gate.shape)}")
+    _key_scales(op, key_scale, kcache)
+    gate_heads = _gate_cols(op, gate, T, heads, vdim, q.dtype)
     f = _fn("attention_flex", "vob_flex_attention", [_P, _L, _P, _L, _P, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P,
-                                                     _L, _F, _I, _F, _P, _P, _I, _P])
+                                                     _L, _F, _I, _F, _P, _P, _I, _I, _P, _I, _P])
     _check(f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), _code(q, op), _ptr(block_tables),
              block_tables.shape[1], _ptr(row_seq), _ptr(positions), T, heads, kv_heads, dim, vdim, kcache.shape[2], int(window),
              float(scale), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, float(out_scale), int(chunk),
-             float(softcap), _ptr(r1), _ptr(r2), int(pool), _stream()), op)
+             float(softcap), _ptr(r1), _ptr(r2), int(pool), int(keep_first), _ptr(key_scale), gate_heads, _stream()), op)
 
 
 # ------------------------------------------------------------------------------------ attention
@@ -1678,31 +1785,43 @@ def attn_mma_supported(num_heads: int, num_kv_heads: int, head_dim: int, page_si
     return bool(f(num_heads, num_kv_heads, head_dim, page_size, int(decode)))
 
 
-def _attn_tail(op, q, sink, gate, num_heads, out_scale):
+def _attn_tail(op, q, sink, gate, num_heads, out_scale, per_head: bool = False):
     """Checked arguments of what may follow the weighted sum: a sink per head (float32 [H]), a gate ([T, H * hd] bfloat16,
-    any row stride: the result times its sigmoid) and a constant factor."""
+    any row stride: the result times its sigmoid; `per_head`: [T, H] is fine too) and a constant factor."""
     _cuda(op, q, sink, gate)
     _f32_vec(sink, num_heads, op, "sink")
-    if gate is not None:
-        _rows_2d(gate, op, "gate")
-        if gate.shape != q.shape or gate.dtype != torch.bfloat16:
-            raise ShapeError(op, f"gate must be bfloat16 {list(q.shape)}, got {gate.dtype} {list(gate.shape)}")
+    if _gate_cols(op, gate, q.shape[0], num_heads, q.shape[1] // num_heads, torch.bfloat16) and not per_head:
+        raise ShapeError(op, f"gate must be bfloat16 {list(q.shape)}, got {list(gate.shape)}")
     return _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, float(out_scale)
 
 
-def _score_shape(op, q, num_heads, chunk, softcap, dist_bias):
+def _score_shape(op, q, num_heads, chunk, softcap, dist_bias, window=0, keep_first=0, dist_slopes=None, key_scale=None, kcache=None,
+                 vcache=None, gate=None):
     """Checked arguments of what may shape a score before the softmax, or None where there is nothing: blocks of `chunk`
     positions (a query reads its own block's keys only), score <- softcap * tanh(score / softcap), and dist_bias = (r1, r2),
-    float32 [H] each: r1 * ln(1 + r2 * distance) taken off."""
-    if not chunk and not softcap and dist_bias is None:
+    float32 [H] each: r1 * ln(1 + r2 * distance) taken off; or dist_slopes, float32 [H]: slope * distance taken off.
+    `keep_first` (with a window): the keys of the first so many positions are seen whatever the window. `vcache is kcache`: the
+    values are the cached keys; q . k is then first multiplied by key j's number in `key_scale` (float32 [pages, 1, page_size, 1],
+    or None). Returns ((chunk, softcap, r1, r2), (keep_first, key_scale))."""
+    shared = kcache is not None and kcache is vcache
+    per_head = gate is not None and gate.shape[1] == num_heads and gate.shape[1] != q.shape[1]
+    if not chunk and not softcap and dist_bias is None and not keep_first and dist_slopes is None and not shared and not per_head:
         return None
-    if chunk < 0 or softcap < 0:
-        raise ShapeError(op, f"blocks of {chunk} and a cap of {softcap} must not be negative")
-    r1, r2 = dist_bias if dist_bias is not None else (None, None)
-    _cuda(op, q, r1, r2)
+    if chunk < 0 or softcap < 0 or keep_first < 0:
+        raise ShapeError(op, f"blocks of {chunk}, a cap of {softcap} and {keep_first} kept tokens must not be negative")
+    if keep_first and (window <= 0 or chunk):
+        raise ShapeError(op, "kept first tokens go with a window and without blocks of positions")
+    if dist_bias is not None and dist_slopes is not None:
+        raise ShapeError(op, "a bias on the logarithm of the distance or on the distance, not both")
+    if key_scale is not None and not shared:
+        raise ShapeError(op, "numbers per key go with values that are the cached keys")
+    r1, r2 = dist_bias if dist_bias is not None else (dist_slopes, None)
+    _cuda(op, q, r1, r2, key_scale)
+    if key_scale is not None:
+        _key_scales(op, key_scale, kcache)
     _f32_vec(r1, num_heads, op, "dist_bias[0]")
     _f32_vec(r2, num_heads, op, "dist_bias[1]")
-    return int(chunk), float(softcap), _ptr(r1), _ptr(r2)
+    return (int(chunk), float(softcap), _ptr(r1), _ptr(r2)), (int(keep_first), _ptr(key_scale))
 
 
 def _attn_common_checks(op, q, out, kcache, vcache, block_tables, num_heads, num_kv_heads, head_dim):
@@ -1761,16 +1880,18 @@ def attn_prefill_mma_any_supported(num_heads: int, num_kv_heads: int, dim: int, 
 @_timed
 def attn_prefill_mma_any(q, out, kcache, vcache, block_tables, seq_starts, context_lens, num_seqs: int, max_new: int,
                          num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float, window: int = 0, sink=None, gate=None,
-                         out_scale: float = 1.0, chunk: int = 0, softcap: float = 0.0, dist_bias=None, pooled=None) -> None:
+                         out_scale: float = 1.0, chunk: int = 0, softcap: float = 0.0, dist_bias=None, pooled=None,
+                         keep_first: int = 0, dist_slopes=None, key_scale=None) -> None:
     """Tensor-core attention for portions of prompts and mixed batches (bfloat16) with keys of `dim` and values of `vdim`
     features: q [T, H * dim], out [T, H * vdim] (any row stride), kcache [pages, KV, page, dim], vcache [pages, KV, page, vdim].
     The tiles in shared memory are padded with zero columns to the sizes the kernel is built for. Everything else as
-    `attn_prefill_mma`. `chunk`, `softcap`, `dist_bias`: see `_score_shape` (the kernel built for shaped scores runs then).
+    `attn_prefill_mma`. `chunk`, `softcap`, `dist_bias`, `keep_first`, `dist_slopes`, `key_scale` and `vcache is kcache`: see
+    `_score_shape` (the kernel built for shaped scores runs then; `gate` may have one column per head there).
     `pooled` = (kpool, vpool, pool), with a window: beside the window's tokens a query at position p sees the first
     floor((p + 1 - window) / pool) entries of kpool and vpool (laid out like the caches, entry b where a token at position b
     would be: the mean key and value of tokens b * pool .. b * pool + pool - 1, as `pool_blocks` leaves them)."""
     op = "attn_prefill_mma_any"
-    shape = _score_shape(op, q, num_heads, chunk, softcap, dist_bias)
+    shape = _score_shape(op, q, num_heads, chunk, softcap, dist_bias, window, keep_first, dist_slopes, key_scale, kcache, vcache, gate)
     pool_args = (_P(0), _P(0), 0)
     if pooled is not None:
         kpool, vpool, pool = pooled
@@ -1778,11 +1899,13 @@ def attn_prefill_mma_any(q, out, kcache, vcache, block_tables, seq_starts, conte
         if kpool.shape != kcache.shape or vpool.shape != vcache.shape or kpool.dtype != kcache.dtype or vpool.dtype != vcache.dtype \
                 or not kpool.is_contiguous() or not vpool.is_contiguous():
             raise ShapeError(op, "the pooled entries are laid out like the caches")
-        if pool <= 0 or window <= 0 or chunk or dist_bias is not None:
-            raise ShapeError(op, "pooled entries go with a window, without blocks of positions and without a distance bias")
+        if pool <= 0 or window <= 0 or chunk or dist_bias is not None or dist_slopes is not None or keep_first or kcache is vcache:
+            raise ShapeError(op, "pooled entries go with a window, without blocks of positions, kept first tokens and a distance bias")
         pool_args = (_ptr(kpool), _ptr(vpool), int(pool))
         if shape is None:
-            shape = (0, 0.0, _P(0), _P(0))
+            shape = ((0, 0.0, _P(0), _P(0)), (0, _P(0)))
+    if keep_first and kcache is not vcache:
+        raise ShapeError(op, "this kernel takes kept first tokens where the values are the cached keys")
     if shape is None and not scale > 0:
         raise ShapeError(op, f"the score scale must be positive, got {scale}")
     _cuda(op, q, out, kcache, vcache, block_tables, seq_starts, context_lens)
@@ -1804,10 +1927,9 @@ def attn_prefill_mma_any(q, out, kcache, vcache, block_tables, seq_starts, conte
     _int32_vec(context_lens, num_seqs, op, "context_lens")
     _cuda(op, q, sink, gate)
     _f32_vec(sink, num_heads, op, "sink")
-    if gate is not None:
-        _rows_2d(gate, op, "gate")
-        if gate.shape != out.shape or gate.dtype != torch.bfloat16:
-            raise ShapeError(op, f"gate must be bfloat16 {list(out.shape)}, got {gate.dtype} {list(gate.shape)}")
+    gate_heads = _gate_cols(op, gate, T, num_heads, vdim, torch.bfloat16)
+    if gate_heads and shape is None:
+        shape = ((0, 0.0, _P(0), _P(0)), (0, _P(0)))
     sig = [_P, _L, _P, _L, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _L, _F]
     args = (_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), _ptr(block_tables),
             block_tables.shape[1], _ptr(seq_starts), _ptr(context_lens), num_seqs, max_new, num_heads, num_kv_heads,
@@ -1816,7 +1938,8 @@ def attn_prefill_mma_any(q, out, kcache, vcache, block_tables, seq_starts, conte
     if shape is None:
         _check(_fn("attention_mma", "vob_attn_prefill_mma_any", sig + [_P])(*args, _stream()), op)
     else:
-        _check(_fn("attention_mma", "vob_attn_prefill_shaped", sig + [_I, _F, _P, _P, _P, _P, _I, _P])(*args, *shape, *pool_args, _stream()), op)
+        _check(_fn("attention_mma", "vob_attn_prefill_shaped", sig + [_I, _F, _P, _P, _P, _P, _I, _I, _P, _I, _P])(*args, *shape[0], *pool_args, *shape[1], gate_heads,
+                                                                                                                _stream()), op)
 
 
 def attn_prefill_sm100_supported(num_heads: int, num_kv_heads: int, head_dim: int, page_size: int, max_pages: int) -> bool:
@@ -1874,8 +1997,10 @@ def attn_prefill_sm100(q, out, kcache, vcache, block_tables, seq_starts, context
 @_timed
 def attn_decode_mma(q, out, kcache, vcache, block_tables, positions, num_heads: int, num_kv_heads: int, head_dim: int,
                     scale: float, window: int = 0, splits: int = 1, partials=None, arrived=None, sink=None, gate=None,
-                    out_scale: float = 1.0, chunk: int = 0, softcap: float = 0.0, dist_bias=None) -> None:
-    """`sink`, `gate`, `out_scale`: see `_attn_tail`; `chunk`, `softcap`, `dist_bias`: see `_score_shape`.
+                    out_scale: float = 1.0, chunk: int = 0, softcap: float = 0.0, dist_bias=None, keep_first: int = 0,
+                    dist_slopes=None, key_scale=None) -> None:
+    """`sink`, `gate`, `out_scale`: see `_attn_tail`; `chunk`, `softcap`, `dist_bias`, `keep_first`, `dist_slopes`, `key_scale` and
+    `vcache is kcache`: see `_score_shape` (`gate` may have one column per head there).
     Tensor-core attention for a step of single tokens, row i belonging to request i (bfloat16).
     With splits > 1 (at most 8) each request's keys are shared out over the blocks of a cluster,
     which merge their partial results through distributed shared memory. With `partials` (float32,
@@ -1883,7 +2008,7 @@ def attn_decode_mma(q, out, kcache, vcache, block_tables, positions, num_heads: 
     the kernel leaves them zero) up to 64 blocks share a request without a cluster and merge
     through global memory: for few requests with long contexts."""
     op = "attn_decode_mma"
-    shape = _score_shape(op, q, num_heads, chunk, softcap, dist_bias)
+    shape = _score_shape(op, q, num_heads, chunk, softcap, dist_bias, window, keep_first, dist_slopes, key_scale, kcache, vcache, gate)
     if shape is None and not scale > 0:
         raise ShapeError(op, f"the score scale must be positive, got {scale}")
     _attn_common_checks(op, q, out, kcache, vcache, block_tables, num_heads, num_kv_heads, head_dim)
@@ -1906,7 +2031,8 @@ def attn_decode_mma(q, out, kcache, vcache, block_tables, positions, num_heads: 
             raise ShapeError(op, f"partials must be contiguous float32, 16-byte aligned, with at least {need} elements")
         if arrived.dtype != torch.int32 or not arrived.is_contiguous() or arrived.numel() < S * num_kv_heads:
             raise ShapeError(op, f"arrived must be contiguous int32 with at least {S * num_kv_heads} elements")
-    tail = _attn_tail(op, q, sink, gate, num_heads, out_scale)
+    tail = _attn_tail(op, q, sink, gate, num_heads, out_scale, per_head=shape is not None)
+    gate_heads = _gate_cols(op, gate, S, num_heads, head_dim, torch.bfloat16)
     sig = [_P, _L, _P, _L, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _P, _L, _F]
     args = (_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kcache), _ptr(vcache), _ptr(block_tables),
             block_tables.shape[1], _ptr(positions), S, num_heads, num_kv_heads, head_dim, kcache.shape[2], int(window),
@@ -1914,7 +2040,7 @@ def attn_decode_mma(q, out, kcache, vcache, block_tables, positions, num_heads: 
     if shape is None:
         _check(_fn("attention_mma", "vob_attn_decode_mma", sig + [_P])(*args, _stream()), op)
     else:
-        _check(_fn("attention_mma", "vob_attn_decode_shaped", sig + [_I, _F, _P, _P, _P])(*args, *shape, _stream()), op)
+        _check(_fn("attention_mma", "vob_attn_decode_shaped", sig + [_I, _F, _P, _P, _I, _P, _I, _P])(*args, *shape[0], *shape[1], gate_heads, _stream()), op)
 
 
 def attn_decode_partial_floats(num_seqs: int, num_kv_heads: int, head_dim: int, splits: int) -> int:

@@ -45,14 +45,15 @@ class CacheSpec:
     """Pages a mixer needs. The mixer says which tensors a page holds: keys and values of
     `num_kv_heads` x `head_dim` (the default, `CacheSpec(kv_heads, head_dim)`), or any other set
     given as `tensors` (one latent vector per token, keys and values of different widths, ...),
-    and whether every token is kept ("full"), only the last `window` ("window") or only the current block of
-    `window` positions ("chunk")."""
+    and whether every token is kept ("full"), only the last `window` and the first `keep_first` ("window") or only the
+    current block of `window` positions ("chunk")."""
     num_kv_heads: int = 0
     head_dim: int = 0
     kind: str = "full"          # "full": every key is kept; "window": the last `window` keys; "chunk": the keys of
                                 # the query's own block of `window` positions (blocks counted from position 0)
     window: int = 0
     tensors: Tuple[PagedTensorSpec, ...] = ()
+    keep_first: int = 0         # "window": so many first tokens of a request are kept whatever the window
 
     def paged_tensors(self) -> Tuple[PagedTensorSpec, ...]:
         """The tensors of one page: `tensors` if given, else a key and a value tensor."""
@@ -62,7 +63,7 @@ class CacheSpec:
         return (kv, kv)
 
     def group_key(self) -> Tuple:
-        return (self.kind, self.window, self.paged_tensors())
+        return (self.kind, self.window, self.paged_tensors(), self.keep_first)
 
 
 @dataclass(frozen=True)
@@ -245,6 +246,7 @@ class Norm:
     # True for a norm that is a per-token scale times a per-feature weight (`weight`, `eps`):
     # that form commutes with a matrix product and can be folded into it (see FoldedState).
     scale_and_weight = False
+    scalar_scale = False        # True for a norm whose `forward` takes one number as `delta_scale`
 
     def workspace_bytes(self, rows: int, act_bytes: int) -> int:
         return 0
@@ -254,9 +256,9 @@ class Norm:
 
     def forward(self, resid: torch.Tensor, delta: Optional[torch.Tensor], ctx: StepContext,
                 rows: Optional[torch.Tensor] = None, num_rows: Optional[int] = None,
-                delta_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """`delta_scale` (float32 [hidden], only passed where a block has one): the delta is multiplied
-        by it, feature by feature, before it is added."""
+                delta_scale=None) -> torch.Tensor:
+        """`delta_scale` (only passed where a block has one): the delta is multiplied by it before it is added, feature by
+        feature (float32 [hidden]), or, for norms with `scalar_scale`, by one number."""
         raise NotImplementedError
 
 

@@ -9,7 +9,8 @@ at once: it is handed on as `pending` and the next norm's kernel adds it while i
 
 Options: a per-feature scale on each part's output before it is added (`mixer_scale`, `ff_scale`:
 the norm's kernel multiplies while it adds; `pending_scale` tells whoever adds this block's
-output which one goes with it), and a block without a feed-forward (`feed_forward` None:
+output which one goes with it), one number `residual_mult` in their place
+    (residual += m * mixer(norm1(residual)), and so on), and a block without a feed-forward (`feed_forward` None:
     residual += mixer(norm1(residual)) only; `norm2` is None then).
 """
 from __future__ import annotations
@@ -24,8 +25,15 @@ from .base import FeedForward, FoldedState, LayerCache, Mixer, Norm, StateSpec, 
 
 class Block:
     def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm], feed_forward: Optional[FeedForward],
-                 mixer_scale: Optional[torch.Tensor] = None, ff_scale: Optional[torch.Tensor] = None):
+                 mixer_scale: Optional[torch.Tensor] = None, ff_scale: Optional[torch.Tensor] = None,
+                 residual_mult: Optional[float] = None):
+        """`residual_mult`: one number every output is multiplied by before it is added (norms with `scalar_scale`)."""
         self.norm1, self.mixer, self.norm2, self.feed_forward = norm1, mixer, norm2, feed_forward
+        if residual_mult is not None:
+            if mixer_scale is not None or ff_scale is not None:
+                raise ValueError("a block has scales per feature or one multiplier, not both")
+            if not all(getattr(n, "scalar_scale", False) for n in (norm1, norm2) if n is not None):
+                raise ValueError("a block with a residual multiplier needs norms that take one number as the pending result's scale")
         if (norm2 is None) != (feed_forward is None):
             raise ValueError("a block has a second norm exactly when it has a feed-forward")
         dev = getattr(norm1, "weight", None)
@@ -35,6 +43,8 @@ class Block:
                 return None
             return t.to(device=dev.device if dev is not None else t.device, dtype=torch.float32).contiguous()
         self.mixer_scale, self.ff_scale = vec(mixer_scale), vec(ff_scale)
+        if residual_mult is not None and float(residual_mult) != 1.0:
+            self.mixer_scale = self.ff_scale = float(residual_mult)
         # the scale that goes with the output this block hands on
         self.pending_scale = self.ff_scale if feed_forward is not None else self.mixer_scale
 
@@ -42,7 +52,7 @@ class Block:
         return [p for p in (self.norm1, self.mixer, self.norm2, self.feed_forward) if p is not None]
 
     def weight_bytes(self) -> int:
-        scales = sum(t.numel() * 4 for t in (self.mixer_scale, self.ff_scale) if t is not None)
+        scales = sum(t.numel() * 4 for t in (self.mixer_scale, self.ff_scale) if isinstance(t, torch.Tensor))
         return scales + sum(getattr(p, "weight_bytes", lambda: 0)() for p in self._parts())
 
     def workspace_bytes(self, rows: int, hidden: int, act_bytes: int) -> int:
@@ -86,9 +96,9 @@ class Block:
             self.feed_forward.forward_folded(st, self.norm2.eps, ctx, next_norm.weight)
 
     def forward(self, resid: torch.Tensor, pending: Optional[torch.Tensor], ctx: StepContext,
-                cache: Optional[LayerCache], state, out: torch.Tensor, pending_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                cache: Optional[LayerCache], state, out: torch.Tensor, pending_scale=None) -> torch.Tensor:
         """Runs the block. `pending` is the previous block's output that is still to be added to
-        the residual (times `pending_scale`, if that block had one); the feed-forward's output
+        the residual (times `pending_scale`, per feature or one number, if that block had one); the feed-forward's output
         (again not yet added) is written to `out`, which outlives the block's own scratch."""
         ws = ctx.workspace
 

@@ -9,6 +9,8 @@ as parameters:
 * `dim` / `vdim`     key and value sizes of a head (the cache holds two tensors of different widths);
 * `bias_*`           biases of the q, k, v and output projections;
 * `window`           a query sees itself and the window - 1 tokens before it (pages behind are given back);
+* `keep_first`       (with `window`) every query also sees the request's first so many tokens, at their true distances
+                     (their pages stay);
 * `rot_dims`, `rot_base`   partial rotary positions, feature i paired with i + rot_dims / 2;
 * `unit_rms_eps`     q and k divided by sqrt(mean(x^2) + eps) per head, after the rotation;
 * `q_norm_weight`, `k_norm_weight`   [dim] each, shared by the heads: q and k times it behind that division;
@@ -24,13 +26,19 @@ as parameters:
                      (pages of earlier blocks are given back);
 * `softcap`          score <- softcap * tanh(score / softcap);
 * `dist_bias`        (r1, r2), one number per head each: r1 * ln(1 + r2 * (i - j)) is taken off the score of key j;
+* `dist_slopes`      one number per head: slope * (i - j) is taken off the score of key j;
+* `values_are_keys`  (`wv` None) the values are the keys as projected, before their norm. The cache holds them once, and
+                     beside them one float32 per token: the factor 1 / rms its keys are normed with. The norm's weights are
+                     taken into the query, q . (k / rms * w) = (q * w) . k / rms, so the normed keys are never stored; the
+                     attention kernels fetch one tile for both products. Goes with `q_pre_norm` and `k_pre_norm`, without rotation;
 * `shared_kv`        the layer has no key and value projections: it reads the cache another layer wrote (the run order
                      names it: `LayerCall(cache=that layer's, write=False)`), with its own queries, mask and the rest;
 * `cache_keep`       ("full" | "window" | "chunk", size): what the cache keeps where that is more than this layer's own
                      mask asks for (a cache that layers with different masks read must serve them all);
 * `q_temp`           (coef, every): q times 1 + coef * ln(floor((pos + 1) / every) + 1);
 * `sink`             one number per head whose exponential joins the softmax's denominator (no key, no value);
-* `gate_weight`      the heads' results times sigmoid(W_g x) before the output projection;
+* `gate_weight`      the heads' results times sigmoid(W_g x) before the output projection ([heads * vdim, hidden]: feature by
+                     feature; [heads, hidden] with `gate_per_head`: one number per head);
 * `value_mix`        "first": this layer's values of the step's tokens are left in `ctx.shared[shared_name]`;
                      "mix": v <- (1 - lambda) v + lambda * those values, before v is cached.
 
@@ -61,7 +69,17 @@ class SoftmaxAttention(Mixer):
                  k_norm_weight: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, dist_bias=None,
                  shared_kv: bool = False, cache_keep: Optional[Tuple[str, int]] = None, dtype=torch.bfloat16, device="cuda",
                  q_pre_norm: Optional[torch.Tensor] = None, k_pre_norm: Optional[torch.Tensor] = None,
-                 pre_norm_eps: Optional[float] = None, pool: int = 0, pooled_sizes: Optional[Tuple[int, ...]] = None):
+                 pre_norm_eps: Optional[float] = None, pool: int = 0, pooled_sizes: Optional[Tuple[int, ...]] = None,
+                 keep_first: int = 0, dist_slopes: Optional[torch.Tensor] = None, values_are_keys: bool = False,
+                 gate_per_head: bool = False):
+        self.values_are_keys = bool(values_are_keys)
+        if self.values_are_keys:
+            if wv is not None or bias_v is not None or shared_kv or value_mix or pool or rot_dims or unit_rms_eps is not None or q_temp:
+                raise ValueError("values that are the keys: no value tensors, no rotation, no norm per head, no query factor, no pooled "
+                                 "blocks and no other layer's keys")
+            if q_pre_norm is None or k_pre_norm is None or int(dim) != int(vdim):
+                raise ValueError("values that are the keys go with norms over the whole q and k projections and vdim = dim")
+            wv = torch.zeros((0, wq.shape[1]), dtype=wq.dtype, device=wq.device)
         self.H, self.G, self.D, self.DV = int(heads), int(kv_heads), int(dim), int(vdim)
         self.shared_kv = bool(shared_kv)
         if self.shared_kv:
@@ -77,16 +95,22 @@ class SoftmaxAttention(Mixer):
         nq, nk, nv = self.H * self.D, self.G * self.D, self.G * self.DV
         if self.shared_kv:
             nk = nv = 0
+        if self.values_are_keys:
+            nv = 0
         self.n_pre = self.H * self.DV
         if wq.shape != (nq, hidden) or wk.shape != (nk, hidden) or wv.shape != (nv, hidden) or wo.shape != (hidden, self.n_pre):
             raise ValueError(f"projection shapes {list(wq.shape)} / {list(wk.shape)} / {list(wv.shape)} / {list(wo.shape)} do not fit "
                              f"{self.H} heads on {self.G} of {self.D} / {self.DV} over a width of {hidden}")
         mats = [wq, wk, wv]
         self.gated = gate_weight is not None
+        self.n_gate = (self.H if gate_per_head else self.n_pre) if self.gated else 0
         if self.gated:
-            if gate_weight.shape != (self.n_pre, hidden):
-                raise ValueError(f"gate projection {list(gate_weight.shape)} does not fit {self.n_pre} x {hidden}")
+            if gate_weight.shape != (self.n_gate, hidden):
+                raise ValueError(f"gate projection {list(gate_weight.shape)} does not fit {self.n_gate} x {hidden}")
             mats.append(gate_weight)
+            pad = -(nq + nk + nv + self.n_gate) % 8
+            if gate_per_head and pad:            # the projection's rows keep starting on 16-byte boundaries
+                mats.append(torch.zeros((pad, hidden), dtype=wq.dtype, device=gate_weight.device))
         self.w_in = to_compute(torch.cat(mats, dim=0), dtype, device)
         self.q_off, self.k_off, self.v_off, self.g_off = 0, nq, nq + nk, nq + nk + nv
         biases = (bias_q, bias_k, bias_v)
@@ -97,8 +121,7 @@ class SoftmaxAttention(Mixer):
                 if b is not None and b.shape != (n,):
                     raise ValueError(f"a bias of {list(b.shape)} does not fit {n}")
                 parts.append(b.float() if b is not None else torch.zeros(n))
-            if self.gated:
-                parts.append(torch.zeros(self.n_pre))
+            parts.append(torch.zeros(self.w_in.shape[0] - nq - nk - nv))
             self.b_in = to_compute(torch.cat([p.to("cpu") for p in parts]), dtype, device)
         self.w_o = to_compute(wo, dtype, device)
         if bias_o is not None and bias_o.shape != (hidden,):
@@ -108,6 +131,9 @@ class SoftmaxAttention(Mixer):
         self.chunk = int(chunk) if chunk else 0
         if self.window < 0 or self.chunk < 0 or (self.window and self.chunk):
             raise ValueError(f"a window of {window} and blocks of {chunk}: one of them at most, none negative")
+        self.keep_first = int(keep_first) if keep_first else 0
+        if self.keep_first < 0 or (self.keep_first and (not self.window or pool)):
+            raise ValueError(f"{keep_first} kept first tokens go with a window and without pooled blocks")
         self.softcap = float(softcap) if softcap else 0.0
         if self.softcap < 0:
             raise ValueError(f"softcap {softcap} must be positive")
@@ -120,6 +146,8 @@ class SoftmaxAttention(Mixer):
             raise ValueError(f"the cache's block sizes {self.pooled_sizes} must be distinct, positive and hold this layer's {self.pool}")
         own = ("full", 0) if self.pool else ("window", self.window) if self.window else ("chunk", self.chunk) if self.chunk else ("full", 0)
         self.cache_keep = (str(cache_keep[0]), int(cache_keep[1])) if cache_keep is not None else own
+        if self.keep_first and (self.cache_keep != own or self.shared_kv):
+            raise ValueError("kept first tokens go with a cache that serves this layer alone")
         if self.cache_keep != own and self.cache_keep[0] != "full":
             raise ValueError(f"a cache that keeps {self.cache_keep} cannot serve a layer that reads {own}")
         self.scale = float(scale)
@@ -142,6 +170,10 @@ class SoftmaxAttention(Mixer):
             raise ValueError("a norm over the whole projection needs its eps and does not go with the norm per head")
         self.q_pre_w = q_pre_norm.to(**f32).contiguous() if q_pre_norm is not None else None
         self.k_pre_w = k_pre_norm.to(**f32).contiguous() if k_pre_norm is not None else None
+        self.qk_w = None
+        if self.values_are_keys:                 # a query head's weights times those of the kv head it reads
+            kw = self.k_pre_w.view(self.G, 1, self.D).expand(self.G, self.H // self.G, self.D)
+            self.qk_w = (self.q_pre_w.view(self.G, self.H // self.G, self.D) * kw).reshape(-1).contiguous()
         if pre_norm_eps is not None and not self.unit_rms:
             self.eps = float(pre_norm_eps)
         self.dist_bias = None
@@ -150,6 +182,11 @@ class SoftmaxAttention(Mixer):
             if r1.shape != (self.H,) or r2.shape != (self.H,):
                 raise ValueError(f"the distance bias takes two numbers per head, got {list(r1.shape)} and {list(r2.shape)}")
             self.dist_bias = (r1.to(**f32).contiguous(), r2.to(**f32).contiguous())
+        self.dist_slopes = None
+        if dist_slopes is not None:
+            if dist_bias is not None or dist_slopes.shape != (self.H,):
+                raise ValueError(f"a linear distance bias takes one number per head and excludes the other, got {list(dist_slopes.shape)}")
+            self.dist_slopes = dist_slopes.to(**f32).contiguous()
         if sink is not None and sink.shape != (self.H,):
             raise ValueError(f"sink {list(sink.shape)} does not fit {self.H} heads")
         self.sink = sink.to(**f32).contiguous() if sink is not None else None
@@ -168,8 +205,12 @@ class SoftmaxAttention(Mixer):
 
     # ------------------------------------------------------------------ what the runtime asks
     def cache_spec(self) -> Optional[CacheSpec]:
+        if self.values_are_keys:
+            return CacheSpec(kind=self.cache_keep[0], window=self.cache_keep[1], keep_first=self.keep_first,
+                             tensors=(PagedTensorSpec(self.G, self.D), PagedTensorSpec(1, 1, torch.float32)))
         kv = (PagedTensorSpec(self.G, self.D), PagedTensorSpec(self.G, self.DV))
-        return CacheSpec(kind=self.cache_keep[0], window=self.cache_keep[1], tensors=kv * (1 + len(self.pooled_sizes)))
+        return CacheSpec(kind=self.cache_keep[0], window=self.cache_keep[1], keep_first=self.keep_first,
+                         tensors=kv * (1 + len(self.pooled_sizes)))
 
     def shared_buffer(self) -> Optional[Tuple[str, int]]:
         """(name, columns) of the step buffer this mixer writes or reads, or None."""
@@ -188,7 +229,8 @@ class SoftmaxAttention(Mixer):
     def plain_scores(self) -> bool:
         """Scores that are q . k * scale and nothing else, over all earlier keys or a window: what the framework's
         tensor-core attention kernels compute."""
-        return not (self.chunk or self.softcap or self.dist_bias is not None or self.pool)
+        return not (self.chunk or self.softcap or self.dist_bias is not None or self.pool or self.keep_first
+                    or self.dist_slopes is not None or self.values_are_keys or self.n_gate not in (0, self.n_pre))
 
     def tensor_core_sizes(self) -> bool:
         """Keys and values of one size that the framework's tensor-core attention kernels are built for."""
@@ -196,7 +238,14 @@ class SoftmaxAttention(Mixer):
 
     def shape_args(self) -> dict:
         """What shapes this layer's scores before the softmax, as the kernels' keyword arguments."""
-        return dict(chunk=self.chunk, softcap=self.softcap, dist_bias=self.dist_bias)
+        return dict(chunk=self.chunk, softcap=self.softcap, dist_bias=self.dist_bias, keep_first=self.keep_first,
+                    dist_slopes=self.dist_slopes)
+
+    def kv(self, cache: LayerCache):
+        """(keys, values, a number per key or None) of this layer's cache, as the kernels take them."""
+        if self.values_are_keys:
+            return cache.tensors[0], cache.tensors[0], cache.tensors[1]
+        return cache.tensors[0], cache.tensors[1], None
 
     def padded_tile_sizes(self) -> bool:
         """Keys and values of sizes the portion kernel with padded tiles takes."""
@@ -225,8 +274,14 @@ class SoftmaxAttention(Mixer):
         if cache is None:
             raise ValueError("attention needs a cache")
         T = proj.shape[0]
-        kc, vc = cache.tensors[0], cache.tensors[1]
         q = ctx.alloc((T, self.H * self.D))
+        gate = proj[:, self.g_off:self.g_off + self.n_gate] if self.gated else None
+        if self.values_are_keys:
+            kernels.whole_norm_prep(proj, self.q_off, ctx.positions, ctx.slot_mapping[cache.group], self.qk_w, self.eps, q, cache.tensors[0],
+                                    cache.tensors[1], self.H, self.G, self.D)
+            self.attend(q, pre_out, ctx, cache, gate, out_scale)
+            return
+        kc, vc = cache.tensors[0], cache.tensors[1]
         v_first = ctx.shared.get(self.shared_name) if self.v_mode else None
         if self.v_mode and v_first is None:
             raise ValueError(f"the step has no buffer {self.shared_name!r} for the values that layers mix")
@@ -240,7 +295,6 @@ class SoftmaxAttention(Mixer):
             for i, size in enumerate(self.pooled_sizes):
                 kernels.pool_blocks(kc, vc, cache.tensors[2 + 2 * i], cache.tensors[3 + 2 * i], ctx.block_tables[cache.group], ctx.row_seq,
                                     ctx.positions, size)
-        gate = proj[:, self.g_off:self.g_off + self.n_pre] if self.gated else None
         self.attend(q, pre_out, ctx, cache, gate, out_scale)
 
     def attend(self, q, out, ctx: StepContext, cache: LayerCache, gate, out_scale: float) -> None:
@@ -250,11 +304,11 @@ class SoftmaxAttention(Mixer):
         go to the decode kernel and the portions behind them to the portion kernel. bfloat16 with keys and values of
         other sizes (multiples of 8 up to 128 each, different or not): portions and mixed steps go to the mma.sync
         portion kernel that pads its tiles, steps of single tokens to the general kernel. Scores that are shaped
-        before the softmax (blocks of positions, a cap, a distance bias) take the same two mma.sync kernels in their
+        before the softmax (blocks of positions, a cap, a distance bias, kept first tokens, a number per key) take the same two mma.sync kernels in their
         shaped build: the padded portion kernel for portions and mixed steps of any of those sizes, the split-key
         decode kernel for steps of single tokens with keys and values of one size of 64 or 128. Everything else
         (float32, other sizes) goes to the general kernel."""
-        kc, vc = cache.tensors[0], cache.tensors[1]
+        kc, vc, key_scale = self.kv(cache)
         page, bt = kc.shape[2], ctx.block_tables[cache.group]
         H, G, D = self.H, self.G, self.D
         if (self.dtype == torch.bfloat16 and self.impl != "general" and self.scale > 0 and self.tensor_core_sizes()
@@ -293,12 +347,13 @@ class SoftmaxAttention(Mixer):
             self._attend_single(q, out, ctx, cache, bt, ctx.rows, gate, out_scale)
             return
         if (self.dtype == torch.bfloat16 and self.impl != "general" and (self.scale > 0 or shaped) and not ctx.decode_only and ctx.max_new > 1
+                and (not self.keep_first or self.values_are_keys)
                 and kernels.attn_prefill_mma_any_supported(H, G, D, self.DV, page) and out.data_ptr() % 4 == 0 and out.stride(0) % 2 == 0):
             kernels.attn_prefill_mma_any(q, out, kc, vc, bt, ctx.seq_starts, ctx.context_lens, ctx.seqs, ctx.max_new, H, G, D, self.DV,
-                                         self.scale, self.window, self.sink, gate, out_scale, **self.shape_args())
+                                         self.scale, self.window, self.sink, gate, out_scale, key_scale=key_scale, **self.shape_args())
             return
         kernels.flex_attention(q, out, kc, vc, bt, ctx.row_seq, ctx.positions, H, G, D, self.DV, self.scale, self.window, self.sink,
-                               gate, out_scale, self.chunk, self.softcap, self.dist_bias)
+                               gate, out_scale, key_scale=key_scale, **self.shape_args())
 
     def _attend_single(self, q, out, ctx: StepContext, cache: LayerCache, bt, count: int, gate, out_scale: float) -> None:
         """The decode kernel on the first `count` rows, row i belonging to request i."""
@@ -307,10 +362,11 @@ class SoftmaxAttention(Mixer):
             floats = kernels.attn_decode_partial_floats(1, 1, self.D, 3 * self.num_sms)    # requests x kv heads x splits <= 3 SMs
             self._partials = torch.empty(floats, dtype=torch.float32, device=q.device)
             self._arrived = torch.zeros(self.num_sms, dtype=torch.int32, device=q.device)
-        kernels.attn_decode_mma(q[:count], out[:count], cache.tensors[0], cache.tensors[1], bt, ctx.positions[:count], self.H, self.G,
+        kc, vc, key_scale = self.kv(cache)
+        kernels.attn_decode_mma(q[:count], out[:count], kc, vc, bt, ctx.positions[:count], self.H, self.G,
                                 self.D, self.scale, self.window, splits, self._partials if wide else None,
                                 self._arrived if wide else None, self.sink, gate[:count] if gate is not None else None, out_scale,
-                                **self.shape_args())
+                                key_scale=key_scale, **self.shape_args())
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: Optional[LayerCache], state=None, out=None) -> torch.Tensor:
         T = x.shape[0]

@@ -1,7 +1,7 @@
 """Layer norm with weight and (optionally) bias: LN(z) = (z - mean) / sqrt(mean((z - mean)^2) + eps) * w + b, sums in float32.
 
 Two uses. As any norm of this engine it normalises the float32 residual (after adding what is still
-pending) for the part that follows: `forward`. In a block whose residual takes the NORMED result of each
+pending, times a constant if its block has one) for the part that follows: `forward`. In a block whose residual takes the NORMED result of each
 sub-layer (`PostNormBlock`) it normalises that result and adds it into the residual: `add_normed`, which
 can also leave the new residual in the activations' type for the sub-layer that reads it next.
 """
@@ -16,6 +16,7 @@ from .base import Norm, StepContext, aligned
 
 
 class LayerNorm(Norm):
+    scalar_scale = True           # `forward` takes one number as `delta_scale`
     scale_and_weight = False      # the mean and the bias do not commute with a matrix product: no folded form
 
     def __init__(self, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, device):
@@ -38,12 +39,17 @@ class LayerNorm(Norm):
 
     def forward(self, resid: torch.Tensor, delta: Optional[torch.Tensor], ctx: StepContext,
                 rows: Optional[torch.Tensor] = None, num_rows: Optional[int] = None,
-                delta_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
-        if delta is not None:
-            raise ValueError("this layer norm normalises the residual as it stands; a pending result must be added first")
+                delta_scale=None) -> torch.Tensor:
+        """`delta_scale`: one number."""
+        if isinstance(delta_scale, torch.Tensor):
+            raise ValueError("a layer norm adds the pending result times one number, not feature by feature")
         n = resid.shape[0] if rows is None else (num_rows if num_rows is not None else rows.numel())
         out = ctx.alloc((n, self.width))
-        kernels.layernorm_rows(resid, self.weight, self.bias, self.eps, out, rows[:n] if rows is not None else None)
+        r = rows[:n] if rows is not None else None
+        if delta is not None:
+            kernels.add_layernorm(resid, delta, self.weight, self.bias, self.eps, out, r, 1.0 if delta_scale is None else float(delta_scale))
+        else:
+            kernels.layernorm_rows(resid, self.weight, self.bias, self.eps, out, r)
         return out
 
     def add_normed(self, resid: torch.Tensor, result: torch.Tensor, copy: Optional[torch.Tensor] = None, depth=None, conv=None) -> None:

@@ -1,4 +1,4 @@
-"""Feed-forward made of many small gated experts of which every token uses a few.
+"""Feed-forward made of many small experts of which every token uses a few.
 
     z = W_router x (float32);  s = softmax(z) over all experts
     the experts form `groups` runs of neighbours; a run scores as its best expert; only experts of the `keep` best
@@ -8,6 +8,10 @@
 Options: `activation` "clamped_swish" with `limit` (g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) *
 (u + 1) in place of silu(gate) * up); `shared` = (w_gate, w_up, w_down, w_gate_scalar or None, limit): one more expert of the
 same form that every token uses, added to the sum, times sigmoid(w_gate_scalar x) (one number per token) where that is given.
+Experts without a gate (`w_gate` None) compute W_down[e] act(W_up[e] x) with `activation` "relu2" (relu squared). `score`
+"sigmoid": s = sigmoid(z); `correction` [E]: the election (groups and experts) goes by s + correction, the weights by s;
+`group_best` 2: a run scores as the sum of its two best experts; `renormalize` divides by the sum + `renorm_eps`; `weight_scale`
+multiplies the weights.
 Softmax over all experts followed by `renormalize` over the chosen ones is the softmax over the chosen logits alone.
 
 Per step: the election (one warp per token), the (token, expert) pairs put in order of their expert on the device
@@ -19,7 +23,7 @@ multiply-add chains over the features in order.
 """
 from __future__ import annotations
 
-from typing import Sequence
+from typing import Optional, Sequence
 
 import torch
 
@@ -30,13 +34,18 @@ from .linear import to_compute
 
 
 class RoutedExperts(FeedForward):
-    def __init__(self, w_router: torch.Tensor, w_gate: Sequence[torch.Tensor], w_up: Sequence[torch.Tensor],
+    def __init__(self, w_router: torch.Tensor, w_gate: Optional[Sequence[torch.Tensor]], w_up: Sequence[torch.Tensor],
                  w_down: Sequence[torch.Tensor], top: int, groups: int = 0, keep: int = 0, renormalize: bool = False,
-                 dtype=torch.bfloat16, device="cuda", activation: str = "silu", limit: float = 0.0, shared=None):
+                 dtype=torch.bfloat16, device="cuda", activation: str = "silu", limit: float = 0.0, shared=None,
+                 score: str = "softmax", correction: Optional[torch.Tensor] = None, group_best: int = 1, renorm_eps: float = 0.0,
+                 weight_scale: float = 1.0):
         E, hidden = w_router.shape
+        self.gated = w_gate is not None
+        if not self.gated:
+            w_gate = w_up                    # for the checks of sizes below
         if not (len(w_gate) == len(w_up) == len(w_down) == E):
             raise ValueError(f"the router names {E} experts, got {len(w_gate)} / {len(w_up)} / {len(w_down)} sets of weights")
-        ff = w_gate[0].shape[0]
+        ff = w_up[0].shape[0]
         for e in range(E):
             if w_gate[e].shape != (ff, hidden) or w_up[e].shape != (ff, hidden) or w_down[e].shape != (hidden, ff):
                 raise ValueError(f"expert {e}: shapes {list(w_gate[e].shape)} / {list(w_up[e].shape)} / {list(w_down[e].shape)} do not "
@@ -50,12 +59,24 @@ class RoutedExperts(FeedForward):
         self.renorm = bool(renormalize)
         # the router is float32 whatever the engine computes in
         self.w_router = w_router.to(device=device, dtype=torch.float32).contiguous()
-        self.w_gu = to_compute(torch.stack([torch.cat([g, u], dim=0) for g, u in zip(w_gate, w_up)]), dtype, device)
+        # [E, 2 ff, hidden], an expert's gate rows, then its up rows; without a gate [E, ff, hidden]
+        self.w_gu = to_compute(torch.stack([torch.cat([g, u], dim=0) for g, u in zip(w_gate, w_up)] if self.gated else list(w_up)), dtype, device)
         self.w_down = to_compute(torch.stack(list(w_down)), dtype, device)
         self.dtype = dtype
         self.tensor_cores = dtype == torch.bfloat16
         self.meta = torch.zeros(4, dtype=torch.int32, device=device)
-        if activation not in kernels.MOE_ACTIVATIONS or (activation == "clamped_swish" and not limit > 0):
+        if score not in kernels.MOE_SCORES or group_best not in (1, 2):
+            raise ValueError(f"score {score!r} ({', '.join(kernels.MOE_SCORES)}) or group_best {group_best} (1 or 2) is not known")
+        if correction is not None and correction.shape != (E,):
+            raise ValueError(f"a correction of {list(correction.shape)} does not fit {E} experts")
+        self.rule = dict(score=score, group_best=int(group_best), eps=float(renorm_eps), out_scale=float(weight_scale),
+                         correction=correction.to(device=device, dtype=torch.float32).contiguous() if correction is not None else None)
+        if not self.gated:
+            if activation not in kernels.MOE_UNGATED:
+                raise ValueError(f"activation {activation!r} of experts without a gate is not known ({', '.join(kernels.MOE_UNGATED)})")
+            if shared is not None:
+                raise ValueError("the shared expert has the routed experts' form, and this one is gated")
+        elif activation not in kernels.MOE_ACTIVATIONS or (activation == "clamped_swish" and not limit > 0):
             raise ValueError(f"activation {activation!r} with limit {limit}: known are {', '.join(kernels.MOE_ACTIVATIONS)}, and the "
                              f"clamped one needs a positive limit")
         self.activation, self.limit = activation, float(limit)
@@ -77,7 +98,7 @@ class RoutedExperts(FeedForward):
         """What a step of one token reads: the router and `top` experts."""
         es = self.w_down.element_size()
         shared = (self.shared[0].numel() + self.shared[1].numel()) * es if self.shared is not None else 0
-        return self.w_router.numel() * 4 + self.top * 3 * self.ff * self.hidden * es + shared
+        return self.w_router.numel() * 4 + self.top * (3 if self.gated else 2) * self.ff * self.hidden * es + shared
 
     def workspace_bytes(self, rows: int) -> int:
         es = 2 if self.dtype == torch.bfloat16 else 4
@@ -122,14 +143,17 @@ class RoutedExperts(FeedForward):
                     self._shared_expert(x, gu, hs, sh)
             else:
                 self._shared_expert(x, gu, hs, sh)
-        kernels.moe_route(x, self.w_router, ctx.positions, self.top, self.groups, self.keep, self.renorm, idx, w)
+        kernels.moe_route(x, self.w_router, ctx.positions, self.top, self.groups, self.keep, self.renorm, idx, w, **self.rule)
         large = x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
         tile = kernels.moe_tile_rows(P, self.E, self.hidden, self.ff, self.tensor_cores and large)
         cap = kernels.moe_sorted_rows(P, self.E, tile)
         order, tile_expert = ctx.alloc((cap,), torch.int32), ctx.alloc((cap // tile,), torch.int32)
         kernels.moe_align(idx, self.E, order, tile_expert, self.meta, tile)
         h = ctx.alloc((P, self.ff))
-        kernels.moe_gate_up(x, self.w_gu, order, tile_expert, self.top, h, self.tensor_cores, tile, self.activation, self.limit)
+        if self.gated:
+            kernels.moe_gate_up(x, self.w_gu, order, tile_expert, self.top, h, self.tensor_cores, tile, self.activation, self.limit)
+        else:
+            kernels.moe_up(x, self.w_gu, order, tile_expert, self.top, h, self.activation, self.tensor_cores, tile)
         y = ctx.alloc((P, self.hidden), torch.float32)
         kernels.moe_down(h, self.w_down, order, tile_expert, w, y, self.tensor_cores, tile)
         out = out if out is not None else ctx.alloc((T, self.hidden))
