@@ -1805,7 +1805,7 @@ def _score_shape(op, q, num_heads, chunk, softcap, dist_bias, window=0, keep_fir
     or None). Returns ((chunk, softcap, r1, r2), (keep_first, key_scale))."""
     shared = kcache is not None and kcache is vcache
     per_head = gate is not None and gate.shape[1] == num_heads and gate.shape[1] != q.shape[1]
-    if not chunk and not softcap and dist_bias is None and not keep_first and dist_slopes is None and not shared and not per_head:
+    if not chunk and not softcap and dist_bias is None and not keep_first and dist_slopes is None and not shared and not per_head and key_scale is None:
         return None
     if chunk < 0 or softcap < 0 or keep_first < 0:
         raise ShapeError(op, f"blocks of {chunk}, a cap of {softcap} and {keep_first} kept tokens must not be negative")
