@@ -1210,6 +1210,123 @@ def pironex_compare(a):
     return 0
 
 
+# Layer sizes at which the Fanopel design is measured beside Bufulorn, the closest design the engine has (capped scores with a
+# distance bias, a gate on the heads' results, routed experts chosen among the best groups, layer norms), both built of the same
+# number of layers of attention and experts with the same width, heads and experts (those of BUFULORN_SIZES).
+FANOPEL_SIZES = {
+    "1b": dict(bufulorn="1b", window=1024, keep_first=16, softcap=30.0, scale=2.5),
+    "3b": dict(bufulorn="3b", window=1024, keep_first=16, softcap=30.0, scale=2.5),
+}
+
+
+def make_experts_engine(arch, fs, layers, max_seqs, tokens_per_request, context):
+    """(config, LLM): `layers` layers of attention and routed experts, of the Fanopel or the Bufulorn design, random weights
+    drawn on the device."""
+    import torch
+    from vllm_oxide_b200 import models
+    from vllm_oxide_b200 import config as cf
+    from vllm_oxide_b200.engine import LLM, ModelRunner
+    from vllm_oxide_b200.weights import random_tensors
+    bs = BUFULORN_SIZES[fs["bufulorn"]]
+    ls = LOMOPEL_SIZES[bs["lomopel"]]
+    at = ls["attn"]
+    common = dict(vocab=128256, width=ls["width"], norm_eps=1e-5, max_positions=context)
+    if arch == "fanopel":
+        a = cf.KeyValueAttentionConfig(heads=at["heads"], kv_heads=at["kv_heads"], dim=at["dim"], scale=at["dim"] ** -0.5, softcap=fs["softcap"],
+                                       window=fs["window"], keep_first=fs["keep_first"])
+        cfg = cf.FanopelConfig(layers=(cf.FanopelLayer(a, cf.PlainExpertsConfig(scale=fs["scale"], **bs["moe"])),) * layers, residual_mult=0.5, **common)
+        manifest = models.fanopel_manifest(cfg)
+    else:
+        a = cf.ChunkAttentionConfig(scale=at["dim"] ** -0.5, softcap=bs["softcap"], chunk=bs["chunk"], **at)
+        cfg = cf.BufulornConfig(layers=(cf.BufulornLayer("attention", attention=a, mlp=cf.FeedForwardConfig("moe", **bs["moe"])),) * layers, **common)
+        manifest = models.bufulorn_manifest(cfg)
+    pages_per_req = -(-(tokens_per_request + 16) // 16)
+    fields = dict(max_batch_tokens=2048, max_seqs=max_seqs, max_model_len=context, block_size=16,
+                  num_pages=max_seqs * pages_per_req + 8, dtype="bfloat16", cuda_graphs=True)
+    fields.update(ENGINE_OVERRIDES)
+    tensors = random_tensors(manifest, seed=0, std=0.02, dtype=torch.bfloat16, device="cuda:0")
+    runner = ModelRunner(cfg, tensors, cf.EngineConfig(**fields))
+    del tensors
+    return cfg, LLM(runner)
+
+
+def experts_roofline(arch, fs, layers, n, batch, peaks, prefill, decode):
+    """The kernels of attention-and-experts layers against their rooflines: algorithmic bytes (or FLOPs) of all their launches in
+    one step over the measured time, as a fraction of the measured copy bandwidth (or the measured bfloat16 product rate)."""
+    bs = BUFULORN_SIZES[fs["bufulorn"]]
+    ls = LOMOPEL_SIZES[bs["lomopel"]]
+    at, W, m, new = ls["attn"], ls["width"], bs["moe"], arch == "fanopel"
+    out = {}
+
+    def add(names, label, phase, totals, nbytes=None, flops=None):
+        ms = sum(t for op, _, t in totals if op in names)
+        if ms <= 0:
+            return
+        e = {"ms": round(ms, 4)}
+        if nbytes is not None:
+            e["gbs"] = round(nbytes / ms / 1e6, 1)
+            e["of_measured_hbm"] = round(nbytes / ms / 1e6 / peaks["hbm_gbs"], 4)
+        if flops is not None:
+            e["tflops"] = round(flops / ms / 1e9, 2)
+            e["of_measured_bf16"] = round(flops / ms / 1e9 / peaks["bf16_tflops"], 4)
+        out[f"{phase}:{label}"] = e
+    qd, kd, vd = at["heads"] * at["dim"], at["kv_heads"] * at["dim"], at["kv_heads"] * at["vdim"]
+
+    def seen(p):       # keys a query at position p reads
+        return min(p + 1, fs["window"]) + max(0, min(fs["keep_first"], p + 1 - fs["window"])) if new else p % bs["chunk"] + 1
+    for phase, rows, totals in (("prefill", n, prefill), ("decode", batch, decode)):
+        # every norm: the float32 residual read and written, the sub-layer's result read, the type the next product reads written
+        add(("add_layernorm", "layernorm_add", "layernorm_rows", "cast_rows"), "layer norms", phase, totals, nbytes=2 * layers * rows * W * (2 + 2 * 4 + 2))
+        keys = sum(seen(i) for i in range(n)) if phase == "prefill" else batch * seen(n + 2)
+        per_key = kd * 2 + 4 if new else (kd + vd) * 2
+        add(("flex_attention", "attn_prefill_mma_any", "attn_prefill_mma", "attn_decode_mma"), "attention", phase, totals,
+            nbytes=layers * keys * per_key if phase == "decode" else None, flops=layers * keys * at["heads"] * 2 * (at["dim"] + at["vdim"]))
+        add(("flex_prep", "whole_norm_prep"), "preparation of q, k (and v)", phase, totals,
+            nbytes=layers * rows * 2 * (qd + kd + (0 if new else vd)) * 2)
+        P, used, mats = rows * m["top"], min(m["experts"], rows * m["top"]), 2 if new else 3
+        add(("moe_gate_up", "moe_up", "moe_down"), "expert products", phase, totals,
+            nbytes=layers * (used * mats * m["ff"] * W * 2 + P * (W * 2 + 2 * m["ff"] * 2 + W * 4)), flops=layers * P * mats * 2 * m["ff"] * W)
+        add(("moe_route", "moe_align", "moe_combine"), "election, order, sum", phase, totals,
+            nbytes=layers * (rows * W * 2 + m["experts"] * W * 4 + P * W * 4 + rows * W * 2))
+    return out
+
+
+def fanopel_compare(a):
+    """Prefill and decode of the Fanopel design beside Bufulorn layers of attention and experts of the same width, layer count,
+    heads and experts; one JSON line. Device-timed like the benchmark's own points: one step of 2,048 prompt tokens (median of 5
+    after 3), decode steps replayed from CUDA graphs (`--steps` steps a region, median region)."""
+    import torch
+    peaks = load_peaks()
+    n, B, layers = 2048, a.batch, 8
+    gen = a.warmup + max(a.steps, MAX_TIMED_STEPS) + 64
+    sampler = ClockSampler()
+    sampler.start()
+    points = []
+    for key in a.fanopel.split(","):
+        fs = FANOPEL_SIZES[key]
+        point = {"sizes": key, "layers": layers, "prompt_len": n, "batch": B}
+        for arch in ("fanopel", "bufulorn"):
+            cfg, llm = make_experts_engine(arch, fs, layers, B, n + gen, 8192)
+            g = torch.Generator().manual_seed(1)
+            prompts = [torch.randint(0, cfg.vocab, (n,), generator=g).tolist() for _ in range(B)]
+            ms_prefill = timed_prefill(llm, prompts[0], n)
+            ms_step, ctx_tokens, launches, regions = decode_device(llm, prompts, B, a.steps, a.warmup, n, gen)
+            prefill, decode = op_profile(llm, prompts, n, B)
+            point[arch] = {"prefill_tok_s": round(n / ms_prefill * 1e3, 1), "prefill_ms": round(ms_prefill, 3),
+                           "decode_tok_s": round(B / ms_step * 1e3, 1), "decode_ms_per_step": round(ms_step, 4),
+                           "cache_bytes_per_token": llm.runner.pools.bytes_per_token(), "launches_per_decode_step": launches // a.steps,
+                           "ops_prefill_ms": {op: round(t, 4) for op, _, t in prefill}, "ops_decode_ms": {op: round(t, 4) for op, _, t in decode},
+                           "kernels": experts_roofline(arch, fs, layers, n, B, peaks, prefill, decode)}
+            free_engine(llm)
+            del llm
+        points.append(point)
+    clocks = sampler.stop()
+    print(json.dumps({"metric": "Fanopel beside Bufulorn (attention and experts in every layer) at equal width, layer count, heads and experts: "
+                                "prefill and decode tok/s",
+                      "dtype": "bf16", "data": "synthetic", "peaks": peaks, "points": points, "clocks": clocks, "run": run_record()}))
+    return 0
+
+
 def main():
     if "--kernel" in sys.argv[1:]:
         return kernel_case(sys.argv[1:])
@@ -1248,6 +1365,9 @@ def main():
     ap.add_argument("--pironex", default=None, metavar="SIZES", const="1b,3b", nargs="?",
                     help="instead of the benchmark's line: the Pironex design beside Bufulorn at equal sizes (1b, 3b or both), "
                          "prefill and decode, with the time and roofline fraction of every kernel")
+    ap.add_argument("--fanopel", default=None, metavar="SIZES", const="1b,3b", nargs="?",
+                    help="instead of the benchmark's line: the Fanopel design beside Bufulorn at equal sizes (1b, 3b or both), "
+                         "prefill and decode, with the time and roofline fraction of every kernel")
     ap.add_argument("--tuning", action="append", default=[], metavar="FIELD=VALUE",
                     help="set a field of vllm_oxide_b200.tuning.TUNING (experiments)")
     ap.add_argument("--fold-rows", type=int, default=None, metavar="R",
@@ -1281,6 +1401,8 @@ def main():
         return bufulorn_compare(a)
     if a.pironex:
         return pironex_compare(a)
+    if a.fanopel:
+        return fanopel_compare(a)
     prompt_len, gen_len = a.prompt_len, a.gen_len
     max_b = max(a.batch, 1 if (a.no_points or a.serve or a.timeline) else 64)
     if a.serve:

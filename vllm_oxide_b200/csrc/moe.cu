@@ -578,7 +578,8 @@ template <int N> __device__ __forceinline__ void moe_cp_wait() { asm volatile("c
 
 enum MoeProduct { MOE_GATE_UP = 0, MOE_DOWN = 1, MOE_UP = 2 };
 
-template <int BM, int STAGES, int KIND>
+// WROWS: weight rows of a block, 128, or 64 (single products in tiles of 32: twice the blocks where few tiles are in use).
+template <int BM, int STAGES, int KIND, int WROWS>
 __global__ void __launch_bounds__(BM == 128 ? 256 : 128)
 moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const __nv_bfloat16* __restrict__ w,
                 const int* __restrict__ sorted, const int* __restrict__ tile_expert, const float* __restrict__ pair_w,
@@ -588,7 +589,9 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
     constexpr int WR = BM == 128 ? 2 : 1;             // warps along the rows
     constexpr int NT = 128 * WR;
     constexpr int RF = BM / WR / 16;                   // 16-row fragments a warp owns
-    constexpr int ROWS = BM + 128;                     // rows of a stage: the pairs, then the weight rows
+    static_assert(WROWS == 128 || KIND != MOE_GATE_UP, "a gate and its up rows take 64 rows each");
+    constexpr bool TWO = WROWS == 128;                 // a warp owns two fragments of columns, 64 apart
+    constexpr int ROWS = BM + WROWS;                   // rows of a stage: the pairs, then the weight rows
     constexpr int CHUNKS = (ROWS * (VOB_MOE_PK / 8) + NT - 1) / NT;
     const int tile = blockIdx.x;
     const int e = tile_expert[tile];
@@ -597,7 +600,7 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
     __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(moe_smem);
     __shared__ int pair_of[BM];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wc = warp & 3, wr = warp >> 2;
-    const int col0 = blockIdx.y * (KIND != MOE_GATE_UP ? 128 : 64);
+    const int col0 = blockIdx.y * (KIND != MOE_GATE_UP ? WROWS : 64);
     // the rows this thread fetches, the same in every stage
     const __nv_bfloat16* src[CHUNKS];
     int dst_off[CHUNKS], feat[CHUNKS];
@@ -654,13 +657,13 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
         for (int kk = 0; kk < VOB_MOE_PK; kk += 16) {
             wmma::fragment<wmma::matrix_b, 16, 16, 16, __nv_bfloat16, wmma::col_major> b0, b1;
             wmma::load_matrix_sync(b0, Bs + (wc * 16) * VOB_MOE_PLD + kk, VOB_MOE_PLD);
-            wmma::load_matrix_sync(b1, Bs + (64 + wc * 16) * VOB_MOE_PLD + kk, VOB_MOE_PLD);
+            if (TWO) wmma::load_matrix_sync(b1, Bs + (64 + wc * 16) * VOB_MOE_PLD + kk, VOB_MOE_PLD);
 #pragma unroll
             for (int i = 0; i < RF; ++i) {
                 wmma::fragment<wmma::matrix_a, 16, 16, 16, __nv_bfloat16, wmma::row_major> fa;
                 wmma::load_matrix_sync(fa, As + (wr * (BM / WR) + 16 * i) * VOB_MOE_PLD + kk, VOB_MOE_PLD);
                 wmma::mma_sync(c0[i], fa, b0, c0[i]);
-                wmma::mma_sync(c1[i], fa, b1, c1[i]);
+                if (TWO) wmma::mma_sync(c1[i], fa, b1, c1[i]);
             }
         }
     }
@@ -670,7 +673,7 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
 #pragma unroll
     for (int i = 0; i < RF; ++i) {
         wmma::store_matrix_sync(Cs, c0[i], 16, wmma::mem_row_major);
-        wmma::store_matrix_sync(Cs + 256, c1[i], 16, wmma::mem_row_major);
+        if (TWO) wmma::store_matrix_sync(Cs + 256, c1[i], 16, wmma::mem_row_major);
         __syncwarp();
         for (int el = lane; el < 256; el += 32) {
             const int r = el >> 4, c = el & 15;
@@ -680,13 +683,13 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
                 __nv_bfloat16* ho = reinterpret_cast<__nv_bfloat16*>(out) + (size_t)p * N;
                 const int ca = col0 + wc * 16 + c, cb = ca + 64;
                 if (ca < N) ho[ca] = __float2bfloat16_rn(moe_act(Cs[el], act));
-                if (cb < N) ho[cb] = __float2bfloat16_rn(moe_act(Cs[256 + el], act));
+                if (TWO && cb < N) ho[cb] = __float2bfloat16_rn(moe_act(Cs[256 + el], act));
             } else if (KIND == MOE_DOWN) {
                 float* y = reinterpret_cast<float*>(out);
                 const float wgt = pair_w[p];
                 const int ca = col0 + wc * 16 + c, cb = ca + 64;
                 if (ca < N) y[(size_t)p * N + ca] = wgt * Cs[el];
-                if (cb < N) y[(size_t)p * N + cb] = wgt * Cs[256 + el];
+                if (TWO && cb < N) y[(size_t)p * N + cb] = wgt * Cs[256 + el];
             } else {
                 const int col = col0 + wc * 16 + c;
                 if (col < N) {
@@ -700,17 +703,17 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
     }
 }
 
-template <int BM, int STAGES, int KIND>
+template <int BM, int STAGES, int KIND, int WROWS = 128>
 static int moe_pipe_launch(dim3 grid, cudaStream_t stream, const __nv_bfloat16* a, long ld_a, int a_div, const __nv_bfloat16* w,
                            const int* sorted, const int* tile_expert, const float* pair_w, int K, int N, void* out, int act = 0, float limit = 0.f) {
-    const size_t smem = (size_t)STAGES * (BM + 128) * VOB_MOE_PLD * sizeof(__nv_bfloat16);
+    const size_t smem = (size_t)STAGES * (BM + WROWS) * VOB_MOE_PLD * sizeof(__nv_bfloat16);
     static bool raised = false;
     if (!raised) {
-        cudaError_t err = cudaFuncSetAttribute(moe_pipe_kernel<BM, STAGES, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t err = cudaFuncSetAttribute(moe_pipe_kernel<BM, STAGES, KIND, WROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (err != cudaSuccess) return (int)err;
         raised = true;
     }
-    return vob_launch(moe_pipe_kernel<BM, STAGES, KIND>, grid, dim3(BM == 128 ? 256 : 128), smem, stream, a, ld_a, a_div, w, sorted,
+    return vob_launch(moe_pipe_kernel<BM, STAGES, KIND, WROWS>, grid, dim3(BM == 128 ? 256 : 128), smem, stream, a, ld_a, a_div, w, sorted,
                       tile_expert, pair_w, K, N, out, act, limit);
 }
 
@@ -756,7 +759,7 @@ VOB_EXPORT int vob_moe_down(const void* h, int code, const void* w_down, const i
         if (moe_rows_by16(h, ff, ff) && moe_rows_by16(w_down, ff, ff)) {
             const dim3 grid(max_tiles, (width + 127) / 128);
             if (tile_rows == 128) return moe_pipe_launch<128, 3, MOE_DOWN>(grid, stream, ha, ff, 1, wa, sorted, tile_expert, pair_w, ff, width, y);
-            return moe_pipe_launch<32, 4, MOE_DOWN>(grid, stream, ha, ff, 1, wa, sorted, tile_expert, pair_w, ff, width, y);
+            return moe_pipe_launch<32, 6, MOE_DOWN>(grid, stream, ha, ff, 1, wa, sorted, tile_expert, pair_w, ff, width, y);
         }
         if (tile_rows != VOB_MOE_BM) return VOB_ERR_UNSUPPORTED;
         return vob_launch(moe_single_tc_kernel<false>, dim3(max_tiles, (width + 63) / 64), dim3(128), 0, stream, ha, (long)ff, 1, wa, sorted,
@@ -781,7 +784,7 @@ VOB_EXPORT int vob_moe_up(const void* x, int code, long ld_x, const void* w_up, 
         if (moe_rows_by16(x, ld_x, width) && moe_rows_by16(w_up, width, width)) {
             const dim3 grid(max_tiles, (ff + 127) / 128);
             if (tile_rows == 128) return moe_pipe_launch<128, 3, MOE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act);
-            return moe_pipe_launch<32, 4, MOE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act);
+            return moe_pipe_launch<32, 8, MOE_UP, 64>(dim3(max_tiles, (ff + 63) / 64), stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act);
         }
         if (tile_rows != VOB_MOE_BM) return VOB_ERR_UNSUPPORTED;
         return vob_launch(moe_single_tc_kernel<true>, dim3(max_tiles, (ff + 63) / 64), dim3(128), 0, stream, xa, ld_x, top, wa, sorted, tile_expert,
