@@ -24,9 +24,11 @@
 VOB_PDL_SWITCH(moe)
 
 #define VOB_MOE_BM 32
+#define VOB_MOE_ROUTE_FEW 128      // tokens of a step up to which the election takes a block per token
 
 // ---------------------------------------------------------------------------------------------
-// Routing. Four tokens per block, one warp per token for the election; 2 E floats of shared memory per token.
+// Routing. Four tokens per block of four warps, or one token per block of sixteen warps where the step has few tokens (the
+// same sums bit for bit); one warp per token for the election; 3 E floats of shared memory per token.
 // Rows with a negative position (padding) choose nothing: their indices are -1.
 // ---------------------------------------------------------------------------------------------
 __device__ __forceinline__ void warp_argmax(float& v, int& i) {
@@ -49,8 +51,8 @@ template <> __device__ __forceinline__ void moe_ld4<__nv_bfloat16>(const __nv_bf
     v[0] = __bfloat162float(lo.x); v[1] = __bfloat162float(lo.y); v[2] = __bfloat162float(hi.x); v[3] = __bfloat162float(hi.y);
 }
 
-// The block's four warps first share out the experts: a warp reads an expert's router row once and multiplies it with
-// the rows of all four tokens (a lane's chain runs over its own features in order, whoever the other tokens are; rows
+// The block's warps first share out the experts: a warp reads an expert's router row once and multiplies it with
+// the rows of all the block's tokens (a lane's chain runs over its own features in order, whoever the other tokens are; rows
 // whose width and addresses allow are read four features at a time). Then warp w holds the election of token w.
 struct RouteRule {
     int sigmoid;               // scores: 0 softmax over all experts, 1 sigmoid of each logit
@@ -60,8 +62,9 @@ struct RouteRule {
     float eps, out_scale;
 };
 
-template <typename T>
-__global__ void __launch_bounds__(128)
+// TPB: tokens per block; WARPS: its warps, at least TPB.
+template <typename T, int TPB, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32)
 moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w_router, const int* __restrict__ positions,
                  int T_rows, int width, int E, int top, int n_groups, int keep, RouteRule rule, int* __restrict__ idx_out,
                  float* __restrict__ w_out) {
@@ -69,20 +72,22 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
     pdl_wait(71);
     extern __shared__ float sc_all[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int t0 = blockIdx.x * 4;
-    const T* rows[4];
+    const int t0 = blockIdx.x * TPB;
+    const T* rows[TPB];
 #pragma unroll
-    for (int k = 0; k < 4; ++k) rows[k] = x + (size_t)min(t0 + k, T_rows - 1) * ld_x;
+    for (int k = 0; k < TPB; ++k) rows[k] = x + (size_t)min(t0 + k, T_rows - 1) * ld_x;
     const bool by4 = width % 4 == 0 && ld_x % 4 == 0 && (((uintptr_t)x) & (4 * sizeof(T) - 1)) == 0 && (((uintptr_t)w_router) & 15) == 0;
-    for (int e = warp; e < E; e += 4) {
+    for (int e = warp; e < E; e += WARPS) {
         const float* wr = w_router + (size_t)e * width;
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        float acc[TPB];
+#pragma unroll
+        for (int k = 0; k < TPB; ++k) acc[k] = 0.f;
         if (by4) {
-#pragma unroll 2
+#pragma unroll (TPB == 1 ? 8 : 2)
             for (int i = lane * 4; i < width; i += 128) {
                 const float4 w4 = *reinterpret_cast<const float4*>(wr + i);
 #pragma unroll
-                for (int k = 0; k < 4; ++k) {
+                for (int k = 0; k < TPB; ++k) {
                     float v[4];
                     moe_ld4<T>(rows[k] + i, v);
                     acc[k] = fmaf(v[0], w4.x, acc[k]); acc[k] = fmaf(v[1], w4.y, acc[k]);
@@ -93,25 +98,25 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
             for (int i = lane; i < width; i += 32) {
                 const float w1 = wr[i];
 #pragma unroll
-                for (int k = 0; k < 4; ++k) acc[k] = fmaf(ld_f(rows[k] + i), w1, acc[k]);
+                for (int k = 0; k < TPB; ++k) acc[k] = fmaf(ld_f(rows[k] + i), w1, acc[k]);
             }
         }
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
+        for (int k = 0; k < TPB; ++k) {
             const float total = warp_sum(acc[k]);
-            if (lane == 0) sc_all[(size_t)k * 2 * E + e] = total;
+            if (lane == 0) sc_all[(size_t)k * 3 * E + e] = total;
         }
     }
     __syncthreads();
     const int t = t0 + warp;
-    if (t >= T_rows) return;
+    if (warp >= TPB || t >= T_rows) return;
     if (positions && positions[t] < 0) {
         for (int k = lane; k < top; k += 32) { idx_out[(size_t)t * top + k] = -1; w_out[(size_t)t * top + k] = 0.f; }
         return;
     }
-    // the scores, then the choice scores the election strikes names from (-inf: does not stand)
-    float* sc = sc_all + (size_t)warp * 2 * E;
-    float* cand = sc + E;
+    // the scores, the choice scores, and the choice scores the election strikes names from (-inf: does not stand)
+    float* sc = sc_all + (size_t)warp * 3 * E;
+    float *choice = sc + E, *cand = sc + 2 * E;
     __syncwarp();
     float m = 0.f, sum = 1.f;
     if (!rule.sigmoid) {
@@ -122,10 +127,12 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
         for (int e = lane; e < E; e += 32) sum += expf(sc[e] - m);
         sum = warp_sum(sum);
     }
-    auto choice = [&](int e) { return rule.correction ? sc[e] + rule.correction[e] : sc[e]; };
     for (int e = lane; e < E; e += 32) {
-        sc[e] = rule.sigmoid ? 1.0f / (1.0f + expf(-sc[e])) : expf(sc[e] - m) / sum;
-        cand[e] = (n_groups > 1) ? -INFINITY : choice(e);         // with groups: nobody stands until the group is kept
+        const float s = rule.sigmoid ? 1.0f / (1.0f + expf(-sc[e])) : expf(sc[e] - m) / sum;
+        const float c = rule.correction ? s + rule.correction[e] : s;
+        sc[e] = s;
+        choice[e] = c;
+        cand[e] = (n_groups > 1) ? -INFINITY : c;         // with groups: nobody stands until the group is kept
     }
     __syncwarp();
     if (n_groups > 1) {
@@ -138,7 +145,7 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
                 if (cand[g * per] > -INFINITY) continue;            // group already kept (its experts stand)
                 float best = -INFINITY, second = -INFINITY;
                 for (int j = 0; j < per; ++j) {
-                    const float c = choice(g * per + j);
+                    const float c = choice[g * per + j];
                     second = fmaxf(second, fminf(best, c));
                     best = fmaxf(best, c);
                 }
@@ -148,7 +155,7 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
             warp_argmax(bv, bi);
             __syncwarp();
             if (bi != 0x7fffffff)
-                for (int j = lane; j < per; j += 32) cand[bi * per + j] = choice(bi * per + j);
+                for (int j = lane; j < per; j += 32) cand[bi * per + j] = choice[bi * per + j];
             __syncwarp();
         }
     }
@@ -186,9 +193,13 @@ VOB_EXPORT int vob_moe_route(const void* x, int code, long ld_x, const float* w_
     const RouteRule rule{sigmoid, group_best, renorm, correction, eps, out_scale};
     if (width <= 0 || E <= 0 || top <= 0 || top > E) return VOB_ERR_BAD_ARG;
     if (n_groups > 1 && (E % n_groups != 0 || keep <= 0 || keep > n_groups || top > keep * (E / n_groups))) return VOB_ERR_BAD_ARG;
-    const size_t smem = (size_t)4 * 2 * E * sizeof(float);
+    const size_t smem = (size_t)4 * 3 * E * sizeof(float);
     if (smem > 48 * 1024) return VOB_ERR_UNSUPPORTED;
-    VOB_DISPATCH_ELEM(code, return vob_launch(moe_route_kernel<ElemT>, dim3((T + 3) / 4), dim3(128), smem, stream, (const ElemT*)x, ld_x, w_router,
+    if (T <= VOB_MOE_ROUTE_FEW) {
+        VOB_DISPATCH_ELEM(code, return vob_launch(moe_route_kernel<ElemT, 1, 16>, dim3(T), dim3(512), smem / 4, stream, (const ElemT*)x, ld_x,
+                                                  w_router, positions, T, width, E, top, n_groups, keep, rule, idx_out, w_out));
+    }
+    VOB_DISPATCH_ELEM(code, return vob_launch(moe_route_kernel<ElemT, 4, 4>, dim3((T + 3) / 4), dim3(128), smem, stream, (const ElemT*)x, ld_x, w_router,
                                               positions, T, width, E, top, n_groups, keep, rule, idx_out, w_out));
     return 0;
 }
