@@ -318,14 +318,14 @@ def test_window_with_kept_first_tokens_linear_bias_and_values_that_are_keys(dtyp
     wide = torch.full((T, H * DV + 8), float("nan"), dtype=dtype, device=DEV)
     kernels.flex_attention(qd, wide[:, 8:], kc, vals, tables.to(DEV), row_seq, positions, H, G, D, DV, scale, window, None, gd, 1.0, **kw)
     outs["general"] = wide[:, 8:]
-    if dtype == torch.bfloat16 and kernels.attn_prefill_mma_any_supported(H, G, D, DV, page) and (shared or not keep):
+    if dtype == torch.bfloat16 and kernels.attn_prefill_mma_any_supported(H, G, D, DV, page) and (shared or not (keep or bias)):
         wide2 = torch.full((T, H * DV + 8), float("nan"), dtype=dtype, device=DEV)
         kernels.attn_prefill_mma_any(qd, wide2[:, 8:], kc, vals, tables.to(DEV), _ints([0, lens[0], T]), _ints(ctxs), 2, max(lens), H, G, D, DV,
                                      scale, window, None, gd, 1.0, **kw)
         assert bool(torch.isnan(wide2[:, :8]).all())
         outs["portions"] = wide2[:, 8:]
     decode = {}
-    if dtype == torch.bfloat16 and D == DV and D in (64, 128) and (cap or shared or keep or bias):
+    if dtype == torch.bfloat16 and D == DV and D in (64, 128) and (shared or not (keep or bias)):
         last = torch.tensor([lens[0] - 1, T - 1], device=DEV)
         for splits in (1, 2, 3, 8, 20):
             o2 = torch.full((2, H * DV), float("nan"), dtype=dtype, device=DEV)

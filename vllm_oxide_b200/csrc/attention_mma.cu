@@ -78,13 +78,12 @@ __device__ __forceinline__ float tail_val(const AttnTail& t, long long row, int 
 // What may lie between q . k and the softmax (all optional; the kernels built with SHAPED take it):
 //   chunk > 0    a query reads only the keys of its own block of `chunk` positions, blocks counted from position 0;
 //   a cap        score <- softcap * tanh(score / softcap);
-//   r1, r2       [H] each: r1 * ln(1 + r2 * (i - j)) is taken off the score of key j for the query at i; with `linear`
-//                r1 * (i - j) is (r2 is not used);
-//   keep         (with a window) the keys of the first `keep` positions are seen by every query behind them (the portion kernel
-//                takes it where the values are the keys, KV1);
+//   r1, r2       [H] each: r1 * ln(1 + r2 * (i - j)) is taken off the score of key j for the query at i.
+// Only in the kernels built with KV1 (the values are the cached keys), which take no logarithmic bias and no pooled keys:
+//   linear       r1 * (i - j) is taken off (r2 is not used);
+//   keep         (with a window) the keys of the first `keep` positions are seen by every query behind them;
 //   kscale       one float per cached token (laid out [pages][page_size]): q . k is multiplied by key j's before anything else
-//                (kernels built with KV1, where the cache holds the keys as projected: those are the values, and their norm,
-//                one number per token and a weight per feature, is this number and a factor on q).
+//                (the keys' norm, one number per token and a weight per feature, is this number and a factor on q).
 // Scores leave in base-2 units (times log2 e), and the launchers' scale_log2 is not used by a shaped kernel. The struct
 // is a kernel parameter: what the inner loop reads of it comes from the constant bank and holds no register.
 //   pooled keys  (with a window, portion kernel only) beside the window's tokens a query at position p sees the first
@@ -233,8 +232,9 @@ __device__ __forceinline__ void pv_tile(float (&o)[HD / 8][4], const uint32_t (&
 // starting at key index key0; this thread's rows are r and r+8 with limits [lo, pos]. With MASK
 // false the caller knows that every key of the tile is visible to every row of the warp. SHAPED: the scores
 // first become what `rs` makes of them (cap, distance bias), in base-2 units, and `scale_log2` is not used.
-// KSC: q . k is first multiplied by key j's number, ksc[j - key0].
-template <int NB, int HDN, bool MASK, bool SHAPED = false, bool KSC = false, bool KEPT = KSC>
+// KV1: q . k is first multiplied by key j's number, ksc[j - key0]; the distance bias is the linear one (a slope of 0: none), and
+// keys of kept first tokens are seen too.
+template <int NB, int HDN, bool MASK, bool SHAPED = false, bool KV1 = false>
 __device__ __forceinline__ void softmax_step(float (&s)[NB][4], uint32_t (&pa)[NB / 2][4], float (&o)[HDN][4],
                                              float (&m)[2], float (&l)[2], int key0, const int (&lo)[2],
                                              const int (&pos)[2], float scale_log2, const ScoreShape* sh = nullptr,
@@ -250,15 +250,15 @@ __device__ __forceinline__ void softmax_step(float (&s)[NB][4], uint32_t (&pa)[N
             if (SHAPED) {
                 int j = key0 + nb * 8 + (lane & 3) * 2 + (i & 1);
                 float t = s[nb][i] * sh->pre;
-                if (KSC) t *= ksc[nb * 8 + (lane & 3) * 2 + (i & 1)];
+                if (KV1) t *= ksc[nb * 8 + (lane & 3) * 2 + (i & 1)];
                 if (sh->cap_log2 > 0.f) t = sh->cap_log2 * fast_tanh(t);
-                if (sh->linear) t = fmaf(-rs->r1[h], (float)(pos[h] - j), t);
+                if (KV1) t = fmaf(-rs->r1[h], (float)(pos[h] - j), t);
                 else if (sh->r1) t -= rs->r1[h] * __log2f(fmaf(rs->r2[h], (float)max(pos[h] - j, 0), 1.f));
                 s[nb][i] = t;
             }
             if (MASK) {
                 int j = key0 + nb * 8 + (lane & 3) * 2 + (i & 1);
-                if (!((j >= lo[h] || (KEPT && j < sh->keep)) && j <= pos[h])) s[nb][i] = -INFINITY;
+                if (!((j >= lo[h] || (KV1 && j < sh->keep)) && j <= pos[h])) s[nb][i] = -INFINITY;
             }
             mx[h] = fmaxf(mx[h], s[nb][i]);
         }
@@ -458,9 +458,9 @@ __device__ __forceinline__ void load_rows_padded(__nv_bfloat16* dst, const __nv_
     }
 }
 
-// Blocks per SM the compiler is told to aim at, where its own choice of registers would spill a few bytes.
+// Blocks per SM the compiler is told to aim at, where its own choice of registers would spill a few bytes (0: its own choice).
 constexpr int any_min_blocks(int hd, int hdv, bool shaped, bool kv1) {
-    return shaped && !kv1 && hd == 96 && hdv == 64 ? 2 : kv1 && hd == 32 ? 3 : 1;
+    return shaped && !kv1 && hd == 32 && hdv == 32 ? 3 : 0;
 }
 template <int HD, int HDV, bool SHAPED, bool KV1>
 __global__ void __launch_bounds__(NTHREADS, any_min_blocks(HD, HDV, SHAPED, KV1))
@@ -513,26 +513,29 @@ attn_prefill_mma_any_kernel(const __nv_bfloat16* __restrict__ q, long long q_str
     // pooled entries the block's last row sees (the most of all its rows)
     const int hi_pool = pool > 0 && window > 0 && hi - window >= pool ? (hi - window) / pool : 0;
 
-    // the last pooled entry a query at position p sees (-1: none); it grows with p
-    auto last_pooled = [&](int p) { return p >= 0 && p + 1 - window >= pool ? (p + 1 - window) / pool - 1 : -1; };
-    int pos[2], lo[2], hd[2];
+    int pos[2], lo[2], hd[2], pos_p[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         int rr = tile_row0 + warp * 16 + (lane >> 2) + h * 8;
         pos[h] = rr < total_rows ? ctx + rr / G : -1;
         hd[h] = rr < total_rows ? kvh * G + rr % G : -1;
         lo[h] = first_key(pos[h], window, chunk);
+        // the last pooled entry this row sees (-1: none)
+        pos_p[h] = pool > 0 && pos[h] >= 0 && pos[h] + 1 - window >= pool ? (pos[h] + 1 - window) / pool - 1 : -1;
     }
     RowShape rs;
     if (SHAPED) rs = row_shape(shape, hd[0], hd[1]);
     int warp_last_pos = max(pos[0], pos[1]), warp_first_pos = min(pos[0], pos[1]), warp_max_lo = max(lo[0], lo[1]);
     int warp_min_lo = 0;                             // blocks of positions: the first key any row of the warp reads
     if (SHAPED) warp_min_lo = min(pos[0] < 0 ? 0x7fffffff : lo[0], pos[1] < 0 ? 0x7fffffff : lo[1]);
+    int warp_last_p = max(pos_p[0], pos_p[1]), warp_first_p = min(pos_p[0], pos_p[1]);
 #pragma unroll
     for (int x = 4; x < 32; x <<= 1) {
         warp_last_pos = max(warp_last_pos, __shfl_xor_sync(0xffffffffu, warp_last_pos, x));
         warp_first_pos = min(warp_first_pos, __shfl_xor_sync(0xffffffffu, warp_first_pos, x));
         warp_max_lo = max(warp_max_lo, __shfl_xor_sync(0xffffffffu, warp_max_lo, x));
+        if (SHAPED && !KV1) warp_last_p = max(warp_last_p, __shfl_xor_sync(0xffffffffu, warp_last_p, x));
+        if (SHAPED && !KV1) warp_first_p = min(warp_first_p, __shfl_xor_sync(0xffffffffu, warp_first_p, x));
         if (SHAPED) warp_min_lo = min(warp_min_lo, __shfl_xor_sync(0xffffffffu, warp_min_lo, x));
     }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
@@ -586,9 +589,9 @@ attn_prefill_mma_any_kernel(const __nv_bfloat16* __restrict__ q, long long q_str
         }
         const bool pooled = SHAPED && !KV1 && it < tp_end;
         const int t = SHAPED && it < tp_end ? it : t_begin + it - tp_end;
-        const int w_last = pooled ? last_pooled(warp_last_pos) : warp_last_pos, w_first = pooled ? last_pooled(warp_first_pos) : warp_first_pos;
+        const int w_last = pooled ? warp_last_p : warp_last_pos, w_first = pooled ? warp_first_p : warp_first_pos;
         const int w_max_lo = pooled ? 0 : warp_max_lo, w_min_lo = pooled ? 0 : warp_min_lo;
-        const int lo_r[2] = {pooled ? 0 : lo[0], pooled ? 0 : lo[1]}, pos_r[2] = {pooled ? last_pooled(pos[0]) : pos[0], pooled ? last_pooled(pos[1]) : pos[1]};
+        const int lo_r[2] = {pooled ? 0 : lo[0], pooled ? 0 : lo[1]}, pos_r[2] = {pooled ? pos_p[0] : pos[0], pooled ? pos_p[1] : pos[1]};
         // a tile behind the warp's last key needs no work, nor has one whose rows all begin to read behind this tile's last key
         // (unless it holds kept first tokens)
         if (t * BN <= w_last && (!SHAPED || (t + 1) * BN > w_min_lo || (KV1 && t * BN < keep))) {
@@ -748,11 +751,11 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
     const int hi = p + 1;
     const int lo_key = first_key(p, window, SHAPED ? shape.chunk : 0);
     const int t_first = lo_key / BN;
-    const int keep = SHAPED ? shape.keep : 0;
-    const int kt = SHAPED ? min((keep + BN - 1) / BN, t_first) : 0;      // tiles of kept first tokens in front of the window's
+    const int keep = KV1 ? shape.keep : 0;
+    const int kt = KV1 ? min((keep + BN - 1) / BN, t_first) : 0;      // tiles of kept first tokens in front of the window's
     const int n_tiles = p >= 0 ? (hi + BN - 1) / BN - t_first + kt : 0;
     // the request's tile number n (0 .. n_tiles - 1) holds the keys from BN * tile_of(n) on
-    auto tile_of = [&](int n) { return SHAPED && n < kt ? n : t_first + n - kt; };
+    auto tile_of = [&](int n) { return KV1 && n < kt ? n : t_first + n - kt; };
     if (partials) {
         splits = max(1, min(splits, n_tiles / DEC_MIN_TILES));
         const int share = max(1, (n_tiles + splits - 1) / splits);
@@ -846,7 +849,7 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, 
         float s[2][4];
         qk_tile<HD, 2>(s, qf, sK, warp * 2);                    // this warp's 16 keys of the tile
         uint32_t pa[1][4];
-        softmax_step<2, HD / 8, true, SHAPED, KV1, SHAPED>(s, pa, o, m, l, t * BN + warp * 16, lo, pos, scale_log2, &shape, &rs,
+        softmax_step<2, HD / 8, true, SHAPED, KV1>(s, pa, o, m, l, t * BN + warp * 16, lo, pos, scale_log2, &shape, &rs,
                                                    sR0 + buf * BN + warp * 16);
         pv_tile<HD, 1>(o, pa, sV, warp);
     }
@@ -1082,7 +1085,6 @@ int prefill_any(const void* q, long long q_stride, void* out, long long out_stri
     if (KV <= 0 || H % KV != 0 || page_size <= 0 || BN % page_size != 0) return VOB_ERR_UNSUPPORTED;
     if (D <= 0 || DV <= 0 || D % 8 != 0 || DV % 8 != 0 || D > 128 || DV > 128) return VOB_ERR_UNSUPPORTED;
     if (q_stride % 8 != 0 || out_stride % 2 != 0 || S > 65535 || KV > 65535) return VOB_ERR_BAD_ARG;
-    if (shape.keep > 0 && kcache != vcache) return VOB_ERR_UNSUPPORTED;
     if (SHAPED && kcache == vcache) {          // the values are the cached keys
         if (D != DV || shape.pool > 0) return VOB_ERR_BAD_ARG;
 #define VOB_KV1(HD_)                                                                                                                \
@@ -1154,15 +1156,16 @@ static int shape_args_ok(int chunk, float softcap, const float* r1, const float*
                          const void* kcache, const void* vcache) {
     if (chunk < 0 || softcap < 0.f || (r2 && !r1)) return 0;
     if (keep < 0 || (keep > 0 && (window <= 0 || chunk > 0))) return 0;
-    if (kscale && kcache != vcache) return 0;
-    return 1;
+    // the kernels whose values are the cached keys take a linear bias, kept first tokens and a number per key; the others none of them
+    if (kcache != vcache) return !(kscale || keep > 0 || (r1 && !r2));
+    return !r2;
 }
 
 // The same with scores that are shaped before the softmax: a query reads the keys of its own block of `chunk` positions
 // (0: no blocks), score <- softcap * tanh(score / softcap) (0: no cap), r1[head] * ln(1 + r2[head] * distance) is taken
-// off (r1, r2 float32 [H], or both null), or r1[head] * distance (r2 null). Any sign of `scale`. `keep`: the first so many keys are
-// seen whatever the window. kcache == vcache: the values are the cached keys, q . k is multiplied by kscale [pages][page_size]
-// (null: by nothing). `gate_heads`: the gate has one column per head.
+// off (r1, r2 float32 [H], or both null). Any sign of `scale`. kcache == vcache: the values are the cached keys; then r1[head] *
+// distance is taken off (r2 null), q . k is multiplied by kscale [pages][page_size] (null: by nothing), and the first `keep` keys are
+// seen whatever the window. `gate_heads`: the gate has one column per head.
 VOB_EXPORT int vob_attn_prefill_shaped(const void* q, long long q_stride, void* out, long long out_stride, const void* kcache,
                                        const void* vcache, const int* block_tables, int max_pages, const int* seq_starts,
                                        const int* context_lens, int S, int max_new, int H, int KV, int D, int DV, int page_size,

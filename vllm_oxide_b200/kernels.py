@@ -1799,10 +1799,10 @@ def _score_shape(op, q, num_heads, chunk, softcap, dist_bias, window=0, keep_fir
                  vcache=None, gate=None):
     """Checked arguments of what may shape a score before the softmax, or None where there is nothing: blocks of `chunk`
     positions (a query reads its own block's keys only), score <- softcap * tanh(score / softcap), and dist_bias = (r1, r2),
-    float32 [H] each: r1 * ln(1 + r2 * distance) taken off; or dist_slopes, float32 [H]: slope * distance taken off.
-    `keep_first` (with a window): the keys of the first so many positions are seen whatever the window. `vcache is kcache`: the
-    values are the cached keys; q . k is then first multiplied by key j's number in `key_scale` (float32 [pages, 1, page_size, 1],
-    or None). Returns ((chunk, softcap, r1, r2), (keep_first, key_scale))."""
+    float32 [H] each: r1 * ln(1 + r2 * distance) taken off. `vcache is kcache`: the values are the cached keys; then, instead of
+    dist_bias, dist_slopes, float32 [H]: slope * distance taken off, `keep_first` (with a window): the keys of the first so many
+    positions are seen whatever the window, and q . k is first multiplied by key j's number in `key_scale` (float32
+    [pages, 1, page_size, 1], or None). Returns ((chunk, softcap, r1, r2), (keep_first, key_scale))."""
     shared = kcache is not None and kcache is vcache
     per_head = gate is not None and gate.shape[1] == num_heads and gate.shape[1] != q.shape[1]
     if not chunk and not softcap and dist_bias is None and not keep_first and dist_slopes is None and not shared and not per_head and key_scale is None:
@@ -1813,8 +1813,10 @@ def _score_shape(op, q, num_heads, chunk, softcap, dist_bias, window=0, keep_fir
         raise ShapeError(op, "kept first tokens go with a window and without blocks of positions")
     if dist_bias is not None and dist_slopes is not None:
         raise ShapeError(op, "a bias on the logarithm of the distance or on the distance, not both")
-    if key_scale is not None and not shared:
-        raise ShapeError(op, "numbers per key go with values that are the cached keys")
+    if not shared and (key_scale is not None or keep_first or dist_slopes is not None):
+        raise ShapeError(op, "numbers per key, kept first tokens and a linear bias go with values that are the cached keys here")
+    if shared and dist_bias is not None:
+        raise ShapeError(op, "where the values are the cached keys the bias is linear in the distance")
     r1, r2 = dist_bias if dist_bias is not None else (dist_slopes, None)
     _cuda(op, q, r1, r2, key_scale)
     if key_scale is not None:
@@ -1904,8 +1906,6 @@ def attn_prefill_mma_any(q, out, kcache, vcache, block_tables, seq_starts, conte
         pool_args = (_ptr(kpool), _ptr(vpool), int(pool))
         if shape is None:
             shape = ((0, 0.0, _P(0), _P(0)), (0, _P(0)))
-    if keep_first and kcache is not vcache:
-        raise ShapeError(op, "this kernel takes kept first tokens where the values are the cached keys")
     if shape is None and not scale > 0:
         raise ShapeError(op, f"the score scale must be positive, got {scale}")
     _cuda(op, q, out, kcache, vcache, block_tables, seq_starts, context_lens)

@@ -247,13 +247,18 @@ class SoftmaxAttention(Mixer):
             return cache.tensors[0], cache.tensors[0], cache.tensors[1]
         return cache.tensors[0], cache.tensors[1], None
 
+    def shaped_kernels(self) -> bool:
+        """Whether the tensor-core kernels compute this layer's scores: kept first tokens and a linear bias where the values are the
+        keys, the logarithmic bias elsewhere."""
+        return self.dist_bias is None if self.values_are_keys else not self.keep_first and self.dist_slopes is None
+
     def padded_tile_sizes(self) -> bool:
         """Keys and values of sizes the portion kernel with padded tiles takes."""
         return self.D % 8 == 0 and self.DV % 8 == 0 and self.D <= 128 and self.DV <= 128
 
     def shaped_decode_sizes(self) -> bool:
         """Shaped scores with keys and values of one size the split-key decode kernel is built for."""
-        return not self.plain_scores() and self.D == self.DV and self.D in kernels.TENSOR_CORE_HEAD_DIMS and self.H // self.G <= 16
+        return not self.plain_scores() and self.shaped_kernels() and self.D == self.DV and self.D in kernels.TENSOR_CORE_HEAD_DIMS and self.H // self.G <= 16
 
     def kernel_modules(self, dtype, max_rows):
         if dtype == torch.float32:
@@ -304,7 +309,7 @@ class SoftmaxAttention(Mixer):
         go to the decode kernel and the portions behind them to the portion kernel. bfloat16 with keys and values of
         other sizes (multiples of 8 up to 128 each, different or not): portions and mixed steps go to the mma.sync
         portion kernel that pads its tiles, steps of single tokens to the general kernel. Scores that are shaped
-        before the softmax (blocks of positions, a cap, a distance bias, kept first tokens, a number per key) take the same two mma.sync kernels in their
+        before the softmax (blocks of positions, a cap, a distance bias, kept first tokens, a number per key; see `shaped_kernels`) take the same two mma.sync kernels in their
         shaped build: the padded portion kernel for portions and mixed steps of any of those sizes, the split-key
         decode kernel for steps of single tokens with keys and values of one size of 64 or 128. Everything else
         (float32, other sizes) goes to the general kernel."""
@@ -347,7 +352,7 @@ class SoftmaxAttention(Mixer):
             self._attend_single(q, out, ctx, cache, bt, ctx.rows, gate, out_scale)
             return
         if (self.dtype == torch.bfloat16 and self.impl != "general" and (self.scale > 0 or shaped) and not ctx.decode_only and ctx.max_new > 1
-                and (not self.keep_first or self.values_are_keys)
+                and self.shaped_kernels()
                 and kernels.attn_prefill_mma_any_supported(H, G, D, self.DV, page) and out.data_ptr() % 4 == 0 and out.stride(0) % 2 == 0):
             kernels.attn_prefill_mma_any(q, out, kc, vc, bt, ctx.seq_starts, ctx.context_lens, ctx.seqs, ctx.max_new, H, G, D, self.DV,
                                          self.scale, self.window, self.sink, gate, out_scale, key_scale=key_scale, **self.shape_args())
