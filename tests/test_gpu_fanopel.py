@@ -418,6 +418,34 @@ def test_the_mixer_whole_in_portions_and_token_by_token(dtype, H, G, D, window, 
         assert _diff(torch.cat(got), want) < (2e-5 if dtype == torch.float32 else 3e-2), cuts
 
 
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,G,D,DV,keep,slopes", [(4, 2, 64, 64, 5, True), (2, 2, 24, 40, 3, False), (2, 1, 128, 128, 0, True)])
+def test_kept_first_tokens_and_the_linear_bias_with_values_of_their_own(dtype, H, G, D, DV, keep, slopes):
+    """The same options in a mixer that has value projections and no norms (any of the kernels may take it)."""
+    from vllm_oxide_b200.parts.base import LayerCache
+    from vllm_oxide_b200.parts.flex_attention import SoftmaxAttention
+    torch.manual_seed(D)
+    width, T, page, window = 40, 70, 8, 17
+    w = {n: (torch.randn(r, width) * 0.3).bfloat16() for n, r in (("q", H * D), ("k", G * D), ("v", G * DV))}
+    wo, sl = (torch.randn(width, H * DV) * 0.2).bfloat16(), torch.rand(H) * 0.1
+    mixer = SoftmaxAttention(w["q"], w["k"], w["v"], wo, H, G, D, DV, 0.1, window=window, keep_first=keep, softcap=6.0,
+                             dist_slopes=sl if slopes else None, dtype=dtype, device=DEV)
+    x = torch.randn(T, width).to(dtype)
+    q, k, v = ((x.double() @ w[n].double().T).reshape(T, -1, z) for n, z in (("q", D), ("k", D), ("v", DV)))
+    want, _ = _attention_plain(q, k, v, 0, window, keep, 0.1, 6.0, sl.double() if slopes else None, torch.full((T, H), 50.0, dtype=torch.float64))
+    want = want @ wo.double().T
+    for cuts in ([T], [9, 2, 40] + [1] * 19):
+        tables, caches = _paged([T], page, [(G, D), (G, DV)], [dtype, dtype])
+        cache = LayerCache(tensors=tuple(caches), group=0, write=True)
+        got, at = [], 0
+        for n in cuts:
+            pos = list(range(at, at + n))
+            ctx = _step_ctx(pos, [0, n], tables, [int(tables[0, p // page]) * page + p % page for p in pos], dtype, n, n == 1, at)
+            got.append(mixer.forward(x[at:at + n].to(DEV), ctx, cache, None).clone())
+            at += n
+        assert _diff(torch.cat(got), want) < (2e-5 if dtype == torch.float32 else 3e-2), cuts
+
+
 # ------------------------------------------------------------------------------------ experts
 @pytest.mark.parametrize("E,top,groups,keep,shift", [(6, 2, 3, 2, -0.7), (12, 4, 2, 1, 0.0), (5, 3, 0, 0, -0.5), (4, 1, 4, 3, -2.0), (7, 4, 1, 1, 0.4),
                                                       (40, 8, 8, 3, -1.0), (64, 6, 16, 5, -1.8)])
