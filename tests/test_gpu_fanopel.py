@@ -447,7 +447,7 @@ def test_kept_first_tokens_and_the_linear_bias_with_values_of_their_own(dtype, H
 
 
 # ------------------------------------------------------------------------------------ experts
-@pytest.mark.parametrize("E,top,groups,keep,shift", [(6, 2, 3, 2, -0.7), (12, 4, 2, 1, 0.0), (5, 3, 0, 0, -0.5), (4, 1, 4, 3, -2.0), (7, 4, 1, 1, 0.4),
+@pytest.mark.parametrize("E,top,groups,keep,shift", [(6, 2, 3, 2, -0.7), (10, 3, 2, 1, 0.0), (5, 3, 0, 0, -0.5), (4, 1, 4, 3, -2.0), (7, 4, 1, 1, 0.4),
                                                       (40, 8, 8, 3, -1.0), (64, 6, 16, 5, -1.8)])
 def test_election_by_sigmoid_scores_with_a_correction(E, top, groups, keep, shift):
     """Choice scores on both sides of zero; groups scored by their two best experts; the weights are made of the scores without

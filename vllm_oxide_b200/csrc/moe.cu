@@ -83,7 +83,7 @@ moe_route_kernel(const T* __restrict__ x, long ld_x, const float* __restrict__ w
 #pragma unroll
         for (int k = 0; k < TPB; ++k) acc[k] = 0.f;
         if (by4) {
-#pragma unroll (TPB == 1 ? 8 : 2)
+#pragma unroll (TPB == 1 ? 4 : 2)
             for (int i = lane * 4; i < width; i += 128) {
                 const float4 w4 = *reinterpret_cast<const float4*>(wr + i);
 #pragma unroll
