@@ -21,6 +21,8 @@ from ..csrc.build import runtime_module
 from ..errors import CapacityError, ConfigError
 from ..parts.base import CacheSpec, LayerCache, ModelSpec
 
+EMBEDDING_STATE = "embedding"       # under this key `CachePools.state` holds the embedding's state, beside the calls' by number
+
 
 class CachePools:
     def __init__(self, spec: ModelSpec, page_size: int, max_seqs: int, dtype: torch.dtype, device: str,
@@ -90,7 +92,7 @@ class CachePools:
                                for t in cs.paged_tensors())
         # fixed-size per-request state, one tensor per call whose mixer asks for it
         # (a mixer that names several tensors gets a tuple of them)
-        self.state: Dict[int, object] = {}
+        self.state: Dict[object, object] = {}
         for idx, call in enumerate(spec.schedule):
             # a block may keep state of its own beside its mixer's (the last inputs of a convolution in front of its
             # sub-layers, say): it then answers for both
@@ -101,6 +103,10 @@ class CachePools:
             made = tuple(torch.zeros((max_seqs,) + tuple(x.shape), dtype=x.dtype, device=device)
                          for x in (ss if isinstance(ss, (tuple, list)) else (ss,)))
             self.state[idx] = made if isinstance(ss, (tuple, list)) else made[0]
+        # an embedding may keep state too (the token before the next one, say)
+        es = spec.embedding.state_spec() if hasattr(spec.embedding, "state_spec") else None
+        if es is not None:
+            self.state[EMBEDDING_STATE] = torch.zeros((max_seqs,) + tuple(es.shape), dtype=es.dtype, device=device)
 
     @property
     def num_groups(self) -> int:

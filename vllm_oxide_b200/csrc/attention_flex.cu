@@ -33,7 +33,7 @@ VOB_PDL_SWITCH(attention_flex)
 // the head's features are asked for before the token's position and slot are known (padding rows are rows of
 // the projection like any other).
 //   q, k:  the first `rot` features of a head are rotated, feature i with i + rot / 2, by
-//          float(pos) * inv_freq[i]; then (unit_rms) the head is divided by sqrt(mean(x^2) + eps) and, where a
+//          float(pos) * inv_freq[i], cosine and sine both times `mag`; then (unit_rms) the head is divided by sqrt(mean(x^2) + eps) and, where a
 //          weight of D entries is given (`q_norm_w`, `k_norm_w`, shared by the heads), multiplied by it;
 //          q is also multiplied by 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1) (temp_every > 0).
 //          With `q_pre_w` [H * D] / `k_pre_w` [G * D]: BEFORE the rotation the whole projection (all heads at once) is
@@ -47,7 +47,7 @@ VOB_PDL_SWITCH(attention_flex)
 template <typename T, int NI>
 __global__ void __launch_bounds__(256, 4)
 flex_prep_kernel(const T* __restrict__ proj, long ld, int q_off, int k_off, int v_off, const int* __restrict__ positions,
-                 const int* __restrict__ slots, const float* __restrict__ inv_freq, int rot, int unit_rms, float eps,
+                 const int* __restrict__ slots, const float* __restrict__ inv_freq, int rot, float mag, int unit_rms, float eps,
                  float temp_coef, int temp_every, const float* __restrict__ q_norm_w, const float* __restrict__ k_norm_w,
                  const float* __restrict__ q_pre_w, const float* __restrict__ k_pre_w, const float* __restrict__ vmix, T* __restrict__ v_first, int v_mode, T* __restrict__ q_out, long ld_q, T* __restrict__ kcache, T* __restrict__ vcache, int H, int G, int D, int DV,
                  int page_size) {
@@ -100,7 +100,7 @@ flex_prep_kernel(const T* __restrict__ proj, long ld, int q_off, int k_off, int 
                 const int f = lane + 32 * i;
                 if (f < rot) {
                     const float ang = fpos * inv_freq[f < half ? f : f - half];
-                    const float sn = sinf(ang), cs = cosf(ang);
+                    const float sn = sinf(ang) * mag, cs = cosf(ang) * mag;
                     x[i] = f < half ? x[i] * cs - y[i] * sn : x[i] * cs + y[i] * sn;
                 }
                 ss = fmaf(x[i], x[i], ss);
@@ -139,7 +139,7 @@ flex_prep_kernel(const T* __restrict__ proj, long ld, int q_off, int k_off, int 
 }
 
 VOB_EXPORT int vob_flex_prep(const void* proj, int code, long ld, int q_off, int k_off, int v_off, const int* positions,
-                             const int* slots, const float* inv_freq, int rot, int unit_rms, float eps, float temp_coef,
+                             const int* slots, const float* inv_freq, int rot, float mag, int unit_rms, float eps, float temp_coef,
                              int temp_every, const float* q_norm_w, const float* k_norm_w, const float* q_pre_w, const float* k_pre_w,
                              const float* vmix, void* v_first,
                              int v_mode, void* q_out, long ld_q, void* kcache,
@@ -153,7 +153,7 @@ VOB_EXPORT int vob_flex_prep(const void* proj, int code, long ld, int q_off, int
     if ((H + 2 * G + 7) / 8 > 65535) return VOB_ERR_UNSUPPORTED;
 #define VOB_PREP(NI_)                                                                                                                  \
     VOB_DISPATCH_ELEM(code, return vob_launch(flex_prep_kernel<ElemT, NI_>, dim3(T, (H + 2 * G + 7) / 8), dim3(256), 0, stream,              \
-                                              (const ElemT*)proj, ld, q_off, k_off, v_off, positions, slots, inv_freq, rot, unit_rms, eps,  \
+                                              (const ElemT*)proj, ld, q_off, k_off, v_off, positions, slots, inv_freq, rot, mag, unit_rms, eps,  \
                                               temp_coef, temp_every, q_norm_w, k_norm_w, q_pre_w, k_pre_w, vmix, (ElemT*)v_first, v_mode, (ElemT*)q_out,  \
                                               ld_q, (ElemT*)kcache,                                                                      \
                                               (ElemT*)vcache, H, G, D, DV, page_size))

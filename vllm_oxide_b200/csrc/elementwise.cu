@@ -8,6 +8,29 @@
 #include "common.cuh"
 VOB_PDL_SWITCH(elementwise)
 
+// Four neighbouring elements (aligned to their 8 or 16 bytes) as floats, and back.
+template <typename T> __device__ __forceinline__ void ld4_f(const T* p, float (&v)[4]);
+template <> __device__ __forceinline__ void ld4_f<float>(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+template <> __device__ __forceinline__ void ld4_f<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[4]) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&a.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&a.y);
+    v[0] = __bfloat162float(lo.x); v[1] = __bfloat162float(lo.y); v[2] = __bfloat162float(hi.x); v[3] = __bfloat162float(hi.y);
+}
+template <typename T> __device__ __forceinline__ void st4_f(T* p, const float (&v)[4]);
+template <> __device__ __forceinline__ void st4_f<float>(float* p, const float (&v)[4]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+template <> __device__ __forceinline__ void st4_f<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[4]) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    uint2 a;
+    a.x = *reinterpret_cast<const unsigned*>(&lo);
+    a.y = *reinterpret_cast<const unsigned*>(&hi);
+    *reinterpret_cast<uint2*>(p) = a;
+}
+
 // ---------------------------------------------------------------------------------------------
 // Embedding gather: out[t, :] = table[tokens[t], :] * scale (+ pos_table[positions[t], :])   (float32 out; scale 1 leaves
 // the row as it is). The learned position vector is optional; a row with a negative position (padding) gets none.
@@ -46,6 +69,110 @@ VOB_EXPORT int vob_embed(const void* table, int table_code, const int* tokens, f
     if (!pos_table) max_pos = 0x7fffffff;
     VOB_DISPATCH_ELEM(table_code, return vob_launch(embed_kernel<ElemT>, dim3(T), dim3(256), 0, stream, (const ElemT*)table, tokens, out, h, vocab, err_flag, scale,
                                                     (const ElemT*)pos_table, positions, max_pos));
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// Embedding gather with a vector for every pair of neighbouring tokens:
+//   out[t, :] = table[c, :] * scale (+ pos_table[position, :]) + pair_table[row, :]
+//   row = (p * mul_prev + c * mul_cur) mod buckets, c the row's token and p the one before it in its request (64-bit
+//   arithmetic); a request's first token (position 0) takes row number `buckets`, the table's last.
+// p is the row in front, or, for the first row a request brings to a step, the last token of the request's previous step,
+// which `last_token` holds per state slot. The block of that first row reads the old entry and then writes the new one (the
+// last token the request brings): no other block touches it, so one launch does both. Padding rows (negative position) get
+// no pair vector and touch no state. `keep` (optional) receives a copy of the row: what a later layer adds once more.
+// Launch: one block per token; four features a thread where the width and the addresses allow. Bound: memory.
+// A token outside [0, vocab) or a position beyond the table writes zeros and raises *err_flag.
+// ---------------------------------------------------------------------------------------------
+struct PairTable {
+    const void* table;          // null: no vector per pair
+    const int* positions;
+    const int* row_seq;
+    const int* seq_starts;
+    const int* state_slots;
+    int* last_token;
+    long long mul_prev, mul_cur, buckets;
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+embed_pairs_kernel(const T* __restrict__ table, const int* __restrict__ tokens, float* __restrict__ out, int h, int vocab,
+                   int* err_flag, float scale, const T* __restrict__ pos_table, int max_pos, PairTable pairs, float* __restrict__ keep) {
+    pdl_launch_dependents();
+    pdl_wait(1);
+    const int t = blockIdx.x;
+    const int tok = tokens[t];
+    const int pos = pairs.positions ? pairs.positions[t] : -1;
+    bool ok = tok >= 0 && tok < vocab && (!pos_table || pos < max_pos);
+    const T* prow = nullptr;
+    if (pairs.table && pos >= 0) {
+        const int s = pairs.row_seq[t], first = pairs.seq_starts[s];
+        long long row = pairs.buckets;
+        int prev = 0;
+        if (t > first) {
+            prev = tokens[t - 1];
+        } else {
+            const int slot = pairs.state_slots[s];
+            prev = pairs.last_token[slot];
+            __syncthreads();                                    // everyone has read the old entry
+            if (threadIdx.x == 0) pairs.last_token[slot] = tokens[pairs.seq_starts[s + 1] - 1];
+        }
+        if (pos > 0) row = ((long long)prev * pairs.mul_prev + (long long)tok * pairs.mul_cur) % pairs.buckets;
+        if (row < 0) ok = false;
+        else prow = (const T*)pairs.table + (size_t)row * h;
+    }
+    if (!ok && threadIdx.x == 0 && err_flag) atomicExch(err_flag, 1);
+    const T* src = table + (size_t)(ok ? tok : 0) * h;
+    const T* psrc = (ok && pos_table && pos >= 0) ? pos_table + (size_t)pos * h : nullptr;
+    float* dst = out + (size_t)t * h;
+    float* kd = keep ? keep + (size_t)t * h : nullptr;
+    for (int i = threadIdx.x * V; i < h; i += blockDim.x * V) {
+        float v[V];
+        if constexpr (V == 4) {
+            ld4_f<T>(src + i, v);
+        } else {
+            v[0] = ld_f(src + i);
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] = ok ? v[k] * scale : 0.f;
+        for (int part = 0; part < 2; ++part) {
+            const T* add = part == 0 ? psrc : prow;
+            if (!add || !ok) continue;
+            float a[V];
+            if constexpr (V == 4) {
+                ld4_f<T>(add + i, a);
+            } else {
+                a[0] = ld_f(add + i);
+            }
+#pragma unroll
+            for (int k = 0; k < V; ++k) v[k] += a[k];
+        }
+        if constexpr (V == 4) {
+            st4_f<float>(dst + i, v);
+            if (kd) st4_f<float>(kd + i, v);
+        } else {
+            dst[i] = v[0];
+            if (kd) kd[i] = v[0];
+        }
+    }
+}
+
+VOB_EXPORT int vob_embed_pairs(const void* table, int table_code, const int* tokens, float* out, int T, int h, int vocab, int* err_flag,
+                               float scale, const void* pos_table, const int* positions, int max_pos, const void* pair_table,
+                               long long buckets, long long mul_prev, long long mul_cur, const int* row_seq, const int* seq_starts,
+                               const int* state_slots, int* last_token, float* keep, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (h <= 0 || vocab <= 0) return VOB_ERR_BAD_ARG;
+    if (pos_table && (!positions || max_pos <= 0)) return VOB_ERR_BAD_ARG;
+    if (pair_table && (!positions || !row_seq || !seq_starts || !state_slots || !last_token || buckets <= 0)) return VOB_ERR_BAD_ARG;
+    PairTable pt{pair_table, positions, row_seq, seq_starts, state_slots, last_token, mul_prev, mul_cur, buckets};
+    const bool four = h % 4 == 0 && (((uintptr_t)table | (uintptr_t)out | (uintptr_t)pos_table | (uintptr_t)pair_table | (uintptr_t)keep) & 15) == 0;
+    if (four) {
+        VOB_DISPATCH_ELEM(table_code, return vob_launch(embed_pairs_kernel<ElemT, 4>, dim3(T), dim3(256), 0, stream, (const ElemT*)table, tokens, out,
+                                                        h, vocab, err_flag, scale, (const ElemT*)pos_table, max_pos, pt, keep));
+    }
+    VOB_DISPATCH_ELEM(table_code, return vob_launch(embed_pairs_kernel<ElemT, 1>, dim3(T), dim3(256), 0, stream, (const ElemT*)table, tokens, out,
+                                                    h, vocab, err_flag, scale, (const ElemT*)pos_table, max_pos, pt, keep));
     return 0;
 }
 
@@ -95,6 +222,8 @@ VOB_EXPORT int vob_embed_fold(const void* table, int table_code, const int* toke
 // ---------------------------------------------------------------------------------------------
 // Residual add + RMSNorm:
 //   x = resid[src] (+ delta[src] (* dscale, per feature));  if no row list: resid[src] = x  (the residual sum, float32)
+//   delta may come in `parts` tensors `part_stride` elements apart (the results of sub-layers that ran side by side): all are
+//   added; `extra` (a float32 row per token) and `vec` (one float32 vector) are added behind them (AddMore)
 //   out[r] = w * (x * 1/sqrt(mean(x^2) + eps))
 // Reference ops: add (crates/engine/src/backend/cpu/mod.rs:351-358) followed by rmsnorm
 // (:182-197); the weight multiplies last, as there. With a row list (`rows`, R entries) only
@@ -104,10 +233,17 @@ VOB_EXPORT int vob_embed_fold(const void* table, int table_code, const int* toke
 // once. Sum of squares: per-thread strided partial sums, then a fixed tree, so a row's value is
 // the same in every batch. Bound: memory.
 // ---------------------------------------------------------------------------------------------
-template <typename TD, typename TO>
+struct AddMore {
+    int parts;                  // delta tensors (0: none)
+    long long part_stride;      // elements from one to the next
+    const float* extra;         // [T, h], or null
+    const float* vec;           // [h], or null
+};
+
+template <typename TD, typename TO, bool MORE>
 __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const TD* __restrict__ delta,
                                    const float* __restrict__ weight, const int* __restrict__ rows,
-                                   TO* __restrict__ out, int h, float eps, const float* __restrict__ dscale) {
+                                   TO* __restrict__ out, int h, float eps, const float* __restrict__ dscale, AddMore more) {
     pdl_launch_dependents();
     pdl_wait(2);
     extern __shared__ float row[];
@@ -119,7 +255,14 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const TD* __restri
     float ss = 0.f;
     for (int i = threadIdx.x; i < h; i += blockDim.x) {
         float v = x[i];
-        if (d) {
+        if (MORE) {
+            float sum = 0.f;
+            for (int p = 0; p < more.parts; ++p) sum += ld_f(d + p * more.part_stride + i);
+            v += sum;
+            if (more.extra) v += more.extra[(size_t)src * h + i];
+            if (more.vec) v += more.vec[i];
+            if (!rows) x[i] = v;
+        } else if (d) {
             v += dscale ? ld_f(d + i) * dscale[i] : ld_f(d + i);
             if (!rows) x[i] = v;
         }
@@ -172,12 +315,13 @@ template <> struct Store4<__nv_bfloat16> {
     }
 };
 
-template <typename TD, typename TO, int NV>
+template <typename TD, typename TO, int NV, bool MORE>
 __global__ void __launch_bounds__(256)
 add_rmsnorm_vec_kernel(float* __restrict__ resid, const TD* __restrict__ delta, const float* __restrict__ weight,
-                       const int* __restrict__ rows, TO* __restrict__ out, int h, float eps, const float* __restrict__ dscale) {
+                       const int* __restrict__ rows, TO* __restrict__ out, int h, float eps, const float* __restrict__ dscale, AddMore more) {
     pdl_launch_dependents();
     pdl_wait(2);
+    constexpr bool LATE = MORE && NV == 8;      // the weight is read last: held from the start it would not fit the registers
     __shared__ float red[32];
     int r = blockIdx.x;
     int src = rows ? rows[r] : r;
@@ -191,11 +335,25 @@ add_rmsnorm_vec_kernel(float* __restrict__ resid, const TD* __restrict__ delta, 
         if (i < nvec) {
             v[k] = *reinterpret_cast<const float4*>(x + 4 * i);
             dv[k] = d ? Load4<TD>::ld(d + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
-            if (d && dscale) {
+            if (!MORE && d && dscale) {
                 const float4 sc = *reinterpret_cast<const float4*>(dscale + 4 * i);
                 dv[k].x *= sc.x; dv[k].y *= sc.y; dv[k].z *= sc.z; dv[k].w *= sc.w;
             }
-            w[k] = *reinterpret_cast<const float4*>(weight + 4 * i);
+            if (MORE) {
+                for (int p = 1; p < more.parts; ++p) {
+                    const float4 a = Load4<TD>::ld(d + p * more.part_stride + 4 * i);
+                    dv[k].x += a.x; dv[k].y += a.y; dv[k].z += a.z; dv[k].w += a.w;
+                }
+                if (more.extra) {
+                    const float4 a = *reinterpret_cast<const float4*>(more.extra + (size_t)src * h + 4 * i);
+                    dv[k].x += a.x; dv[k].y += a.y; dv[k].z += a.z; dv[k].w += a.w;
+                }
+                if (more.vec) {
+                    const float4 a = *reinterpret_cast<const float4*>(more.vec + 4 * i);
+                    dv[k].x += a.x; dv[k].y += a.y; dv[k].z += a.z; dv[k].w += a.w;
+                }
+            }
+            if (!LATE) w[k] = *reinterpret_cast<const float4*>(weight + 4 * i);
         }
     }
     float ss = 0.f;
@@ -204,7 +362,7 @@ add_rmsnorm_vec_kernel(float* __restrict__ resid, const TD* __restrict__ delta, 
         int i = threadIdx.x + k * 256;
         if (i < nvec) {
             v[k].x += dv[k].x; v[k].y += dv[k].y; v[k].z += dv[k].z; v[k].w += dv[k].w;
-            if (d && !rows) *reinterpret_cast<float4*>(x + 4 * i) = v[k];
+            if ((MORE || d) && !rows) *reinterpret_cast<float4*>(x + 4 * i) = v[k];
             ss += v[k].x * v[k].x; ss += v[k].y * v[k].y; ss += v[k].z * v[k].z; ss += v[k].w * v[k].w;
         }
     }
@@ -223,40 +381,48 @@ add_rmsnorm_vec_kernel(float* __restrict__ resid, const TD* __restrict__ delta, 
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         int i = threadIdx.x + k * 256;
+        if (LATE && i < nvec) w[k] = *reinterpret_cast<const float4*>(weight + 4 * i);
         if (i < nvec)
             Store4<TO>::st(o + 4 * i, make_float4(w[k].x * (v[k].x * inv), w[k].y * (v[k].y * inv),
                                                   w[k].z * (v[k].z * inv), w[k].w * (v[k].w * inv)));
     }
 }
 
-template <typename TD, typename TO>
+template <typename TD, typename TO, bool MORE>
 static int launch_add_rmsnorm(float* resid, const void* delta, const float* weight, const int* rows, void* out, int R,
-                              int h, float eps, const float* dscale, cudaStream_t stream) {
+                              int h, float eps, const float* dscale, AddMore more, cudaStream_t stream) {
     bool aligned = (h % 4 == 0) && (((uintptr_t)resid | (uintptr_t)delta | (uintptr_t)weight | (uintptr_t)out | (uintptr_t)dscale) % 16 == 0);
+    if (MORE) aligned = aligned && (((uintptr_t)more.extra | (uintptr_t)more.vec) % 16 == 0) && more.part_stride % 8 == 0;
     int nv = (h / 4 + 255) / 256;
     if (aligned && nv <= 8) {
-#define VEC(NV) return vob_launch(add_rmsnorm_vec_kernel<TD, TO, NV>, dim3(R), dim3(256), 0, stream, resid, (const TD*)delta, weight, rows, (TO*)out, h, eps, dscale)
+#define VEC(NV) return vob_launch(add_rmsnorm_vec_kernel<TD, TO, NV, MORE>, dim3(R), dim3(256), 0, stream, resid, (const TD*)delta, weight, rows, (TO*)out, h, eps, dscale, more)
         if (nv <= 1) VEC(1); else if (nv <= 2) VEC(2); else if (nv <= 4) VEC(4); else VEC(8);
 #undef VEC
     }
     size_t smem = (size_t)h * sizeof(float);
     if (smem > 48 * 1024) return VOB_ERR_UNSUPPORTED;
-    return vob_launch(add_rmsnorm_kernel<TD, TO>, dim3(R), dim3(256), smem, stream, resid, (const TD*)delta, weight, rows, (TO*)out, h, eps, dscale);
+    return vob_launch(add_rmsnorm_kernel<TD, TO, MORE>, dim3(R), dim3(256), smem, stream, resid, (const TD*)delta, weight, rows, (TO*)out, h, eps, dscale, more);
 }
 
 VOB_EXPORT int vob_add_rmsnorm(float* resid, const void* delta, int delta_code, const float* weight,
                                const int* rows, void* out, int out_code, int R, int h, float eps,
-                               const float* dscale, cudaStream_t stream) {
+                               const float* dscale, int parts, long long part_stride, const float* extra, const float* vec,
+                               cudaStream_t stream) {
     if (R <= 0) return 0;
     if (h <= 0) return VOB_ERR_BAD_ARG;
-    if (!delta) delta_code = VOB_F32;
+    if (!delta) { delta_code = VOB_F32; parts = 0; }
+    const bool more = parts > 1 || extra || vec;
+    if (more && dscale) return VOB_ERR_BAD_ARG;
+    const AddMore am{parts, part_stride, extra, vec};
+#define VOB_ARN(TD, TO)                                                                                                    return more ? launch_add_rmsnorm<TD, TO, true>(resid, delta, weight, rows, out, R, h, eps, dscale, am, stream)                      : launch_add_rmsnorm<TD, TO, false>(resid, delta, weight, rows, out, R, h, eps, dscale, am, stream)
     if (out_code == VOB_F32) {
-        if (delta_code == VOB_F32) return launch_add_rmsnorm<float, float>(resid, delta, weight, rows, out, R, h, eps, dscale, stream);
-        if (delta_code == VOB_BF16) return launch_add_rmsnorm<__nv_bfloat16, float>(resid, delta, weight, rows, out, R, h, eps, dscale, stream);
+        if (delta_code == VOB_F32) VOB_ARN(float, float);
+        if (delta_code == VOB_BF16) VOB_ARN(__nv_bfloat16, float);
     } else if (out_code == VOB_BF16) {
-        if (delta_code == VOB_F32) return launch_add_rmsnorm<float, __nv_bfloat16>(resid, delta, weight, rows, out, R, h, eps, dscale, stream);
-        if (delta_code == VOB_BF16) return launch_add_rmsnorm<__nv_bfloat16, __nv_bfloat16>(resid, delta, weight, rows, out, R, h, eps, dscale, stream);
+        if (delta_code == VOB_F32) VOB_ARN(float, __nv_bfloat16);
+        if (delta_code == VOB_BF16) VOB_ARN(__nv_bfloat16, __nv_bfloat16);
     }
+#undef VOB_ARN
     return VOB_ERR_BAD_ARG;
 }
 
@@ -677,27 +843,6 @@ __device__ __forceinline__ float block_sum_256(float v, float* red) {
     return t;
 }
 
-template <typename T> __device__ __forceinline__ void ld4_f(const T* p, float (&v)[4]);
-template <> __device__ __forceinline__ void ld4_f<float>(const float* p, float (&v)[4]) {
-    const float4 a = *reinterpret_cast<const float4*>(p);
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-}
-template <> __device__ __forceinline__ void ld4_f<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[4]) {
-    const uint2 a = *reinterpret_cast<const uint2*>(p);
-    const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&a.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&a.y);
-    v[0] = __bfloat162float(lo.x); v[1] = __bfloat162float(lo.y); v[2] = __bfloat162float(hi.x); v[3] = __bfloat162float(hi.y);
-}
-template <typename T> __device__ __forceinline__ void st4_f(T* p, const float (&v)[4]);
-template <> __device__ __forceinline__ void st4_f<float>(float* p, const float (&v)[4]) {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-}
-template <> __device__ __forceinline__ void st4_f<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[4]) {
-    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
-    uint2 a;
-    a.x = *reinterpret_cast<const unsigned*>(&lo);
-    a.y = *reinterpret_cast<const unsigned*>(&hi);
-    *reinterpret_cast<uint2*>(p) = a;
-}
 
 // What the kernel can do on its way behind resid[r] += LN(delta[r]) (a kernel parameter: what is not asked for costs nothing):
 //   * the stream as a weighted sum over depth (see depth_average_kernel, the same sums in the same order): the new row is
@@ -1055,31 +1200,38 @@ VOB_EXPORT int vob_cast_rows(const float* in, void* out, int out_code, long long
 __device__ __forceinline__ float xielu_f(float z, float ap, float an) {
     return z > 0.f ? fmaf(ap * z, z, 0.5f * z) : fmaf(an, expm1f(z) - z, 0.5f * z);
 }
+enum ActKind { ACT_XIELU = 0, ACT_RELU2 = 1 };      // ACT_RELU2: max(z, 0)^2, no parameters
+template <int KIND>
+__device__ __forceinline__ float act_f(float z, float ap, float an) {
+    if (KIND == ACT_XIELU) return xielu_f(z, ap, an);
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+}
 
-template <typename T>
+template <typename T, int KIND>
 __global__ void __launch_bounds__(256)
-act_kernel(const T* __restrict__ in, long long in_stride, T* __restrict__ out, int I, int act, const float* __restrict__ params) {
+act_kernel(const T* __restrict__ in, long long in_stride, T* __restrict__ out, int I, const float* __restrict__ params) {
     pdl_launch_dependents();
     pdl_wait(7);
     const int t = blockIdx.x;
     const int j = blockIdx.y * 256 + threadIdx.x;
     if (j >= I) return;
-    const float ap = params[0], an = params[1];
+    const float ap = KIND == ACT_XIELU ? params[0] : 0.f, an = KIND == ACT_XIELU ? params[1] : 0.f;
     const float z = ld_f(in + (size_t)t * in_stride + j);
-    st_f(out + (size_t)t * I + j, xielu_f(z, ap, an));
+    st_f(out + (size_t)t * I + j, act_f<KIND>(z, ap, an));
 }
 
 // Rows whose length and addresses allow 16-byte accesses: a thread takes 16 bytes of a row a turn.
-template <typename T>
+template <typename T, int KIND>
 __global__ void __launch_bounds__(256)
-act_vec_kernel(const T* __restrict__ in, long long in_stride, T* __restrict__ out, int I, int act, const float* __restrict__ params) {
+act_vec_kernel(const T* __restrict__ in, long long in_stride, T* __restrict__ out, int I, const float* __restrict__ params) {
     pdl_launch_dependents();
     pdl_wait(7);
     constexpr int PER = 16 / sizeof(T);
     const int t = blockIdx.x;
     const int j = (blockIdx.y * 256 + threadIdx.x) * PER;
     if (j >= I) return;
-    const float ap = params[0], an = params[1];
+    const float ap = KIND == ACT_XIELU ? params[0] : 0.f, an = KIND == ACT_XIELU ? params[1] : 0.f;
     const T* src = in + (size_t)t * in_stride + j;
     T* dst = out + (size_t)t * I + j;
 #pragma unroll
@@ -1087,7 +1239,7 @@ act_vec_kernel(const T* __restrict__ in, long long in_stride, T* __restrict__ ou
         float v[4];
         ld4_f<T>(src + k, v);
 #pragma unroll
-        for (int m = 0; m < 4; ++m) v[m] = xielu_f(v[m], ap, an);
+        for (int m = 0; m < 4; ++m) v[m] = act_f<KIND>(v[m], ap, an);
         st4_f<T>(dst + k, v);
     }
 }
@@ -1095,17 +1247,18 @@ act_vec_kernel(const T* __restrict__ in, long long in_stride, T* __restrict__ ou
 VOB_EXPORT int vob_act(const void* in, long long in_stride, void* out, int code, int T, int I, int act, const float* params,
                        cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (I <= 0 || act != 0 || !params) return VOB_ERR_BAD_ARG;
+    if (I <= 0 || (act != ACT_XIELU && act != ACT_RELU2) || (act == ACT_XIELU && !params)) return VOB_ERR_BAD_ARG;
     const int per = code == VOB_BF16 ? 8 : 4;
-    if (I % per == 0 && in_stride % per == 0 && ((((uintptr_t)in) | ((uintptr_t)out)) & 15) == 0) {
-        const int by = (I / per + 255) / 256;
-        if (by > 65535) return VOB_ERR_UNSUPPORTED;
-        VOB_DISPATCH_ELEM(code, return vob_launch(act_vec_kernel<ElemT>, dim3(T, by), dim3(256), 0, stream, (const ElemT*)in, in_stride,
-                                                  (ElemT*)out, I, act, params));
-        return 0;
-    }
-    if ((I + 255) / 256 > 65535) return VOB_ERR_UNSUPPORTED;
-    VOB_DISPATCH_ELEM(code, return vob_launch(act_kernel<ElemT>, dim3(T, (I + 255) / 256), dim3(256), 0, stream, (const ElemT*)in, in_stride,
-                                              (ElemT*)out, I, act, params));
+    const bool vec = I % per == 0 && in_stride % per == 0 && ((((uintptr_t)in) | ((uintptr_t)out)) & 15) == 0;
+    const int by = vec ? (I / per + 255) / 256 : (I + 255) / 256;
+    if (by > 65535) return VOB_ERR_UNSUPPORTED;
+#define VOB_ACT(KERNEL, KIND)                                                                                                    \
+    VOB_DISPATCH_ELEM(code, return vob_launch(KERNEL<ElemT, KIND>, dim3(T, by), dim3(256), 0, stream, (const ElemT*)in, in_stride, \
+                                              (ElemT*)out, I, params))
+    if (vec && act == ACT_XIELU) VOB_ACT(act_vec_kernel, ACT_XIELU);
+    if (vec) VOB_ACT(act_vec_kernel, ACT_RELU2);
+    if (act == ACT_XIELU) VOB_ACT(act_kernel, ACT_XIELU);
+    VOB_ACT(act_kernel, ACT_RELU2);
+#undef VOB_ACT
     return 0;
 }

@@ -6,9 +6,11 @@
 // and the caller applies W_uv to out_lat. Causal: row i of a request sees the keys 0 .. position(i)
 // of that request, all read from the pages (the step's own tokens were written first).
 //
-// vob_latent_prep: per token, c = weight * x / sqrt(mean(x^2) + eps) of the first L columns of the
-// down projection and the rotary positions on its last R columns, both written to the token's cache
-// slot; the rotated query part of every head to a float32 buffer.
+// vob_latent_prep: per token, any of three jobs: c = weight * x / sqrt(mean(x^2) + eps) of the first L
+// columns of the down projection and the rotary positions on its last R columns, both written to the
+// token's cache slot; the rotated query part of every head to a float32 buffer; the same norm on a
+// latent the queries are made from (designs whose queries go through one), to a buffer of its own.
+// vob_latent_gate: the heads' values times sigmoid(gate), element by element, put side by side per token.
 // vob_latent_attend: scores, softmax weights and the weighted sum in float32, keys in page order
 // from the first, in tiles staged in shared memory; one warp per head, a block takes up to 8 heads
 // of one row, so a key tile is read once for all of them. The order of every sum depends only on the row's
@@ -19,48 +21,67 @@
 #include <math.h>
 VOB_PDL_SWITCH(latent_attention)
 
-// proj [T, ld]: the query of head h at columns q_off + h * (D + R) (D plain features, then R to be
-// rotated); the down projection at columns down_off .. + L + R. lat [pages, 1, page, L], kr [pages,
-// 1, page, R] in the cache's type TC. q_rot float32 [T, H, R]. Rows with position < 0 write nothing
-// (their q_rot is zero); a slot < 0 writes no cache.
+// q [T, ld_q]: the query of head h at columns h * (D + R) (D plain features, then R to be rotated); down [T, ld]: the down
+// projection's L + R columns. lat [pages, 1, page, L], kr [pages, 1, page, R] in the cache's type TC. q_rot float32 [T, H, R].
+// Cosine and sine are both multiplied by `mag`. Rows with position < 0 write nothing (their q_rot is zero); a slot < 0 writes
+// no cache. `q` null: no queries here; `slots` null: no cache write; `low` [T, ld_low] (Q columns) null: no query latent, else
+// low_out [T, Q] = low_w * low / sqrt(mean(low^2) + eps), every row.
 // Launch: one block of 128 threads per token.
 template <typename T, typename TC>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(const T* __restrict__ proj, long ld, int q_off, int H, int D, int R, int down_off, int L,
+latent_prep_kernel(const T* __restrict__ q, long ld_q, int H, int D, int R, const T* __restrict__ down_p, long ld, int L,
                    const float* __restrict__ norm_w, float eps, const int* __restrict__ positions, const int* __restrict__ slots,
-                   const float* __restrict__ inv_freq, TC* __restrict__ lat, TC* __restrict__ kr, float* __restrict__ q_rot) {
+                   const float* __restrict__ inv_freq, float mag, TC* __restrict__ lat, TC* __restrict__ kr, float* __restrict__ q_rot,
+                   const T* __restrict__ low, long ld_low, int Q, const float* __restrict__ low_w, T* __restrict__ low_out) {
     pdl_launch_dependents();
     pdl_wait(45);
-    __shared__ float red[4];
+    __shared__ float red[4], red_low[4];
     const int t = blockIdx.x, tid = threadIdx.x;
     const int pos = positions[t];
-    const T* row = proj + (size_t)t * ld;
     const int half = R >> 1;
-    float* qo = q_rot + (size_t)t * H * R;
-    for (int e = tid; e < H * R; e += blockDim.x) {
-        float v = 0.f;
-        if (pos >= 0) {
-            const int h = e / R, f = e - h * R;
-            const int i = f < half ? f : f - half;
-            const float ang = (float)pos * inv_freq[i];
-            const float cs = cosf(ang), sn = sinf(ang);
-            const T* qh = row + q_off + (size_t)h * (D + R) + D;
-            const float a = ld_f(qh + i), b = ld_f(qh + i + half);
-            v = f < half ? a * cs - b * sn : b * cs + a * sn;
+    if (q) {
+        const T* row = q + (size_t)t * ld_q;
+        float* qo = q_rot + (size_t)t * H * R;
+        for (int e = tid; e < H * R; e += blockDim.x) {
+            float v = 0.f;
+            if (pos >= 0) {
+                const int h = e / R, f = e - h * R;
+                const int i = f < half ? f : f - half;
+                const float ang = (float)pos * inv_freq[i];
+                const float cs = cosf(ang) * mag, sn = sinf(ang) * mag;
+                const T* qh = row + (size_t)h * (D + R) + D;
+                const float a = ld_f(qh + i), b = ld_f(qh + i + half);
+                v = f < half ? a * cs - b * sn : b * cs + a * sn;
+            }
+            qo[e] = v;
         }
-        qo[e] = v;
     }
     const int slot = slots ? slots[t] : -1;
-    if (pos < 0 || slot < 0) return;
-    const T* down = row + down_off;
-    float ss = 0.f;
-    for (int i = tid; i < L; i += blockDim.x) {
-        const float x = ld_f(down + i);
-        ss = fmaf(x, x, ss);
-    }
+    const bool write = pos >= 0 && slot >= 0;
+    if (!write && !low) return;
+    const T* down = down_p + (size_t)t * ld;
+    const T* lrow = low + (size_t)t * ld_low;
+    float ss = 0.f, sl = 0.f;
+    if (write)
+        for (int i = tid; i < L; i += blockDim.x) {
+            const float x = ld_f(down + i);
+            ss = fmaf(x, x, ss);
+        }
+    if (low)
+        for (int i = tid; i < Q; i += blockDim.x) {
+            const float x = ld_f(lrow + i);
+            sl = fmaf(x, x, sl);
+        }
     ss = warp_sum(ss);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
+    sl = warp_sum(sl);
+    if ((tid & 31) == 0) { red[tid >> 5] = ss; red_low[tid >> 5] = sl; }
     __syncthreads();
+    if (low) {
+        const float inv = 1.0f / sqrtf(((red_low[0] + red_low[1]) + (red_low[2] + red_low[3])) / (float)Q + eps);
+        T* o = low_out + (size_t)t * Q;
+        for (int i = tid; i < Q; i += blockDim.x) st_f(o + i, low_w[i] * (ld_f(lrow + i) * inv));
+    }
+    if (!write) return;
     const float inv = 1.0f / sqrtf(((red[0] + red[1]) + (red[2] + red[3])) / (float)L + eps);
     TC* lo = lat + (size_t)slot * L;
     for (int i = tid; i < L; i += blockDim.x) st_f(lo + i, norm_w[i] * (ld_f(down + i) * inv));
@@ -68,20 +89,70 @@ latent_prep_kernel(const T* __restrict__ proj, long ld, int q_off, int H, int D,
     for (int f = tid; f < R; f += blockDim.x) {
         const int i = f < half ? f : f - half;
         const float ang = (float)pos * inv_freq[i];
-        const float cs = cosf(ang), sn = sinf(ang);
+        const float cs = cosf(ang) * mag, sn = sinf(ang) * mag;
         const float a = ld_f(down + L + i), b = ld_f(down + L + i + half);
         st_f(ko + f, f < half ? a * cs - b * sn : b * cs + a * sn);
     }
 }
 
-VOB_EXPORT int vob_latent_prep(const void* proj, int code, long ld, int q_off, int H, int D, int R, int down_off, int L,
-                               const float* norm_w, float eps, const int* positions, const int* slots, const float* inv_freq,
-                               void* lat, void* kr, int cache_code, float* q_rot, int T, cudaStream_t stream) {
+VOB_EXPORT int vob_latent_prep(const void* q, int code, long ld_q, int H, int D, int R, const void* down, long ld, int L,
+                               const float* norm_w, float eps, const int* positions, const int* slots, const float* inv_freq, float mag,
+                               void* lat, void* kr, int cache_code, float* q_rot, const void* low, long ld_low, int Q, const float* low_w,
+                               void* low_out, int T, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0 || D < 0 || R <= 0 || (R & 1) || L <= 0 || code != cache_code) return VOB_ERR_BAD_ARG;
-    VOB_DISPATCH_ELEM(code, return vob_launch(latent_prep_kernel<ElemT, ElemT>, dim3(T), dim3(128), 0, stream, (const ElemT*)proj, ld,
-                                              q_off, H, D, R, down_off, L, norm_w, eps, positions, slots, inv_freq, (ElemT*)lat,
-                                              (ElemT*)kr, q_rot));
+    if ((q && !q_rot) || (slots && (!down || !lat || !kr)) || (low && (Q <= 0 || !low_w || !low_out))) return VOB_ERR_BAD_ARG;
+    VOB_DISPATCH_ELEM(code, return vob_launch(latent_prep_kernel<ElemT, ElemT>, dim3(T), dim3(128), 0, stream, (const ElemT*)q, ld_q, H, D, R,
+                                              (const ElemT*)down, ld, L, norm_w, eps, positions, slots, inv_freq, mag, (ElemT*)lat,
+                                              (ElemT*)kr, q_rot, (const ElemT*)low, ld_low, Q, low_w, (ElemT*)low_out));
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// out[t, h * V + i] = vals(t, h, i) * sigmoid(gate[t, h * V + i]); vals at t * v_ts + h * v_hs + i, gate rows ld_gate apart, out
+// [T, H * V] (may be vals itself where that has its layout). PER elements (16 bytes) a thread where sizes and addresses allow.
+// Launch: grid (rows, ceil(H V / (256 PER))). Bound: memory.
+// ---------------------------------------------------------------------------------------------
+template <typename T, int PER>
+__global__ void __launch_bounds__(256)
+latent_gate_kernel(const T* vals, long v_ts, long v_hs, const T* __restrict__ gate, long ld_gate, int H, int V, T* out) {
+    pdl_launch_dependents();
+    pdl_wait(49);
+    const int t = blockIdx.x, e = (blockIdx.y * 256 + threadIdx.x) * PER;
+    if (e >= H * V) return;
+    const int h = e / V, i = e - h * V;
+    const T* src = vals + (size_t)t * v_ts + (size_t)h * v_hs + i;
+    const T* g = gate + (size_t)t * ld_gate + e;
+    T* o = out + (size_t)t * H * V + e;
+    if constexpr (PER == 1) {
+        st_f(o, ld_f(src) / (1.0f + expf(-ld_f(g))));
+    } else {
+        T a[PER], b[PER];
+        *reinterpret_cast<uint4*>(a) = *reinterpret_cast<const uint4*>(src);
+        *reinterpret_cast<uint4*>(b) = *reinterpret_cast<const uint4*>(g);
+#pragma unroll
+        for (int k = 0; k < PER; ++k) st_f(a + k, ld_f(a + k) / (1.0f + expf(-ld_f(b + k))));
+        *reinterpret_cast<uint4*>(o) = *reinterpret_cast<const uint4*>(a);
+    }
+}
+
+VOB_EXPORT int vob_latent_gate(const void* vals, int code, long v_ts, long v_hs, const void* gate, long ld_gate, int T, int H, int V,
+                               void* out, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    if (H <= 0 || V <= 0 || (H * V + 255) / 256 > 65535) return VOB_ERR_BAD_ARG;
+    const int per = code == VOB_BF16 ? 8 : 4;
+    if (V % per == 0 && v_ts % per == 0 && v_hs % per == 0 && ld_gate % per == 0 && (((uintptr_t)vals | (uintptr_t)gate | (uintptr_t)out) & 15) == 0) {
+        const dim3 grid(T, (H * V / per + 255) / 256);
+        if (code == VOB_BF16)
+            return vob_launch(latent_gate_kernel<__nv_bfloat16, 8>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)vals, v_ts, v_hs,
+                              (const __nv_bfloat16*)gate, ld_gate, H, V, (__nv_bfloat16*)out);
+        if (code == VOB_F32)
+            return vob_launch(latent_gate_kernel<float, 4>, grid, dim3(256), 0, stream, (const float*)vals, v_ts, v_hs, (const float*)gate,
+                              ld_gate, H, V, (float*)out);
+        return VOB_ERR_BAD_ARG;
+    }
+    VOB_DISPATCH_ELEM(code, return vob_launch(latent_gate_kernel<ElemT, 1>, dim3(T, (H * V + 255) / 256), dim3(256), 0, stream, (const ElemT*)vals, v_ts,
+                                              v_hs, (const ElemT*)gate, ld_gate, H, V, (ElemT*)out));
     return 0;
 }
 

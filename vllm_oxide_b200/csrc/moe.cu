@@ -9,9 +9,10 @@
 //                    made of s; a run scores as the sum of its two best experts.
 //   vob_moe_align    the (token, choice) pairs put in order of their expert, every expert's run padded to whole tiles
 //                    of VOB_MOE_BM rows, with the expert of every tile.
-//   vob_moe_gate_up  per tile: h = act(W_gate[e] x) * (W_up[e] x) for the tile's pairs (x gathered by token).
+//   vob_moe_gate_up  per tile: h = act(W_gate[e] x) * (W_up[e] x) for the tile's pairs (x gathered by token). With pair weights
+//                    the experts read weight * x: both sums are multiplied by the pair's weight (float32) ahead of the gate.
 //   vob_moe_up       per tile: h = act(W_up[e] x), experts without a gate.
-//   vob_moe_down     per tile: y[pair] = weight[pair] * (W_down[e] h[pair]), float32.
+//   vob_moe_down     per tile: y[pair] = weight[pair] * (W_down[e] h[pair]), float32 (no weights given: 1).
 //   vob_moe_combine  out[token] = sum over the token's choices, in the order they were chosen, of y.
 //
 // A pair's arithmetic never depends on which other pairs share its tile or where in its expert's run it lies: every
@@ -289,7 +290,8 @@ template <> __device__ __forceinline__ float moe_rounded<__nv_bfloat16>(float v)
 template <typename T>
 __global__ void __launch_bounds__(256, 2)
 moe_gate_up_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ w_gu, const int* __restrict__ sorted,
-                   const int* __restrict__ tile_expert, int top, int width, int ff, T* __restrict__ h_out, int act, float limit) {
+                   const int* __restrict__ tile_expert, int top, int width, int ff, T* __restrict__ h_out, int act, float limit,
+                   const float* __restrict__ pair_w) {
     pdl_launch_dependents();
     pdl_wait(73);
     const int tile = blockIdx.x;
@@ -331,11 +333,12 @@ moe_gate_up_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ w_g
     for (int i = 0; i < 2; ++i) {
         const int p = pair_of[ty + 16 * i];
         if (p < 0) continue;
+        const float wgt = pair_w ? pair_w[p] : 1.f;
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
             const int c = col0 + tx + 16 * j;
             // the two products are rounded to the activations' type before the gate, as separate products would be
-            if (c < ff) st_f(h_out + (size_t)p * ff + c, moe_gate(moe_rounded<T>(g[i][j]), moe_rounded<T>(u[i][j]), act, limit));
+            if (c < ff) st_f(h_out + (size_t)p * ff + c, moe_gate(moe_rounded<T>(wgt * g[i][j]), moe_rounded<T>(wgt * u[i][j]), act, limit));
         }
     }
 }
@@ -395,7 +398,7 @@ moe_single_kernel(const T* __restrict__ a, long ld_a, int a_div, const T* __rest
     for (int i = 0; i < 2; ++i) {
         const int p = pair_of[ty + 16 * i];
         if (p < 0) continue;
-        const float wgt = UP ? 1.f : pair_w[p];
+        const float wgt = UP || !pair_w ? 1.f : pair_w[p];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int c = col0 + tx + 16 * j;
@@ -441,7 +444,7 @@ __device__ __forceinline__ void moe_stage_rows(__nv_bfloat16 (*dst)[VOB_MOE_LDS]
 __global__ void __launch_bounds__(128)
 moe_gate_up_tc_kernel(const __nv_bfloat16* __restrict__ x, long ld_x, const __nv_bfloat16* __restrict__ w_gu,
                       const int* __restrict__ sorted, const int* __restrict__ tile_expert, int top, int width, int ff,
-                      __nv_bfloat16* __restrict__ h_out, int act, float limit) {
+                      __nv_bfloat16* __restrict__ h_out, int act, float limit, const float* __restrict__ pair_w) {
     pdl_launch_dependents();
     pdl_wait(75);
     const int tile = blockIdx.x;
@@ -499,8 +502,9 @@ moe_gate_up_tc_kernel(const __nv_bfloat16* __restrict__ x, long ld_x, const __nv
             const int r = el >> 4, c = el & 15;
             const int p = pair_of[16 * i + r], col = col0 + warp * 16 + c;
             if (p >= 0 && col < ff) {
-                const float gr = __bfloat162float(__float2bfloat16_rn(Cs[warp][0][el]));
-                const float ur = __bfloat162float(__float2bfloat16_rn(Cs[warp][1][el]));
+                const float wgt = pair_w ? pair_w[p] : 1.f;
+                const float gr = __bfloat162float(__float2bfloat16_rn(wgt * Cs[warp][0][el]));
+                const float ur = __bfloat162float(__float2bfloat16_rn(wgt * Cs[warp][1][el]));
                 h_out[(size_t)p * ff + col] = __float2bfloat16_rn(moe_gate(gr, ur, act, limit));
             }
         }
@@ -563,7 +567,7 @@ moe_single_tc_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, 
             const int p = pair_of[16 * i + r], col = col0 + warp * 16 + c;
             if (p >= 0 && col < N) {
                 if (UP) reinterpret_cast<__nv_bfloat16*>(out)[(size_t)p * N + col] = __float2bfloat16_rn(moe_act(Cs[warp][el], act));
-                else reinterpret_cast<float*>(out)[(size_t)p * N + col] = pair_w[p] * Cs[warp][el];
+                else reinterpret_cast<float*>(out)[(size_t)p * N + col] = pair_w ? pair_w[p] * Cs[warp][el] : Cs[warp][el];
             }
         }
         __syncwarp();
@@ -697,15 +701,16 @@ moe_pipe_kernel(const __nv_bfloat16* __restrict__ a, long ld_a, int a_div, const
                 if (TWO && cb < N) ho[cb] = __float2bfloat16_rn(moe_act(Cs[256 + el], act));
             } else if (KIND == MOE_DOWN) {
                 float* y = reinterpret_cast<float*>(out);
-                const float wgt = pair_w[p];
+                const float wgt = pair_w ? pair_w[p] : 1.f;
                 const int ca = col0 + wc * 16 + c, cb = ca + 64;
                 if (ca < N) y[(size_t)p * N + ca] = wgt * Cs[el];
                 if (TWO && cb < N) y[(size_t)p * N + cb] = wgt * Cs[256 + el];
             } else {
                 const int col = col0 + wc * 16 + c;
                 if (col < N) {
-                    const float gr = __bfloat162float(__float2bfloat16_rn(Cs[el]));
-                    const float ur = __bfloat162float(__float2bfloat16_rn(Cs[256 + el]));
+                    const float wgt = pair_w ? pair_w[p] : 1.f;
+                    const float gr = __bfloat162float(__float2bfloat16_rn(wgt * Cs[el]));
+                    const float ur = __bfloat162float(__float2bfloat16_rn(wgt * Cs[256 + el]));
                     reinterpret_cast<__nv_bfloat16*>(out)[(size_t)p * N + col] = __float2bfloat16_rn(moe_gate(gr, ur, act, limit));
                 }
             }
@@ -735,7 +740,7 @@ static inline bool moe_rows_by16(const void* p, long ld, int K) { return K % 8 =
 // grid covers them all and tiles behind the last one in use leave at once.
 VOB_EXPORT int vob_moe_gate_up(const void* x, int code, long ld_x, const void* w_gu, const int* sorted, const int* tile_expert,
                                int max_tiles, int tile_rows, int top, int width, int ff, void* h_out, int tensor_cores, int act, float limit,
-                               cudaStream_t stream) {
+                               const float* pair_w, cudaStream_t stream) {
     if (max_tiles <= 0) return 0;
     if (top <= 0 || width <= 0 || ff <= 0 || (act != 0 && act != 1)) return VOB_ERR_BAD_ARG;
     if (tile_rows != VOB_MOE_BM && !(tile_rows == 128 && tensor_cores)) return VOB_ERR_BAD_ARG;
@@ -745,16 +750,16 @@ VOB_EXPORT int vob_moe_gate_up(const void* x, int code, long ld_x, const void* w
         const dim3 grid(max_tiles, (ff + 63) / 64);
         const __nv_bfloat16 *xa = (const __nv_bfloat16*)x, *wa = (const __nv_bfloat16*)w_gu;
         if (moe_rows_by16(x, ld_x, width) && moe_rows_by16(w_gu, width, width)) {
-            if (tile_rows == 128) return moe_pipe_launch<128, 3, MOE_GATE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act, limit);
-            return moe_pipe_launch<32, 4, MOE_GATE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, nullptr, width, ff, h_out, act, limit);
+            if (tile_rows == 128) return moe_pipe_launch<128, 3, MOE_GATE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, pair_w, width, ff, h_out, act, limit);
+            return moe_pipe_launch<32, 4, MOE_GATE_UP>(grid, stream, xa, ld_x, top, wa, sorted, tile_expert, pair_w, width, ff, h_out, act, limit);
         }
         if (tile_rows != VOB_MOE_BM) return VOB_ERR_UNSUPPORTED;
         return vob_launch(moe_gate_up_tc_kernel, grid, dim3(128), 0, stream, xa, ld_x, wa, sorted, tile_expert, top, width, ff,
-                          (__nv_bfloat16*)h_out, act, limit);
+                          (__nv_bfloat16*)h_out, act, limit, pair_w);
     }
     if ((ff + 31) / 32 > 65535) return VOB_ERR_UNSUPPORTED;
     VOB_DISPATCH_ELEM(code, return vob_launch(moe_gate_up_kernel<ElemT>, dim3(max_tiles, (ff + 31) / 32), dim3(256), 0, stream, (const ElemT*)x,
-                                              ld_x, (const ElemT*)w_gu, sorted, tile_expert, top, width, ff, (ElemT*)h_out, act, limit));
+                                              ld_x, (const ElemT*)w_gu, sorted, tile_expert, top, width, ff, (ElemT*)h_out, act, limit, pair_w));
     return 0;
 }
 

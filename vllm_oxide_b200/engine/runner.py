@@ -22,7 +22,7 @@ from typing import List, Optional
 import torch
 
 from .. import kernels
-from ..cache.pools import CachePools
+from ..cache.pools import EMBEDDING_STATE, CachePools
 from ..config import EngineConfig, architecture_for, read_config_json
 from ..csrc.build import runtime_module
 from ..errors import CapacityError, KernelError, ShapeError
@@ -192,13 +192,13 @@ class ModelRunner:
         """Peak bytes of the workspace over all steps of at most `rows` tokens, to the byte, read
         off the scopes of `_forward` and `_head` (the reference's arena formula,
         crates/engine/src/model.rs:68-90, for this arrangement; its test that the high-water mark
-        of a largest step equals the formula, :400-419, holds here too): the float32 residual,
-        two buffers for block outputs still to be added, and the larger of the largest block and
+        of a largest step equals the formula, :400-419, holds here too): the step buffers, the float32 residual,
+        two sets of buffers for block outputs still to be added, and the larger of the largest block and
         the head's chunk (logits and the normed rows)."""
         es = 2 if self.dtype == torch.bfloat16 else 4
         h, V = self.spec.hidden_size, self.spec.vocab_size
         resid = aligned(rows * h * 4 * self.spec.residual_streams)
-        pending = 2 * aligned(rows * h * es)
+        pending = 2 * aligned(self.spec.pending_parts * rows * h * es)
         block = max((b.workspace_bytes(rows, h, es) for b in self.spec.blocks), default=0)
         n = min(self.logit_chunk, rows)
         head = aligned(n * V * 4) + self.spec.final_norm.workspace_bytes(n, es)
@@ -206,7 +206,7 @@ class ModelRunner:
         embed = getattr(self.spec.embedding, "scratch_bytes", lambda r: 0)(rows)
         shared = sum(aligned(rows * cols * (es if dt is None else torch.empty((), dtype=dt).element_size()))
                      for cols, dt in self.spec.step_buffers.values())
-        total = resid + max(embed, shared + pending + max(block, head))
+        total = shared + resid + max(embed, pending + max(block, head))
         if self._can_fold(1):
             # steps of few rows run in folded form (FoldedState): residual, the next norm's input, the
             # partial sums of squares, and the blocks' folded scratch or the head
@@ -307,7 +307,7 @@ class ModelRunner:
             from ..parts.rmsnorm import RMSNorm
             self._foldable = bool(
                 self.dtype == torch.bfloat16 and self.engine.fold_norms and spec.schedule
-                and hasattr(spec.embedding, "forward_folded") and getattr(spec.embedding, "scale", 1.0) == 1.0
+                and hasattr(spec.embedding, "forward_folded") and getattr(spec.embedding, "can_fold", lambda: True)()
                 and isinstance(spec.final_norm, RMSNorm)
                 and all(getattr(spec.blocks[c.layer], "can_fold", lambda: False)() and c.cache is not None and c.write
                         for c in spec.schedule))
@@ -330,10 +330,13 @@ class ModelRunner:
         if self._can_fold(ctx.rows):
             self._folded = self._forward_folded(ctx)
             return self._folded.resid, None
-        resid = spec.embedding.forward(ctx)
         for name, (cols, dt) in spec.step_buffers.items():
             ctx.shared[name] = ctx.alloc((ctx.rows, cols), dt)
+        estate = self.pools.state.get(EMBEDDING_STATE)
+        resid = spec.embedding.forward(ctx) if estate is None else spec.embedding.forward(ctx, estate)
         es_shape = (ctx.rows, spec.hidden_size)
+        if spec.pending_parts > 1:
+            es_shape = (spec.pending_parts,) + es_shape
         pend = [ctx.alloc(es_shape), ctx.alloc(es_shape)]
         pending = None
         self._pending_scale = None              # the per-feature scale the pending output is added with (a block may have one)
@@ -341,10 +344,10 @@ class ModelRunner:
             block = spec.blocks[call.layer]
             cache = self.pools.layer_cache(call.cache, call.write)
             state = self.pools.state.get(i)
-            if self._pending_scale is not None:
-                pending = block.forward(resid, pending, ctx, cache, state, pend[i & 1], pending_scale=self._pending_scale)
-            else:
-                pending = block.forward(resid, pending, ctx, cache, state, pend[i & 1])
+            kw = {} if self._pending_scale is None else {"pending_scale": self._pending_scale}
+            if call.entry is not None:
+                kw["entry"] = call.entry
+            pending = block.forward(resid, pending, ctx, cache, state, pend[i & 1], **kw)
             self._pending_scale = getattr(block, "pending_scale", None)
             if self.after_block is not None:
                 self.after_block(i, resid, pending)

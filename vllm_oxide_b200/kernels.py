@@ -225,21 +225,69 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, err_flag
              pos_table.shape[0] if pos_table is not None else 0, _stream()), op)
 
 
+@_timed
+def embed_pairs(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, positions: torch.Tensor, err_flag: Optional[torch.Tensor] = None,
+                scale: float = 1.0, pos_table: Optional[torch.Tensor] = None, pairs=None, keep: Optional[torch.Tensor] = None) -> None:
+    """`embed` with two more things in the same pass. `pairs` = (pair_table, mul_prev, mul_cur, row_seq, seq_starts, state_slots,
+    last_token): row (previous token * mul_prev + token * mul_cur) mod (rows - 1) of pair_table is added, its last row for a
+    request's first token; the token before the first row a request brings is last_token[state slot] (int32), which is then set to the
+    last token the request brings; padding rows (negative position) get nothing and touch nothing. `keep` float32 [T, h]: a copy of out."""
+    op = "embed_pairs"
+    T = out.shape[0]
+    _cuda(op, table, tokens, out, positions, err_flag, pos_table, keep)
+    if table.dim() != 2 or not table.is_contiguous():
+        raise ShapeError(op, f"table must be contiguous [vocab, h], got {list(table.shape)}")
+    h = table.shape[1]
+    _int32_vec(tokens, T, op, "tokens")
+    _int32_vec(positions, T, op, "positions")
+    for name, t in (("out", out), ("keep", keep)):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (T, h) or not t.is_contiguous()):
+            raise ShapeError(op, f"{name} must be contiguous float32 [{T}, {h}], got {t.dtype} {list(t.shape)}")
+    for name, t in (("pos_table", pos_table), ("pair_table", pairs[0] if pairs is not None else None)):
+        if t is not None and (t.dim() != 2 or t.shape[1] != h or t.dtype != table.dtype or not t.is_contiguous()):
+            raise ShapeError(op, f"{name} must be contiguous {table.dtype} [rows, {h}], got {t.dtype} {list(t.shape)}")
+    pt = row_seq = seq_starts = slots = last = None
+    mul_prev = mul_cur = 0
+    if pairs is not None:
+        pt, mul_prev, mul_cur, row_seq, seq_starts, slots, last = pairs
+        _cuda(op, pt, row_seq, seq_starts, slots, last)
+        _int32_vec(row_seq, T, op, "row_seq")
+        if pt.shape[0] < 2:
+            raise ShapeError(op, "pair_table needs a row for first tokens and one more")
+        for name, t in (("seq_starts", seq_starts), ("state_slots", slots), ("last_token", last)):
+            if t.dtype != torch.int32 or not t.is_contiguous():
+                raise ShapeError(op, f"{name} must be contiguous int32, got {t.dtype}")
+        if not 0 <= int(mul_prev) < 2 ** 31 or not 0 <= int(mul_cur) < 2 ** 31:
+            raise ShapeError(op, f"the factors {mul_prev} and {mul_cur} must lie in 0 .. 2^31 - 1")
+    f = _fn("elementwise", "vob_embed_pairs", [_P, _I, _P, _P, _I, _I, _I, _P, _F, _P, _P, _I, _P, _L, _L, _L, _P, _P, _P, _P, _P, _P])
+    _check(f(_ptr(table), _code(table, op), _ptr(tokens), _ptr(out), T, h, table.shape[0], _ptr(err_flag), float(scale), _ptr(pos_table),
+             _ptr(positions), pos_table.shape[0] if pos_table is not None else 0, _ptr(pt), pt.shape[0] - 1 if pt is not None else 0,
+             int(mul_prev), int(mul_cur), _ptr(row_seq), _ptr(seq_starts), _ptr(slots), _ptr(last), _ptr(keep), _stream()), op)
+
+
 # ------------------------------------------------------------------------------------ norm
 @_timed
 def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
-                out: torch.Tensor, rows: Optional[torch.Tensor] = None, delta_scale: Optional[torch.Tensor] = None) -> None:
+                out: torch.Tensor, rows: Optional[torch.Tensor] = None, delta_scale: Optional[torch.Tensor] = None,
+                extra: Optional[torch.Tensor] = None, vec: Optional[torch.Tensor] = None) -> None:
     """resid (+= delta, times `delta_scale` per feature if given); out = weight * (x / sqrt(mean(x^2) + eps)).
+    `delta` may be [parts, T, h]: all its parts are added. `extra` (float32 [T, h]) and `vec` (float32 [h]) are added too.
     With `rows` (int32 [R]) only those rows are normalised into out [R, h] and resid is left as it is."""
     op = "add_rmsnorm"
-    _cuda(op, resid, delta, weight, out, rows, delta_scale)
+    _cuda(op, resid, delta, weight, out, rows, delta_scale, extra, vec)
     if resid.dtype != torch.float32 or resid.dim() != 2 or not resid.is_contiguous():
         raise ShapeError(op, f"the residual must be contiguous float32 [T, h], got {resid.dtype} {list(resid.shape)}")
     T, h = resid.shape
     if weight.dtype != torch.float32 or weight.shape != (h,) or not weight.is_contiguous():
         raise ShapeError(op, f"weight must be float32 [{h}], got {weight.dtype} {list(weight.shape)}")
-    if delta is not None and (delta.shape != resid.shape or not delta.is_contiguous()):
-        raise ShapeError(op, f"delta must be contiguous {list(resid.shape)}, got {list(delta.shape)}")
+    parts = 0 if delta is None else delta.shape[0] if delta.dim() == 3 else 1
+    if delta is not None and (delta.shape[-2:] != resid.shape or delta.dim() not in (2, 3) or not delta.is_contiguous()):
+        raise ShapeError(op, f"delta must be contiguous {list(resid.shape)}, or parts of that shape, got {list(delta.shape)}")
+    if extra is not None and (extra.shape != resid.shape or extra.dtype != torch.float32 or not extra.is_contiguous()):
+        raise ShapeError(op, f"extra must be contiguous float32 {list(resid.shape)}, got {extra.dtype} {list(extra.shape)}")
+    _f32_vec(vec, h, op, "vec")
+    if delta_scale is not None and (parts > 1 or extra is not None or vec is not None):
+        raise ShapeError(op, "delta_scale goes with one delta and nothing else to add")
     R = T
     if rows is not None:
         R = rows.numel()
@@ -251,9 +299,9 @@ def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torc
     if delta_scale is not None and (delta is None or delta_scale.dtype != torch.float32 or delta_scale.shape != (h,)
                                     or not delta_scale.is_contiguous()):
         raise ShapeError(op, f"delta_scale must be float32 [{h}] and come with a delta, got {delta_scale.dtype} {list(delta_scale.shape)}")
-    f = _fn("elementwise", "vob_add_rmsnorm", [_P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _P, _P])
+    f = _fn("elementwise", "vob_add_rmsnorm", [_P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _P, _I, _L, _P, _P, _P])
     _check(f(_ptr(resid), _ptr(delta), _code(delta, op) if delta is not None else 0, _ptr(weight), _ptr(rows),
-             _ptr(out), _code(out, op), R, h, float(eps), _ptr(delta_scale), _stream()), op)
+             _ptr(out), _code(out, op), R, h, float(eps), _ptr(delta_scale), parts, T * h, _ptr(extra), _ptr(vec), _stream()), op)
 
 
 @_timed
@@ -376,13 +424,13 @@ def cast_rows(src: torch.Tensor, out: torch.Tensor) -> None:
     _check(f(_ptr(src), _ptr(out), _code(out, op), src.numel(), _stream()), op)
 
 
-ACTIVATIONS = {"xielu": 0}
+ACTIVATIONS = {"xielu": 0, "relu2": 1}
 
 
 @_timed
-def activation(x: torch.Tensor, out: torch.Tensor, kind: str, params: torch.Tensor) -> None:
+def activation(x: torch.Tensor, out: torch.Tensor, kind: str, params: Optional[torch.Tensor] = None) -> None:
     """out[t, j] = act(x[t, j]), float32 arithmetic. "xielu" with params = float32 [ap, an] on the device:
-    z > 0: ap z^2 + z / 2; z <= 0: an (exp(z) - 1 - z) + z / 2. `out` may be `x` itself."""
+    z > 0: ap z^2 + z / 2; z <= 0: an (exp(z) - 1 - z) + z / 2. "relu2": max(z, 0)^2. `out` may be `x` itself."""
     op = "activation"
     _cuda(op, x, out, params)
     _rows_2d(x, op, "x")
@@ -390,6 +438,8 @@ def activation(x: torch.Tensor, out: torch.Tensor, kind: str, params: torch.Tens
         raise ShapeError(op, f"activation {kind!r} is not known ({', '.join(ACTIVATIONS)})")
     if out.shape != x.shape or out.dtype != x.dtype or not out.is_contiguous():
         raise ShapeError(op, f"out must be contiguous {x.dtype} {list(x.shape)}, got {out.dtype} {list(out.shape)}")
+    if kind == "xielu" and params is None:
+        raise ShapeError(op, "xielu takes two numbers")
     _f32_vec(params, 2, op, "params")
     f = _fn("elementwise", "vob_act", [_P, _L, _P, _I, _I, _I, _I, _P, _P])
     _check(f(_ptr(x), x.stride(0), _ptr(out), _code(out, op), x.shape[0], x.shape[1], ACTIVATIONS[kind], _ptr(params), _stream()), op)
@@ -1339,15 +1389,17 @@ def _moe_tiles(op, sorted_pairs, tile_expert, tile_rows, tensor_cores, width, ff
 @_timed
 def moe_gate_up(x: torch.Tensor, w_gu: torch.Tensor, sorted_pairs: torch.Tensor, tile_expert: torch.Tensor, top: int,
                 h_out: torch.Tensor, tensor_cores: bool = False, tile_rows: int = MOE_TILE_ROWS, activation: str = "silu",
-                limit: float = 0.0) -> None:
+                limit: float = 0.0, pair_w: Optional[torch.Tensor] = None) -> None:
     """h_out[pair] = silu(W_gate[e] x[token]) * (W_up[e] x[token]) for every pair of the ordered list; w_gu [E, 2 ff, width]
     (an expert's gate rows, then its up rows) and h_out [T * top, ff] of x's type. `tensor_cores`: the bfloat16 tile form.
-    `activation` "clamped_swish": g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1)."""
+    `activation` "clamped_swish": g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1).
+    `pair_w` (float32 [T, top]): the experts read pair_w * x (both float32 sums are multiplied by it)."""
     op = "moe_gate_up"
     if activation not in MOE_ACTIVATIONS or (activation == "clamped_swish" and not limit > 0):
         raise ShapeError(op, f"activation {activation!r} (limit {limit}) is not known ({', '.join(MOE_ACTIVATIONS)}; the clamped one "
                              f"needs a positive limit)")
-    _cuda(op, x, w_gu, sorted_pairs, tile_expert, h_out)
+    _cuda(op, x, w_gu, sorted_pairs, tile_expert, h_out, pair_w)
+    _f32_vec(pair_w, x.shape[0] * top, op, "pair_w")
     _rows_2d(x, op, "x")
     T, width = x.shape
     if w_gu.dim() != 3 or w_gu.shape[2] != width or w_gu.shape[1] % 2 or w_gu.dtype != x.dtype or not w_gu.is_contiguous():
@@ -1360,9 +1412,9 @@ def moe_gate_up(x: torch.Tensor, w_gu: torch.Tensor, sorted_pairs: torch.Tensor,
     tiles = _moe_tiles(op, sorted_pairs, tile_expert, tile_rows, tensor_cores, width, ff)
     if tile_rows != MOE_TILE_ROWS and (x.stride(0) % 8 or x.data_ptr() % 16):
         raise ShapeError(op, f"tiles of {tile_rows} rows need rows of x that start on 16-byte boundaries")
-    f = _fn("moe", "vob_moe_gate_up", [_P, _I, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P])
+    f = _fn("moe", "vob_moe_gate_up", [_P, _I, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _F, _P, _P])
     _check(f(_ptr(x), _code(x, op), x.stride(0), _ptr(w_gu), _ptr(sorted_pairs), _ptr(tile_expert), tiles, int(tile_rows), int(top), width, ff,
-             _ptr(h_out), 1 if tensor_cores else 0, MOE_ACTIVATIONS[activation], float(limit), _stream()), op)
+             _ptr(h_out), 1 if tensor_cores else 0, MOE_ACTIVATIONS[activation], float(limit), _ptr(pair_w), _stream()), op)
 
 
 @_timed
@@ -1392,10 +1444,10 @@ def moe_up(x: torch.Tensor, w_up: torch.Tensor, sorted_pairs: torch.Tensor, tile
 
 
 @_timed
-def moe_down(h: torch.Tensor, w_down: torch.Tensor, sorted_pairs: torch.Tensor, tile_expert: torch.Tensor, pair_w: torch.Tensor,
+def moe_down(h: torch.Tensor, w_down: torch.Tensor, sorted_pairs: torch.Tensor, tile_expert: torch.Tensor, pair_w: Optional[torch.Tensor],
              y: torch.Tensor, tensor_cores: bool = False, tile_rows: int = MOE_TILE_ROWS) -> None:
     """y[pair] = pair_w[pair] * (W_down[e] h[pair]), float32 [T * top, width]; w_down [E, width, ff] of h's type; pair_w
-    float32 [T, top]."""
+    float32 [T, top], or None for weights of 1."""
     op = "moe_down"
     _cuda(op, h, w_down, sorted_pairs, tile_expert, pair_w, y)
     if h.dim() != 2 or not h.is_contiguous():
@@ -1404,8 +1456,7 @@ def moe_down(h: torch.Tensor, w_down: torch.Tensor, sorted_pairs: torch.Tensor, 
     if w_down.dim() != 3 or w_down.shape[2] != ff or w_down.dtype != h.dtype or not w_down.is_contiguous():
         raise ShapeError(op, f"w_down must be contiguous {h.dtype} [experts, width, {ff}], got {w_down.dtype} {list(w_down.shape)}")
     width = w_down.shape[1]
-    if pair_w.dtype != torch.float32 or pair_w.numel() != P or not pair_w.is_contiguous():
-        raise ShapeError(op, f"pair_w must be contiguous float32 of {P} entries, got {pair_w.dtype} {list(pair_w.shape)}")
+    _f32_vec(pair_w, P, op, "pair_w")
     if y.dtype != torch.float32 or y.shape != (P, width) or not y.is_contiguous():
         raise ShapeError(op, f"y must be contiguous float32 [{P}, {width}], got {y.dtype} {list(y.shape)}")
     if tensor_cores and h.dtype != torch.bfloat16:
@@ -1444,32 +1495,66 @@ def moe_combine(y: torch.Tensor, idx: torch.Tensor, out: torch.Tensor, shared: O
 
 # ------------------------------------------------------------------------------------ attention over a latent cache
 @_timed
-def latent_prep(proj: torch.Tensor, q_off: int, heads: int, dim: int, rot: int, down_off: int, rank: int, norm_w: torch.Tensor,
+def latent_prep(q: Optional[torch.Tensor], heads: int, dim: int, rot: int, down: Optional[torch.Tensor], rank: int, norm_w: torch.Tensor,
                 eps: float, positions: torch.Tensor, slots: Optional[torch.Tensor], inv_freq: torch.Tensor, lat: torch.Tensor,
-                kr: torch.Tensor, q_rot: torch.Tensor) -> None:
-    """Per token: the latent (first `rank` columns of the down projection, RMS norm with weight) and the
-    rotated key part (its last `rot` columns, rotary positions) go to the token's cache slot (lat
-    [pages, 1, page, rank], kr [pages, 1, page, rot]); the rotated query part of every head (the last
-    `rot` of its dim + rot columns) goes to q_rot float32 [T, heads, rot]."""
+                kr: torch.Tensor, q_rot: Optional[torch.Tensor], mag: float = 1.0, low: Optional[torch.Tensor] = None,
+                low_w: Optional[torch.Tensor] = None, low_out: Optional[torch.Tensor] = None) -> None:
+    """Per token, any of three jobs. With `slots`: the latent (first `rank` columns of `down` [T, rank + rot], RMS norm with
+    weight) and the rotated key part (its last `rot` columns, rotary positions) go to the token's cache slot (lat
+    [pages, 1, page, rank], kr [pages, 1, page, rot]). With `q` [T, heads * (dim + rot)]: the rotated query part of every head
+    (the last `rot` of its columns) goes to q_rot float32 [T, heads, rot]. With `low` [T, n]: low_out [T, n] = low_w * low /
+    sqrt(mean(low^2) + eps). Cosine and sine are multiplied by `mag`."""
     op = "latent_prep"
-    _cuda(op, proj, norm_w, positions, slots, inv_freq, lat, kr, q_rot)
-    _rows_2d(proj, op, "proj")
-    T = proj.shape[0]
-    if q_off < 0 or q_off + heads * (dim + rot) > proj.shape[1] or down_off < 0 or down_off + rank + rot > proj.shape[1]:
-        raise ShapeError(op, f"the query or down-projection columns lie outside proj's {proj.shape[1]}")
+    _cuda(op, q, down, norm_w, positions, slots, inv_freq, lat, kr, q_rot, low, low_w, low_out)
+    T = positions.shape[0]
+    dt = lat.dtype
+    for name, t, w in (("q", q, heads * (dim + rot)), ("down", down, rank + rot), ("low", low, low.shape[1] if low is not None else 0)):
+        if t is None:
+            continue
+        _rows_2d(t, op, name)
+        if t.shape != (T, w) or t.dtype != dt:
+            raise ShapeError(op, f"{name} must be {dt} [{T}, {w}], got {t.dtype} {list(t.shape)}")
     for name, t, w in (("lat", lat, rank), ("kr", kr, rot)):
-        if t.dim() != 4 or t.shape[1] != 1 or t.shape[3] != w or not t.is_contiguous() or t.dtype != proj.dtype:
-            raise ShapeError(op, f"{name} must be contiguous {proj.dtype} [pages, 1, page, {w}], got {t.dtype} {list(t.shape)}")
-    if q_rot.shape != (T, heads, rot) or q_rot.dtype != torch.float32 or not q_rot.is_contiguous():
-        raise ShapeError(op, f"q_rot must be contiguous float32 [{T}, {heads}, {rot}], got {q_rot.dtype} {list(q_rot.shape)}")
+        if t.dim() != 4 or t.shape[1] != 1 or t.shape[3] != w or not t.is_contiguous() or t.dtype != dt:
+            raise ShapeError(op, f"{name} must be contiguous {dt} [pages, 1, page, {w}], got {t.dtype} {list(t.shape)}")
+    if q is not None and (q_rot is None or q_rot.shape != (T, heads, rot) or q_rot.dtype != torch.float32 or not q_rot.is_contiguous()):
+        raise ShapeError(op, f"q_rot must be contiguous float32 [{T}, {heads}, {rot}]")
+    if slots is not None and down is None:
+        raise ShapeError(op, "a cache write needs the down projection")
+    if low is not None:
+        if low_out is None or low_out.shape != low.shape or low_out.dtype != dt or not low_out.is_contiguous() or low_w is None:
+            raise ShapeError(op, f"low_out must be contiguous {dt} {list(low.shape)} and low_w is needed")
+        _f32_vec(low_w, low.shape[1], op, "low_w")
     _f32_vec(norm_w, rank, op, "norm_w")
     _f32_vec(inv_freq, rot // 2, op, "inv_freq")
     _int32_vec(positions, T, op, "positions")
     if slots is not None:
         _int32_vec(slots, T, op, "slots")
-    f = _fn("latent_attention", "vob_latent_prep", [_P, _I, _L, _I, _I, _I, _I, _I, _I, _P, _F, _P, _P, _P, _P, _P, _I, _P, _I, _P])
-    _check(f(_ptr(proj), _code(proj, op), proj.stride(0), q_off, heads, dim, rot, down_off, rank, _ptr(norm_w), float(eps), _ptr(positions),
-             _ptr(slots), _ptr(inv_freq), _ptr(lat), _ptr(kr), _code(lat, op), _ptr(q_rot), T, _stream()), op)
+    f = _fn("latent_attention", "vob_latent_prep", [_P, _I, _L, _I, _I, _I, _P, _L, _I, _P, _F, _P, _P, _P, _F, _P, _P, _I, _P, _P, _L, _I,
+                                                    _P, _P, _I, _P])
+    _check(f(_ptr(q), _code(lat, op), q.stride(0) if q is not None else 0, heads, dim, rot, _ptr(down), down.stride(0) if down is not None else 0,
+             rank, _ptr(norm_w), float(eps), _ptr(positions), _ptr(slots), _ptr(inv_freq), float(mag), _ptr(lat), _ptr(kr), _code(lat, op),
+             _ptr(q_rot), _ptr(low), low.stride(0) if low is not None else 0, low.shape[1] if low is not None else 0, _ptr(low_w),
+             _ptr(low_out), T, _stream()), op)
+
+
+@_timed
+def latent_gate(vals: torch.Tensor, gate: torch.Tensor, out: torch.Tensor) -> None:
+    """out[t, h * V + i] = vals[t, h, i] * sigmoid(gate[t, h * V + i]); vals [T, heads, V] through its strides (last stride 1), gate
+    [T, heads * V] (rows any stride), out contiguous [T, heads * V] (may be vals' own memory where vals is contiguous)."""
+    op = "latent_gate"
+    _cuda(op, vals, gate, out)
+    _rows_2d(gate, op, "gate")
+    if vals.dim() != 3 or vals.stride(2) != 1:
+        raise ShapeError(op, f"vals must be [T, heads, V] with unit inner stride, got {list(vals.shape)}")
+    T, H, V = vals.shape
+    for name, t in (("gate", gate), ("out", out)):
+        if t.shape != (T, H * V) or t.dtype != vals.dtype:
+            raise ShapeError(op, f"{name} must be {vals.dtype} [{T}, {H * V}], got {t.dtype} {list(t.shape)}")
+    if not out.is_contiguous():
+        raise ShapeError(op, "out must be contiguous")
+    f = _fn("latent_attention", "vob_latent_gate", [_P, _I, _L, _L, _P, _L, _I, _I, _I, _P, _P])
+    _check(f(_ptr(vals), _code(vals, op), vals.stride(0), vals.stride(1), _ptr(gate), gate.stride(0), T, H, V, _ptr(out), _stream()), op)
 
 
 @_timed
@@ -1581,9 +1666,9 @@ def flex_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, positions:
               v_first: Optional[torch.Tensor], v_mode: int, q_out: torch.Tensor, kcache: Optional[torch.Tensor],
               vcache: Optional[torch.Tensor], heads: int, kv_heads: int, dim: int, vdim: int,
               q_norm_w: Optional[torch.Tensor] = None, k_norm_w: Optional[torch.Tensor] = None,
-              q_pre_w: Optional[torch.Tensor] = None, k_pre_w: Optional[torch.Tensor] = None) -> None:
+              q_pre_w: Optional[torch.Tensor] = None, k_pre_w: Optional[torch.Tensor] = None, rot_mag: float = 1.0) -> None:
     """Per token, from the columns q_off.., k_off.., v_off.. of `proj`: q and k with their first `rot` features rotated
-    (feature i with i + rot / 2, by position * inv_freq[i]), then (unit_rms) divided by sqrt(mean(x^2) + eps) per head;
+    (feature i with i + rot / 2, by position * inv_freq[i], cosine and sine both times `rot_mag`), then (unit_rms) divided by sqrt(mean(x^2) + eps) per head;
     q times 1 + coef * ln(floor((pos + 1) / every) + 1) for q_temp = (coef, every). q goes to q_out [T, heads * dim], k
     and v to their cache slots. v_mode 1 also leaves v in v_first [T, kv_heads * vdim]; v_mode 2 mixes
     v <- (1 - vmix) v + vmix v_first before the write (vmix: one float32 on the device). `q_norm_w`, `k_norm_w` (float32
@@ -1624,10 +1709,10 @@ def flex_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, positions:
     if v_mode == 2:
         _f32_vec(vmix, 1, op, "vmix")
     coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
-    f = _fn("attention_flex", "vob_flex_prep", [_P, _I, _L, _I, _I, _I, _P, _P, _P, _I, _I, _F, _F, _I, _P, _P, _P, _P, _P, _P, _I, _P, _L,
+    f = _fn("attention_flex", "vob_flex_prep", [_P, _I, _L, _I, _I, _I, _P, _P, _P, _I, _F, _I, _F, _F, _I, _P, _P, _P, _P, _P, _P, _I, _P, _L,
                                                 _P, _P, _I, _I, _I, _I, _I, _I, _P])
     _check(f(_ptr(proj), _code(proj, op), proj.stride(0), q_off, k_off, v_off, _ptr(positions), _ptr(slots), _ptr(inv_freq), int(rot),
-             1 if unit_rms else 0, float(eps), coef, every, _ptr(q_norm_w), _ptr(k_norm_w), _ptr(q_pre_w), _ptr(k_pre_w), _ptr(vmix), _ptr(v_first), int(v_mode),
+             float(rot_mag), 1 if unit_rms else 0, float(eps), coef, every, _ptr(q_norm_w), _ptr(k_norm_w), _ptr(q_pre_w), _ptr(k_pre_w), _ptr(vmix), _ptr(v_first), int(v_mode),
              _ptr(q_out), q_out.stride(0), _ptr(kcache), _ptr(vcache), T, heads, kv_heads, dim, vdim,
              kcache.shape[2] if kcache is not None else 1, _stream()), op)
 

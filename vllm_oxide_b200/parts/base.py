@@ -246,6 +246,8 @@ class Norm:
     # True for a norm that is a per-token scale times a per-feature weight (`weight`, `eps`):
     # that form commutes with a matrix product and can be folded into it (see FoldedState).
     scale_and_weight = False
+    several_parts = False       # True for a norm whose `forward` takes a delta of [parts, T, hidden] (the results of sub-layers that
+                                # ran side by side) and, as `extra` / `vec`, a row per token and one vector to add as well
     scalar_scale = False        # True for a norm whose `forward` takes one number as `delta_scale`
 
     def workspace_bytes(self, rows: int, act_bytes: int) -> int:
@@ -267,14 +269,24 @@ class PositionEncoding:
 
 
 # ------------------------------------------------------------------------------ a model as data
+@dataclass(frozen=True, eq=False)
+class CallEntry:
+    """What joins the residual right before one call of a block, in the pass of its first norm: the rows of the step buffer
+    `rows` (float32 [rows, hidden], say the embedding's output) and / or one float32 vector [hidden]."""
+    rows: Optional[str] = None
+    vector: Optional[torch.Tensor] = None
+
+
 @dataclass(frozen=True)
 class LayerCall:
     """One entry of the run order: run `layer` with cache number `cache` (None: the mixer keeps
     no pages). Naming a layer twice runs it twice (with two caches, or sharing one); `write`
-    False lets a call read a cache that an earlier call of the same step wrote."""
+    False lets a call read a cache that an earlier call of the same step wrote. `entry`: what is added to the
+    residual ahead of this call (its block takes `entry`: `ParallelBlock`)."""
     layer: int
     cache: Optional[int] = None
     write: bool = True
+    entry: Optional[CallEntry] = None
 
 
 @dataclass
@@ -289,7 +301,8 @@ class ModelSpec:
     max_position: Optional[int] = None  # longest position the position encodings allow
     eos_token_ids: Tuple[int, ...] = ()
     weight_bytes: int = 0               # bytes a decode step must read of the weights
+    pending_parts: int = 1              # tensors of [rows, hidden_size] a block hands on to be added (ParallelBlock: 2)
     residual_streams: int = 1           # the residual is float32 [rows, residual_streams * hidden_size]
     # buffers that live for one step and that layers hand to later layers through `StepContext.shared`:
-    # name -> (columns, dtype or None for the compute dtype); [rows, columns] each, allocated behind the embedding
+    # name -> (columns, dtype or None for the compute dtype); [rows, columns] each, there before the embedding runs
     step_buffers: Dict[str, Tuple[int, Optional[torch.dtype]]] = field(default_factory=dict)

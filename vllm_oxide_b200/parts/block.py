@@ -1,6 +1,6 @@
 """The arrangements of parts in one layer: the pre-norm residual block (`Block`), the block whose
-residual takes the normed result of each sub-layer (`PostNormBlock`) and the block with a norm on both sides of
-each sub-layer (`SandwichBlock`, at the end of the file).
+residual takes the normed result of each sub-layer (`PostNormBlock`), the block with a norm on both sides of
+each sub-layer (`SandwichBlock`) and the block whose sub-layers read one norm side by side (`ParallelBlock`, at the end).
 
     residual += mixer(norm1(residual));  residual += feed_forward(norm2(residual))
 (crates/engine/src/model.rs:302-332). The residual is float32. Each part's output is not added
@@ -328,3 +328,79 @@ class SandwichBlock:
         if self.depth_weights is not None and depth is None:
             kernels.depth_average(stack, resid, self.depth_weights, self.depth_index + 1)
         return None
+
+
+class ParallelBlock:
+    """h = norm(residual);  residual += mixer(h) + feed_forward(h)
+
+    One norm, read by both sub-layers. Neither result is added at once: both are handed on (`out` is [2, rows, hidden], the
+    model's `pending_parts` is 2) and the next norm's kernel adds them in float32 while it normalises. A block without
+    feed-forward hands on the mixer's alone. `entry` (see `CallEntry`): rows of a step buffer and a vector that join the residual
+    ahead of the norm, in the same kernel. In steps of single tokens the feed-forward may run on a second stream beside the mixer
+    (`TUNING.parallel_side_stream`): neither reads what the other writes."""
+
+    def __init__(self, norm1: Norm, mixer: Mixer, feed_forward: Optional[FeedForward]):
+        if not norm1.several_parts:
+            raise ValueError("the norm of this arrangement must take pending results in parts")
+        self.norm1, self.mixer, self.feed_forward = norm1, mixer, feed_forward
+        self.norm2 = None
+        self.pending_scale = None
+        self._side = None            # the second stream, made at first need
+
+    def _parts(self):
+        return [p for p in (self.norm1, self.mixer, self.feed_forward) if p is not None]
+
+    def weight_bytes(self) -> int:
+        return sum(getattr(p, "weight_bytes", lambda: 0)() for p in self._parts())
+
+    def workspace_bytes(self, rows: int, hidden: int, act_bytes: int) -> int:
+        """The normed rows and the larger of the two sub-layers' scratch; both where they may run at the same time."""
+        both = (self.mixer.workspace_bytes(rows), self.feed_forward.workspace_bytes(rows) if self.feed_forward is not None else 0)
+        return self.norm1.workspace_bytes(rows, act_bytes) + (sum(both) if TUNING.parallel_side_stream else max(both))
+
+    def folded_workspace_bytes(self, rows: int) -> int:
+        return 0
+
+    def kernel_modules(self, dtype, max_rows):
+        mods = ["elementwise"]
+        for p in self._parts():
+            mods += list(getattr(p, "kernel_modules", lambda d, r: ())(dtype, max_rows))
+        return tuple(mods)
+
+    def can_fold(self) -> bool:
+        return False
+
+    @staticmethod
+    def _into(part, dst: torch.Tensor, *args) -> None:
+        got = part.forward(*args, out=dst)
+        if got.data_ptr() != dst.data_ptr():
+            dst.copy_(got)
+
+    def forward(self, resid: torch.Tensor, pending: Optional[torch.Tensor], ctx: StepContext, cache: Optional[LayerCache], state,
+                out: torch.Tensor, pending_scale: Optional[torch.Tensor] = None, entry=None) -> torch.Tensor:
+        if pending_scale is not None:
+            raise ValueError("a block of this arrangement follows blocks whose results are added as they are")
+        if out.dim() != 3 or out.shape[0] < 2:
+            raise ValueError("a block of this arrangement hands on two results: the model's pending_parts must be 2")
+        ws = ctx.workspace
+        with ws.scope():
+            extra = ctx.shared[entry.rows] if entry is not None and entry.rows is not None else None
+            h = self.norm1.forward(resid, pending, ctx, extra=extra, vec=entry.vector if entry is not None else None)
+            if self.feed_forward is None:
+                self._into(self.mixer, out[0], h, ctx, cache, state)
+                return out[0]
+            if ctx.decode_only and TUNING.parallel_side_stream:
+                if self._side is None:
+                    self._side = torch.cuda.Stream(device=h.device)
+                side, main = self._side, torch.cuda.current_stream()
+                side.wait_stream(main)
+                with torch.cuda.stream(side):
+                    self._into(self.feed_forward, out[1], h, ctx)
+                self._into(self.mixer, out[0], h, ctx, cache, state)
+                main.wait_stream(side)
+                return out
+            with ws.scope():
+                self._into(self.mixer, out[0], h, ctx, cache, state)
+            with ws.scope():
+                self._into(self.feed_forward, out[1], h, ctx)
+        return out

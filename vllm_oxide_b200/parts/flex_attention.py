@@ -12,6 +12,7 @@ as parameters:
 * `keep_first`       (with `window`) every query also sees the request's first so many tokens, at their true distances
                      (their pages stay);
 * `rot_dims`, `rot_base`   partial rotary positions, feature i paired with i + rot_dims / 2;
+* `rot_table`        (frequencies, factor) in place of `rot_base`: one frequency per pair, cosine and sine times the factor;
 * `unit_rms_eps`     q and k divided by sqrt(mean(x^2) + eps) per head, after the rotation;
 * `q_norm_weight`, `k_norm_weight`   [dim] each, shared by the heads: q and k times it behind that division;
 * `q_pre_norm`, `k_pre_norm`   [heads * dim] / [kv_heads * dim], with `pre_norm_eps`: BEFORE the rotation the whole q (k)
@@ -71,7 +72,7 @@ class SoftmaxAttention(Mixer):
                  q_pre_norm: Optional[torch.Tensor] = None, k_pre_norm: Optional[torch.Tensor] = None,
                  pre_norm_eps: Optional[float] = None, pool: int = 0, pooled_sizes: Optional[Tuple[int, ...]] = None,
                  keep_first: int = 0, dist_slopes: Optional[torch.Tensor] = None, values_are_keys: bool = False,
-                 gate_per_head: bool = False):
+                 gate_per_head: bool = False, rot_table=None):
         self.values_are_keys = bool(values_are_keys)
         if self.values_are_keys:
             if wv is not None or bias_v is not None or shared_kv or value_mix or pool or rot_dims or unit_rms_eps is not None or q_temp:
@@ -154,7 +155,12 @@ class SoftmaxAttention(Mixer):
         self.rot = int(rot_dims)
         if self.rot % 2 or not 0 <= self.rot <= self.D:
             raise ValueError(f"{self.rot} rotated features do not fit a head of {self.D}")
-        self.inv_freq = torch.from_numpy(rotary_inv_freq(self.rot, rot_base).copy()).to(device) if self.rot else None
+        self.inv_freq, self.rot_mag = None, 1.0
+        if self.rot:
+            freq, self.rot_mag = rot_table if rot_table is not None else (rotary_inv_freq(self.rot, rot_base), 1.0)
+            if len(freq) != self.rot // 2:
+                raise ValueError(f"{len(freq)} frequencies do not fit {self.rot} rotated features")
+            self.inv_freq = torch.from_numpy(freq.copy()).to(device)
         self.unit_rms = unit_rms_eps is not None
         self.eps = float(unit_rms_eps) if self.unit_rms else 0.0
         self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp else None
@@ -295,7 +301,7 @@ class SoftmaxAttention(Mixer):
         kernels.flex_prep(proj, self.q_off, self.k_off, self.v_off, ctx.positions, ctx.slot_mapping[cache.group] if cache.write else None,
                           self.inv_freq, self.rot, self.unit_rms, self.eps, self.q_temp, self.mix_weight, v_first, self.v_mode, q,
                           None if self.shared_kv else kc, None if self.shared_kv else vc, self.H, self.G, self.D, self.DV,
-                          self.q_norm_w, self.k_norm_w, self.q_pre_w, self.k_pre_w)
+                          self.q_norm_w, self.k_norm_w, self.q_pre_w, self.k_pre_w, self.rot_mag)
         if cache.write:        # the blocks that this step's tokens complete, in every size the cache serves
             for i, size in enumerate(self.pooled_sizes):
                 kernels.pool_blocks(kc, vc, cache.tensors[2 + 2 * i], cache.tensors[3 + 2 * i], ctx.block_tables[cache.group], ctx.row_seq,

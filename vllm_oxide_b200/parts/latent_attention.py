@@ -13,7 +13,9 @@ sum to one, so W_uv (sum_j p_j c_j) = sum_j p_j W_uv c_j). A cached token costs 
 elements whatever the number of heads, and a decode step reads each of them once for all heads.
 Scores, softmax and the rotation are float32; the query in the latent space stays float32.
 
-Options: `window` (a query sees itself and the window - 1 tokens before it; pages behind the window are given back) and
+Options: queries that go through a latent of their own (`wdq`, `dq_norm`: c_q = RMSNorm(W_dq h, weight), q = W_q c_q with `wq`
+[heads * (dim + rot_dim), q_rank]); `rot_table` (one frequency per pair and a factor for cosine and sine, in place of `rot_base`);
+`gate_weight` [heads * vdim, hidden] (the heads' values, side by side, times sigmoid(W_g h) ahead of W_o); `window` (a query sees itself and the window - 1 tokens before it; pages behind the window are given back) and
 `pairing` of the rotated features: "half" (feature i with i + rot_dim / 2) or "interleaved" (2i with 2i + 1). The kernels
 rotate halves; the interleaved pairing is the same rotation on another order of the rotated rows of W_q and W_dkv, the same
 order for both (a score is a dot product, so a common order of q's and k's features changes nothing), applied here at load.
@@ -32,11 +34,17 @@ from .rotary import rotary_inv_freq
 
 class LatentAttention(Mixer):
     def __init__(self, wq, wdkv, dkv_norm, wuk, wuv, wo, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float,
-                 rot_base: float, eps: float, dtype=torch.bfloat16, device="cuda", window: int = 0, pairing: str = "half"):
+                 rot_base: float, eps: float, dtype=torch.bfloat16, device="cuda", window: int = 0, pairing: str = "half",
+                 wdq=None, dq_norm=None, rot_table=None, gate_weight=None):
         self.H, self.D, self.R, self.V, self.L = int(heads), int(dim), int(rot_dim), int(vdim), int(kv_rank)
         H, D, R, V, L = self.H, self.D, self.R, self.V, self.L
-        hidden = wq.shape[1]
-        if wq.shape != (H * (D + R), hidden) or wdkv.shape != (L + R, hidden) or wuk.shape != (H * D, L) or wuv.shape != (H * V, L) \
+        hidden = wdkv.shape[1]
+        self.Q = int(wdq.shape[0]) if wdq is not None else 0              # size of the queries' latent, 0: none
+        if (wdq is None) != (dq_norm is None) or (wdq is not None and (wdq.shape != (self.Q, hidden) or dq_norm.shape != (self.Q,))):
+            raise ValueError("a latent for the queries takes a projection from the layer's width and a norm weight of its size")
+        if gate_weight is not None and gate_weight.shape != (H * V, hidden):
+            raise ValueError(f"gate projection {list(gate_weight.shape)} does not fit {H * V} x {hidden}")
+        if wq.shape != (H * (D + R), self.Q or hidden) or wdkv.shape != (L + R, hidden) or wuk.shape != (H * D, L) or wuv.shape != (H * V, L) \
                 or wo.shape != (hidden, H * V) or dkv_norm.shape != (L,):
             raise ValueError(f"projection shapes do not fit {H} heads of {D}+{R} / {V} with a latent of {L} over a width of {hidden}")
         if R % 2 or R <= 0:
@@ -52,13 +60,23 @@ class LatentAttention(Mixer):
             wq = wq[qrows.reshape(-1).to(wq.device)]
             krows = torch.cat([torch.arange(L), L + order])
             wdkv = wdkv[krows.to(wdkv.device)]
-        self.w_in = to_compute(torch.cat([wq, wdkv], dim=0), dtype, device)
+        # one product of the layer's input: queries (or their latent), the down projection, the gate
+        first = [wdq if self.Q else wq, wdkv] + ([gate_weight] if gate_weight is not None else [])
+        self.w_in = to_compute(torch.cat(first, dim=0), dtype, device)
+        self.w_uq = to_compute(wq, dtype, device) if self.Q else None
+        self.low_w = dq_norm.to(device=device, dtype=torch.float32).contiguous() if self.Q else None
+        self.down_off = self.Q or H * (D + R)
+        self.gate_off = self.down_off + L + R
+        self.gated = gate_weight is not None
         # per head, as `linear` wants its weights ([out, in]): latent <- plain query features, values <- latent
         self.w_qlat = to_compute(wuk.reshape(H, D, L).transpose(1, 2), dtype, device)          # [H, L, D]
         self.w_val = to_compute(wuv.reshape(H, V, L), dtype, device)                            # [H, V, L]
         self.w_o = to_compute(wo, dtype, device)
         self.norm_weight = dkv_norm.to(device=device, dtype=torch.float32).contiguous()
-        self.inv_freq = torch.from_numpy(rotary_inv_freq(R, rot_base).copy()).to(device)
+        freq, self.rot_mag = rot_table if rot_table is not None else (rotary_inv_freq(R, rot_base), 1.0)
+        if len(freq) != R // 2:
+            raise ValueError(f"{len(freq)} frequencies do not fit {R} rotated features")
+        self.inv_freq = torch.from_numpy(freq.copy()).to(device)
         self.scale, self.eps, self.hidden, self.dtype = float(scale), float(eps), hidden, dtype
         self.batched = True       # bfloat16: the per-head products as one batched library product (False: one by one, tests)
         self.num_sms = torch.cuda.get_device_properties(device).multi_processor_count
@@ -79,7 +97,8 @@ class LatentAttention(Mixer):
         return CacheSpec(kind=kind, window=self.window, tensors=(PagedTensorSpec(1, self.L), PagedTensorSpec(1, self.R)))
 
     def weight_bytes(self) -> int:
-        return (self.w_in.numel() + self.w_qlat.numel() + self.w_val.numel() + self.w_o.numel()) * self.w_in.element_size()
+        uq = self.w_uq.numel() if self.Q else 0
+        return (self.w_in.numel() + uq + self.w_qlat.numel() + self.w_val.numel() + self.w_o.numel()) * self.w_in.element_size()
 
     def workspace_bytes(self, rows: int) -> int:
         es, H = self.w_in.element_size(), self.H
@@ -87,7 +106,8 @@ class LatentAttention(Mixer):
         if self.splits is None:     # the most any step of at most `rows` rows takes: below one block per SM every row has 32 shares
             few = min(rows, self.num_sms // -(-H // 8))
             parts = max(parts, aligned(few * H * 32 * (self.L + 2) * 4))
-        return (aligned(rows * self.w_in.shape[0] * es) + aligned(rows * H * self.R * 4) + aligned(rows * H * self.L * 4)
+        low = aligned(rows * self.Q * es) + aligned(rows * H * (self.D + self.R) * es) if self.Q else 0
+        return (low + aligned(rows * self.w_in.shape[0] * es) + aligned(rows * H * self.R * 4) + aligned(rows * H * self.L * 4)
                 + aligned(rows * H * self.L * es) + 2 * aligned(rows * H * self.V * es) + parts)
 
     def kernel_modules(self, dtype, max_rows):
@@ -101,9 +121,20 @@ class LatentAttention(Mixer):
         lat, kr = cache.tensors
         proj = matmul(x, self.w_in, ctx.alloc((T, self.w_in.shape[0])))
         q_rot = ctx.alloc((T, H, R), torch.float32)
-        kernels.latent_prep(proj, 0, H, D, R, H * (D + R), L, self.norm_weight, self.eps, ctx.positions,
-                            ctx.slot_mapping[cache.group] if cache.write else None, self.inv_freq, lat, kr, q_rot)
-        q_heads = proj[:, :H * (D + R)].view(T, H, D + R)[:, :, :D]                 # [T, H, D], strided
+        down = proj[:, self.down_off:self.down_off + L + R]
+        slots = ctx.slot_mapping[cache.group] if cache.write else None
+        common = (self.norm_weight, self.eps, ctx.positions)
+        if self.Q:
+            low = ctx.alloc((T, self.Q))
+            kernels.latent_prep(None, H, D, R, down, L, *common, slots, self.inv_freq, lat, kr, None, self.rot_mag, proj[:, :self.Q],
+                                self.low_w, low)
+            q = matmul(low, self.w_uq, ctx.alloc((T, H * (D + R))))
+            kernels.latent_prep(q, H, D, R, None, L, *common, None, self.inv_freq, lat, kr, q_rot, self.rot_mag)
+        else:
+            q = proj[:, :H * (D + R)]
+            kernels.latent_prep(q, H, D, R, down, L, *common, slots, self.inv_freq, lat, kr, q_rot, self.rot_mag)
+        q_heads = q.view(T, H, D + R)[:, :, :D]                                    # [T, H, D], strided
+        gate = proj[:, self.gate_off:self.gate_off + H * V] if self.gated else None
         bt = ctx.block_tables[cache.group]
         splits = self.key_splits(T)
         partials = ctx.alloc((T * H * splits * (L + 2),), torch.float32) if splits > 1 else None
@@ -124,7 +155,10 @@ class LatentAttention(Mixer):
             vals = ctx.alloc((H, T, V))
             torch.bmm(out_lat, self.w_val.transpose(1, 2), out=vals)
             attn = ctx.alloc((T, H * V))
-            attn.view(T, H, V).copy_(vals.transpose(0, 1))
+            if gate is not None:
+                kernels.latent_gate(vals.transpose(0, 1), gate, attn)              # heads side by side and gated in one pass
+            else:
+                attn.view(T, H, V).copy_(vals.transpose(0, 1))
         else:
             q_lat = ctx.alloc((T, H, L), torch.float32)
             for h in range(H):
@@ -134,4 +168,6 @@ class LatentAttention(Mixer):
             attn = ctx.alloc((T, H * V))
             for h in range(H):
                 kernels.linear(out_lat[:, h], self.w_val[h], attn[:, h * V:(h + 1) * V])
+            if gate is not None:
+                kernels.latent_gate(attn.view(T, H, V), gate, attn)
         return matmul(attn, self.w_o, out if out is not None else ctx.alloc((T, self.hidden)))

@@ -3,11 +3,12 @@
 act = "xielu" with two learned numbers p and q (one pair per layer):
     z > 0:  softplus(p) z^2 + z / 2;      z <= 0:  (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2
 The two factors are worked out once, in float32, when the part is built; the activation itself is float32
-arithmetic on the product's result in the activations' type.
+arithmetic on the product's result in the activations' type. act = "relu2": max(z, 0)^2, no numbers.
 """
 from __future__ import annotations
 
 import math
+from typing import Optional
 
 import torch
 
@@ -21,18 +22,21 @@ def _softplus(z: float) -> float:
 
 
 class ActMLP(FeedForward):
-    def __init__(self, w_up: torch.Tensor, w_down: torch.Tensor, act_params: torch.Tensor, dtype=torch.bfloat16, device="cuda",
+    def __init__(self, w_up: torch.Tensor, w_down: torch.Tensor, act_params: Optional[torch.Tensor], dtype=torch.bfloat16, device="cuda",
                  activation: str = "xielu"):
         inter, hidden = w_up.shape
         if w_down.shape != (hidden, inter):
             raise ValueError(f"feed-forward shapes do not fit: up {list(w_up.shape)}, down {list(w_down.shape)}")
         if activation not in kernels.ACTIVATIONS:
             raise ValueError(f"activation {activation!r} is not known ({', '.join(kernels.ACTIVATIONS)})")
-        if act_params.numel() != 2:
-            raise ValueError(f"xielu takes two numbers, got {list(act_params.shape)}")
-        p, q = (float(v) for v in act_params.float().reshape(2).tolist())
-        self.activation = activation
-        self.params = torch.tensor([_softplus(p), 0.5 + _softplus(q)], dtype=torch.float32, device=device)
+        self.activation, self.params = activation, None
+        if activation == "xielu":
+            if act_params is None or act_params.numel() != 2:
+                raise ValueError(f"xielu takes two numbers, got {None if act_params is None else list(act_params.shape)}")
+            p, q = (float(v) for v in act_params.float().reshape(2).tolist())
+            self.params = torch.tensor([_softplus(p), 0.5 + _softplus(q)], dtype=torch.float32, device=device)
+        elif act_params is not None:
+            raise ValueError(f"activation {activation!r} takes no numbers")
         self.inter, self.hidden, self.dtype = inter, hidden, dtype
         self.w_up = to_compute(w_up, dtype, device)
         self.w_down = to_compute(w_down, dtype, device)

@@ -11,7 +11,8 @@ same form that every token uses, added to the sum, times sigmoid(w_gate_scalar x
 Experts without a gate (`w_gate` None) compute W_down[e] act(W_up[e] x) with `activation` "relu2" (relu squared). `score`
 "sigmoid": s = sigmoid(z); `correction` [E]: the election (groups and experts) goes by s + correction, the weights by s;
 `group_best` 2: a run scores as the sum of its two best experts; `renormalize` divides by the sum + `renorm_eps`; `weight_scale`
-multiplies the weights.
+multiplies the weights. `weight_on_input` (gated experts): an expert reads w_e * x and its result is added as it is, in place of
+being multiplied by w_e behind its last product.
 Softmax over all experts followed by `renormalize` over the chosen ones is the softmax over the chosen logits alone.
 
 Per step: the election (one warp per token), the (token, expert) pairs put in order of their expert on the device
@@ -38,7 +39,7 @@ class RoutedExperts(FeedForward):
                  w_down: Sequence[torch.Tensor], top: int, groups: int = 0, keep: int = 0, renormalize: bool = False,
                  dtype=torch.bfloat16, device="cuda", activation: str = "silu", limit: float = 0.0, shared=None,
                  score: str = "softmax", correction: Optional[torch.Tensor] = None, group_best: int = 1, renorm_eps: float = 0.0,
-                 weight_scale: float = 1.0):
+                 weight_scale: float = 1.0, weight_on_input: bool = False):
         E, hidden = w_router.shape
         self.gated = w_gate is not None
         if not self.gated:
@@ -80,6 +81,9 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"activation {activation!r} with limit {limit}: known are {', '.join(kernels.MOE_ACTIVATIONS)}, and the "
                              f"clamped one needs a positive limit")
         self.activation, self.limit = activation, float(limit)
+        self.weight_on_input = bool(weight_on_input)
+        if self.weight_on_input and not self.gated:
+            raise ValueError("a weight on an expert's input goes with gated experts")
         self._side = None           # a second stream for the shared expert in steps of single tokens, made at first need
         self.shared = None
         if shared is not None:
@@ -117,6 +121,11 @@ class RoutedExperts(FeedForward):
 
     def _shared_expert(self, x, gu, hs, sh):
         w_gu, w_down, fs, gated, slimit = self.shared
+        if (self.activation == "silu" and not gated and self.dtype == torch.bfloat16 and x.shape[0] <= TUNING.few_rows
+                and kernels.gemm_sm100_supported(x, w_gu)):
+            kernels.gemm_swiglu(x, w_gu, hs)             # few rows: the gate in the product's epilogue
+            kernels.linear(hs, w_down, sh)
+            return
         kernels.linear(x, w_gu, gu)
         if self.activation == "clamped_swish":
             kernels.glu_clamped(gu[:, :2 * fs], hs, slimit)
@@ -151,11 +160,12 @@ class RoutedExperts(FeedForward):
         kernels.moe_align(idx, self.E, order, tile_expert, self.meta, tile)
         h = ctx.alloc((P, self.ff))
         if self.gated:
-            kernels.moe_gate_up(x, self.w_gu, order, tile_expert, self.top, h, self.tensor_cores, tile, self.activation, self.limit)
+            kernels.moe_gate_up(x, self.w_gu, order, tile_expert, self.top, h, self.tensor_cores, tile, self.activation, self.limit,
+                                w if self.weight_on_input else None)
         else:
             kernels.moe_up(x, self.w_gu, order, tile_expert, self.top, h, self.activation, self.tensor_cores, tile)
         y = ctx.alloc((P, self.hidden), torch.float32)
-        kernels.moe_down(h, self.w_down, order, tile_expert, w, y, self.tensor_cores, tile)
+        kernels.moe_down(h, self.w_down, order, tile_expert, None if self.weight_on_input else w, y, self.tensor_cores, tile)
         out = out if out is not None else ctx.alloc((T, self.hidden))
         if side is not None:
             torch.cuda.current_stream().wait_stream(side)

@@ -3,7 +3,9 @@
 out = weight * (x * 1/sqrt(mean(x^2) + eps)), weight last, sums in float32
 (crates/engine/src/backend/cpu/mod.rs:182-197). The block hands the norm the float32 residual
 and the delta its previous part produced; the kernel adds the delta into the residual (the
-reference's `add`, :351-358) and normalises the sum in one pass over the row.
+reference's `add`, :351-358) and normalises the sum in one pass over the row. A delta in parts
+([parts, T, width], what sub-layers that ran side by side returned) is added part by part, and
+with `extra` / `vec` a float32 row per token and one vector join the residual in the same pass.
 """
 from __future__ import annotations
 
@@ -16,6 +18,7 @@ from .base import Norm, StepContext, aligned
 
 
 class RMSNorm(Norm):
+    several_parts = True          # `forward` takes a delta in parts, and `extra` and `vec`
     scale_and_weight = True       # out = weight * (x * scale(x)): folds into the products around it
 
     def __init__(self, weight: torch.Tensor, eps: float, device, unit_offset: bool = False):
@@ -41,9 +44,10 @@ class RMSNorm(Norm):
 
     def forward(self, resid: torch.Tensor, delta: Optional[torch.Tensor], ctx: StepContext,
                 rows: Optional[torch.Tensor] = None, num_rows: Optional[int] = None,
-                delta_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                delta_scale: Optional[torch.Tensor] = None, extra: Optional[torch.Tensor] = None,
+                vec: Optional[torch.Tensor] = None) -> torch.Tensor:
         n = resid.shape[0] if rows is None else (num_rows if num_rows is not None else rows.numel())
         out = ctx.alloc((n, self.width))
         kernels.add_rmsnorm(resid, delta, self.weight, self.eps, out, rows[:n] if rows is not None else None,
-                            delta_scale if delta is not None else None)
+                            delta_scale if delta is not None else None, extra, vec)
         return out

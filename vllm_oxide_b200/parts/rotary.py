@@ -10,6 +10,8 @@ is computed in float64 and rounded. The rotation (rotate-half pairing, angle = f
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
+from typing import Optional, Tuple
 
 import numpy as np
 import torch
@@ -43,6 +45,34 @@ def rotary_inv_freq(head_dim: int, theta: float, scaling=None) -> np.ndarray:
             smooth = (old_ctx / wavelen - low) / (high - low)
             out[i] = (f32(1.0) - smooth) * v / factor + smooth * v
     return out
+
+
+@dataclass(frozen=True)
+class YarnScaling:
+    """Stretched rotary positions: pairs that turn often over `original` positions keep their frequency, pairs that turn seldom
+    have it divided by `factor`, and between `fast` and `slow` turns the two are blended."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+def rotary_table(dims: int, base: float, scaling: Optional[YarnScaling] = None) -> Tuple[np.ndarray, float]:
+    """(float32 frequency of each pair of features, the factor cosine and sine are multiplied by), worked out in float64 and
+    rounded once. Without scaling base^(-2 i / dims) and 1. With it, let d(n) = dims ln(original / (2 pi n)) / (2 ln base) be the
+    feature index whose pair turns n times over `original` positions: pair i is blended by how far i lies between
+    floor(d(fast)) (not below 0) and ceil(d(slow)) (not above dims - 1), and the factor is 0.1 ln(factor) + 1."""
+    freq = np.power(np.float64(base), -2.0 * np.arange(dims // 2, dtype=np.float64) / dims)
+    if scaling is None:
+        return freq.astype(np.float32), 1.0
+
+    def index_of(turns: float) -> float:
+        return dims * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo = max(math.floor(index_of(scaling.fast)), 0)
+    hi = min(math.ceil(index_of(scaling.slow)), dims - 1)
+    ramp = np.clip((np.arange(dims // 2) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    freq = freq / scaling.factor * ramp + freq * (1.0 - ramp)
+    return freq.astype(np.float32), 0.1 * math.log(scaling.factor) + 1.0
 
 
 class Rotary(PositionEncoding):

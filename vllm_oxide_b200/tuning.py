@@ -40,6 +40,9 @@ class Tuning:
     # a decode step with it, 1.69 ms without (a join between streams ends the overlap of neighbouring kernels that
     # programmatic dependent launch gives a single chain).
     moe_side_stream: int = 0
+    # In steps of single tokens a block whose sub-layers read one norm runs its feed-forward on a second stream beside its mixer
+    # and joins before the next norm. 1: it does; 0: one chain.
+    parallel_side_stream: int = 0
 
 
 TUNING = Tuning()
