@@ -1327,6 +1327,170 @@ def fanopel_compare(a):
     return 0
 
 
+# Layer sizes at which the Robuvik design is measured beside Pironex, the closest design the engine has (latent attention with
+# interleaved rotary positions, attention in a window, routed experts beside a shared one), both built of the same run of layers
+# with the same width, heads, latent, window and experts; Pironex without its convolutions, pooled blocks and caps.
+ROBUVIK_SIZES = {
+    "1b": dict(lomopel="1b", window=1024, q_rank=768, moe=dict(ff=1024, experts=8, top=2, shared_ff=2048)),
+    "3b": dict(lomopel="3b", window=1024, q_rank=1024, moe=dict(ff=1024, experts=8, top=2, shared_ff=2048)),
+}
+ROBUVIK_LAYERS, ROBUVIK_LOOP = "LAALA", (1, 4, 2)          # latent attention / attention; three layers run twice: LAALAALA
+
+
+def robuvik_runs():
+    """The kinds of the layers in the order they run."""
+    a, b, times = ROBUVIK_LOOP
+    return ROBUVIK_LAYERS[:a] + ROBUVIK_LAYERS[a:b] * times + ROBUVIK_LAYERS[b:]
+
+
+def make_side_by_side_engine(arch, rs, max_seqs, tokens_per_request, context):
+    """(config, LLM): eight runs of layers of the Robuvik design, or as many Pironex layers of the same kinds, random weights drawn
+    on the device."""
+    import torch
+    from vllm_oxide_b200 import models
+    from vllm_oxide_b200 import config as cf
+    from vllm_oxide_b200.engine import LLM, ModelRunner
+    from vllm_oxide_b200.weights import random_tensors
+    ls = LOMOPEL_SIZES[rs["lomopel"]]
+    at, lat, m = ls["attn"], ROTEPEL_SIZES[ls["llama"]]["latent"], rs["moe"]
+    scale, lscale = at["dim"] ** -0.5, (lat["dim"] + lat["rot_dim"]) ** -0.5
+    common = dict(vocab=128256, width=ls["width"], norm_eps=1e-5)
+    if arch == "robuvik":
+        def rot(n):
+            return cf.StretchedRotaryConfig(dims=n, base=5e5, factor=8.0, original=8192.0, fast=32.0, slow=1.0)
+        moe = cf.DenseOrExpertsConfig("moe", **m)
+        kinds = {"A": cf.RobuvikLayer("attention", attention=cf.WindowAttentionConfig(scale=scale, rot=rot(at["dim"]), window=rs["window"], **at), mlp=moe),
+                 "L": cf.RobuvikLayer("latent_attention", latent=cf.GatedLatentConfig(q_rank=rs["q_rank"], scale=lscale, rot=rot(lat["rot_dim"]), **lat), mlp=moe)}
+        cfg = cf.RobuvikConfig(layers=tuple(kinds[k] for k in ROBUVIK_LAYERS), loop=ROBUVIK_LOOP,
+                               bigram=cf.BigramConfig(buckets=65521, mul_prev=8191, mul_cur=131), **common)
+        manifest = models.robuvik_manifest(cfg)
+    else:
+        moe = cf.ClampedExpertsConfig(limit=7.0, shared_limit=7.0, **m)
+        kinds = {"A": cf.PironexLayer("attention", attention=cf.PooledAttentionConfig(scale=scale, rot_dims=at["dim"], rot_base=5e5, window=rs["window"], **at), mlp=moe),
+                 "L": cf.PironexLayer("latent_attention", latent=cf.WindowLatentConfig(scale=lscale, rot_base=5e5, **lat), mlp=moe)}
+        cfg = cf.PironexConfig(layers=tuple(kinds[k] for k in robuvik_runs()), **common)
+        manifest = models.pironex_manifest(cfg)
+    pages_per_req = -(-(tokens_per_request + 16) // 16)
+    fields = dict(max_batch_tokens=2048, max_seqs=max_seqs, max_model_len=context, block_size=16,
+                  num_pages=max_seqs * pages_per_req + 8, dtype="bfloat16", cuda_graphs=True)
+    fields.update(ENGINE_OVERRIDES)
+    tensors = random_tensors(manifest, seed=0, std=0.02, dtype=torch.bfloat16, device="cuda:0")
+    runner = ModelRunner(cfg, tensors, cf.EngineConfig(**fields))
+    del tensors
+    return cfg, LLM(runner)
+
+
+def side_by_side_roofline(arch, rs, n, batch, peaks, prefill, decode):
+    """The kernels of both designs against their rooflines: algorithmic bytes (or FLOPs) of all their launches in one step over
+    the measured time, as a fraction of the measured copy bandwidth (or the measured bfloat16 product rate)."""
+    ls = LOMOPEL_SIZES[rs["lomopel"]]
+    at, lat, m, W, new = ls["attn"], ROTEPEL_SIZES[ls["llama"]]["latent"], rs["moe"], ls["width"], arch == "robuvik"
+    runs = robuvik_runs()
+    layers, nA, nL = len(runs), runs.count("A"), runs.count("L")
+    out = {}
+
+    def add(names, label, phase, totals, nbytes=None, flops=None):
+        ms = sum(t for op, _, t in totals if op in names)
+        if ms <= 0:
+            return
+        e = {"ms": round(ms, 4)}
+        if nbytes is not None:
+            e["gbs"] = round(nbytes / ms / 1e6, 1)
+            e["of_measured_hbm"] = round(nbytes / ms / 1e6 / peaks["hbm_gbs"], 4)
+        if flops is not None:
+            e["tflops"] = round(flops / ms / 1e9, 2)
+            e["of_measured_bf16"] = round(flops / ms / 1e9 / peaks["bf16_tflops"], 4)
+        out[f"{phase}:{label}"] = e
+    qd, kd, vd = at["heads"] * at["dim"], at["kv_heads"] * at["dim"], at["kv_heads"] * at["vdim"]
+    lq, lv = lat["heads"] * (lat["dim"] + lat["rot_dim"]), lat["heads"] * lat["vdim"]
+    for phase, rows, totals in (("prefill", n, prefill), ("decode", batch, decode)):
+        add(("embed", "embed_pairs"), "embedding", phase, totals, nbytes=rows * W * (2 + 4 + (2 + 4 if new else 0)))
+        # norms: the float32 residual read and written, the sub-layers' results read, the rounded rows written. One norm adds two
+        # results here; there a norm in front (read, write) and one behind (read a result, read and write the residual) of each
+        add(("add_rmsnorm", "layernorm_rows", "layernorm_add"), "norms", phase, totals,
+            nbytes=layers * rows * W * (2 * 2 + 2 * 4 + 2) if new else 2 * layers * rows * W * ((4 + 2) + (2 + 2 * 4)))
+        keys = sum(min(i + 1, rs["window"]) for i in range(n)) if phase == "prefill" else batch * min(n + 3, rs["window"])
+        add(("flex_attention", "attn_prefill_mma_any", "attn_prefill_mma", "attn_decode_mma"), "attention", phase, totals,
+            nbytes=nA * keys * (kd + vd) * 2 if phase == "decode" else None, flops=nA * keys * at["heads"] * 2 * (at["dim"] + at["vdim"]))
+        add(("flex_prep",), "flex_prep", phase, totals, nbytes=nA * rows * 2 * (qd + kd + vd) * 2)
+        lkeys = sum(i + 1 for i in range(n)) if phase == "prefill" else batch * (n + 3)
+        add(("latent_attend", "latent_attend_tc"), "latent attention", phase, totals,
+            nbytes=nL * lkeys * (lat["kv_rank"] + lat["rot_dim"]) * 2 if phase == "decode" else None,
+            flops=nL * lkeys * lat["heads"] * 2 * (2 * lat["kv_rank"] + lat["rot_dim"]))
+        # the latent and the rotated key part read and written, the rotated query parts read and written (float32); the query
+        # latent read and written, the gate and the values read and the gated values written
+        add(("latent_prep",), "latent_prep", phase, totals, nbytes=nL * rows * (
+            2 * (lat["kv_rank"] + lat["rot_dim"]) * 2 + lat["heads"] * lat["rot_dim"] * (2 + 4) + (2 * rs["q_rank"] * 2 if new else 0)))
+        add(("latent_gate",), "latent_gate", phase, totals, nbytes=nL * rows * lv * 3 * 2)
+        P, used = rows * m["top"], min(m["experts"], rows * m["top"])
+        add(("moe_gate_up", "moe_down"), "expert products", phase, totals,
+            nbytes=layers * (used * 3 * m["ff"] * W * 2 + P * (W * 2 + 2 * m["ff"] * 2 + W * 4)), flops=layers * P * 3 * 2 * m["ff"] * W)
+        add(("moe_route", "moe_align", "moe_combine"), "election, order, sum", phase, totals,
+            nbytes=layers * (rows * W * 2 + m["experts"] * W * 4 + P * W * 4 + 2 * rows * W * 2))
+        add(("glu", "glu_clamped"), "shared expert's gate", phase, totals, nbytes=layers * rows * 3 * m["shared_ff"] * 2)
+    return out
+
+
+def activation_pair(ls, n):
+    """The dense feed-forward's relu squared beside the engine's other activation without a gate (xIELU), one call each on
+    [n, 4 width] bfloat16: ms and the fraction of the bytes' time that is (read and written once)."""
+    import torch
+    from vllm_oxide_b200 import kernels
+    bufs = [torch.randn(n, 4 * ls["width"], device="cuda:0").bfloat16() for _ in range(16)]           # more than the L2 holds
+    params = torch.tensor([0.8, 1.1], device="cuda:0")
+    out = {}
+    for kind, p in (("relu2", None), ("xielu", params)):
+        for b in bufs[:3]:
+            kernels.activation(b, b, kind, p)
+        e = [torch.cuda.Event(enable_timing=True) for _ in range(2)]
+        torch.cuda.synchronize()
+        e[0].record()
+        for b in bufs:
+            kernels.activation(b, b, kind, p)
+        e[1].record()
+        torch.cuda.synchronize()
+        ms = e[0].elapsed_time(e[1]) / len(bufs)
+        out[kind] = {"ms": round(ms, 4), "gbs": round(bufs[0].numel() * 4 / ms / 1e6, 1)}
+    return out
+
+
+def robuvik_compare(a):
+    """Prefill and decode of the Robuvik design beside Pironex layers of the same kinds, width, layer count, heads and experts; one
+    JSON line. Device-timed like the benchmark's own points: one step of 2,048 prompt tokens (median of 5 after 3), decode steps
+    replayed from CUDA graphs (`--steps` steps a region, median region)."""
+    import torch
+    peaks = load_peaks()
+    n, B = 2048, a.batch
+    gen = a.warmup + max(a.steps, MAX_TIMED_STEPS) + 64
+    sampler = ClockSampler()
+    sampler.start()
+    points = []
+    for key in a.robuvik.split(","):
+        rs = ROBUVIK_SIZES[key]
+        point = {"sizes": key, "layers": len(robuvik_runs()), "prompt_len": n, "batch": B, "activations": activation_pair(LOMOPEL_SIZES[rs["lomopel"]], n)}
+        for arch in ("robuvik", "pironex"):
+            cfg, llm = make_side_by_side_engine(arch, rs, B, n + gen, 8192)
+            g = torch.Generator().manual_seed(1)
+            prompts = [torch.randint(0, cfg.vocab, (n,), generator=g).tolist() for _ in range(B)]
+            ms_prefill = timed_prefill(llm, prompts[0], n)
+            ms_step, ctx_tokens, launches, regions = decode_device(llm, prompts, B, a.steps, a.warmup, n, gen)
+            prefill, decode = op_profile(llm, prompts, n, B)
+            point[arch] = {"prefill_tok_s": round(n / ms_prefill * 1e3, 1), "prefill_ms": round(ms_prefill, 3),
+                           "decode_tok_s": round(B / ms_step * 1e3, 1), "decode_ms_per_step": round(ms_step, 4),
+                           "decode_hbm_frac_of_measured": round(llm.runner.step_read_bytes(int(ctx_tokens)) / ms_step / 1e6 / peaks["hbm_gbs"], 3),
+                           "launches_per_decode_step": launches // a.steps,
+                           "ops_prefill_ms": {op: round(t, 4) for op, _, t in prefill}, "ops_decode_ms": {op: round(t, 4) for op, _, t in decode},
+                           "kernels": side_by_side_roofline(arch, rs, n, B, peaks, prefill, decode)}
+            free_engine(llm)
+            del llm
+        points.append(point)
+    clocks = sampler.stop()
+    print(json.dumps({"metric": "Robuvik beside Pironex (latent attention and attention in a window, routed experts with a shared one) at equal "
+                                "width, layer count, heads and experts: prefill and decode tok/s",
+                      "dtype": "bf16", "data": "synthetic", "peaks": peaks, "points": points, "clocks": clocks, "run": run_record()}))
+    return 0
+
+
 def main():
     if "--kernel" in sys.argv[1:]:
         return kernel_case(sys.argv[1:])
@@ -1368,6 +1532,9 @@ def main():
     ap.add_argument("--fanopel", default=None, metavar="SIZES", const="1b,3b", nargs="?",
                     help="instead of the benchmark's line: the Fanopel design beside Bufulorn at equal sizes (1b, 3b or both), "
                          "prefill and decode, with the time and roofline fraction of every kernel")
+    ap.add_argument("--robuvik", default=None, metavar="SIZES", const="1b,3b", nargs="?",
+                    help="instead of the benchmark's line: the Robuvik design beside Pironex at equal sizes (1b, 3b or both), "
+                         "prefill and decode")
     ap.add_argument("--tuning", action="append", default=[], metavar="FIELD=VALUE",
                     help="set a field of vllm_oxide_b200.tuning.TUNING (experiments)")
     ap.add_argument("--fold-rows", type=int, default=None, metavar="R",
@@ -1403,6 +1570,8 @@ def main():
         return pironex_compare(a)
     if a.fanopel:
         return fanopel_compare(a)
+    if a.robuvik:
+        return robuvik_compare(a)
     prompt_len, gen_len = a.prompt_len, a.gen_len
     max_b = max(a.batch, 1 if (a.no_points or a.serve or a.timeline) else 64)
     if a.serve:
