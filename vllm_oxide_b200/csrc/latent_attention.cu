@@ -281,30 +281,37 @@ latent_attend_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, cons
 }
 
 // The shares of a row's keys put together, in share order: out = sum_z acc_z e^(m_z - M) / sum_z l_z e^(m_z - M).
-// Launch: one warp per (row, head).
+// Launch: one block of 128 threads per (row, head), at most VOB_LATENT_SPLITS shares.
+#define VOB_LATENT_SPLITS 64
 template <typename TO>
-__global__ void __launch_bounds__(32)
+__global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part, const int* __restrict__ positions, int H, int L, int splits,
                     TO* __restrict__ out, long o_ts, long o_hs) {
     pdl_launch_dependents();
     pdl_wait(47);
-    const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x;
+    const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     TO* orow = out + (size_t)t * o_ts + (size_t)h * o_hs;
     const float* p = part + ((size_t)t * H + h) * splits * (L + 2);
     if (positions[t] < 0) {
-        for (int i = lane; i < L; i += 32) st_f(orow + i, 0.f);
+        for (int i = tid; i < L; i += blockDim.x) st_f(orow + i, 0.f);
         return;
     }
+    __shared__ float m[VOB_LATENT_SPLITS], sum[VOB_LATENT_SPLITS], wgt[VOB_LATENT_SPLITS];
+    if (tid < splits) { m[tid] = p[(size_t)tid * (L + 2)]; sum[tid] = p[(size_t)tid * (L + 2) + 1]; }
+    __syncthreads();
     float M = -INFINITY;
-    for (int z = 0; z < splits; ++z) M = fmaxf(M, p[(size_t)z * (L + 2)]);
+    for (int z = 0; z < splits; ++z) M = fmaxf(M, m[z]);
+    if (tid < splits) wgt[tid] = sum[tid] > 0.f ? expf(m[tid] - M) : 0.f;      // 0: a share without keys, nothing of it is read
+    __syncthreads();
     float l = 0.f;
-    for (int z = 0; z < splits; ++z) l = fmaf(p[(size_t)z * (L + 2) + 1], expf(p[(size_t)z * (L + 2)] - M), l);
+    for (int z = 0; z < splits; ++z) l = fmaf(sum[z], wgt[z], l);
     const float inv = 1.0f / l;
-    for (int i = lane; i < L; i += 32) {
+    for (int i = tid; i < L; i += blockDim.x) {
         float a = 0.f;
+#pragma unroll 8
         for (int z = 0; z < splits; ++z) {
-            const float* pz = p + (size_t)z * (L + 2);
-            if (pz[1] > 0.f) a = fmaf(pz[2 + i], expf(pz[0] - M), a);
+            const float v = wgt[z] > 0.f ? p[(size_t)z * (L + 2) + 2 + i] : 0.f;
+            a = fmaf(v, wgt[z], a);
         }
         st_f(orow + i, a * inv);
     }
@@ -317,7 +324,7 @@ VOB_EXPORT int vob_latent_attend(const float* q_lat, long q_ts, long q_hs, const
     if (T <= 0) return 0;
     if (window < 0) return VOB_ERR_BAD_ARG;
     if (H <= 0 || L <= 0 || R <= 0 || page_size <= 0 || max_pages <= 0 || cache_code != out_code) return VOB_ERR_BAD_ARG;
-    if (splits < 1 || splits > 65535 || (splits > 1 && !part) || H > 65535) return VOB_ERR_BAD_ARG;
+    if (splits < 1 || splits > VOB_LATENT_SPLITS || (splits > 1 && !part) || H > 65535) return VOB_ERR_BAD_ARG;
     if (L > 1024 || R > 128) return VOB_ERR_UNSUPPORTED;
     const int warps = H < 8 ? H : 8;
     const int W = L + R;
@@ -338,7 +345,7 @@ VOB_EXPORT int vob_latent_attend(const float* q_lat, long q_ts, long q_hs, const
         else if (nl <= 16) { VOB_LA(16, TC); } \
         else { VOB_LA(32, TC); }               \
         if (status == 0 && splits > 1)         \
-            status = vob_launch(latent_merge_kernel<TC>, dim3(T, H), dim3(32), 0, stream, (const float*)part, positions, H, L, splits, \
+            status = vob_launch(latent_merge_kernel<TC>, dim3(T, H), dim3(128), 0, stream, (const float*)part, positions, H, L, splits, \
                                 (TC*)out, o_ts, o_hs);                                                                          \
     } while (0)
     if (cache_code == VOB_F32) VOB_LA_N(float);
@@ -359,6 +366,10 @@ VOB_EXPORT int vob_latent_attend(const float* q_lat, long q_ts, long q_hs, const
 // O (float32) never leave the registers. Needs L and R multiples of 16. Rows are a request's seq_starts[s] + 16
 // * tile ..; their positions are consecutive, so the tile's last row bounds the keys and every row masks what
 // lies behind its own position.
+//
+// Steps of single tokens run the same kernel with HEADS: the 16 rows of a tile are 16 heads of ONE token (they share its
+// keys), the warps of a block share out the latent columns, and `splits` blocks share a token's keys in whole tiles; with more
+// than one share each leaves (max, sum, weighted sum) per head in `part` for latent_merge_kernel, as latent_attend_kernel does.
 // ---------------------------------------------------------------------------------------------
 #define VOB_LTC_BN 32
 #define VOB_LTC_PRE 10        // 16-byte pieces of the next key tile a thread holds ahead (the rest of a tile is copied when it is due)
@@ -381,23 +392,39 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 }
 
 // NT16: groups of 16 latent columns a warp owns at most (its O accumulator is NT16 * 8 registers).
-template <int NT16>
+template <int NT16, bool HEADS>
 __global__ void __launch_bounds__(256, 1)
 latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, const float* __restrict__ q_rot,
                         const __nv_bfloat16* __restrict__ lat, const __nv_bfloat16* __restrict__ kr, const int* __restrict__ block_tables,
                         int max_pages, const int* __restrict__ seq_starts, const int* __restrict__ positions, int page_size, int H, int L,
-                        int R, float scale, __nv_bfloat16* __restrict__ out, long o_ts, long o_hs, int WPH, int colsw, int window) {
+                        int R, float scale, __nv_bfloat16* __restrict__ out, long o_ts, long o_hs, int WPH, int colsw, int window,
+                        const int* __restrict__ row_seq, int splits, float* __restrict__ part) {
     constexpr int BN = VOB_LTC_BN;
     pdl_launch_dependents();
     pdl_wait(48);
-    const int s = blockIdx.z, NW = blockDim.x >> 5, HB = NW / WPH;
+    const int NW = blockDim.x >> 5, HB = NW / WPH;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int hh = warp / WPH, wsub = warp - hh * WPH;
-    const int h = blockIdx.y * HB + hh;
+    const int h = (blockIdx.y * HB + hh) * (HEADS ? 16 : 1);       // this warp's head, or the first of its 16 heads
     const bool head = h < H;
-    const int r0 = seq_starts[s] + blockIdx.x * 16, r1 = seq_starts[s + 1];
-    if (r0 >= r1) return;
-    const int nrows = min(16, r1 - r0);
+    int s, r0, nrows;
+    if (HEADS) {
+        r0 = blockIdx.x;
+        s = row_seq[r0];
+        nrows = max(0, min(16, H - h));
+        if (positions[r0] < 0) {                                   // padding: nothing to see
+            for (int i = lane; head && wsub == 0 && i < nrows * L; i += 32) {
+                if (splits == 1) out[(size_t)r0 * o_ts + (size_t)(h + i / L) * o_hs + i % L] = __float2bfloat16_rn(0.f);
+            }
+            return;                                                // (the merge writes zeros for such rows by itself)
+        }
+    } else {
+        s = blockIdx.z;
+        const int r1 = seq_starts[s + 1];
+        r0 = seq_starts[s] + blockIdx.x * 16;
+        if (r0 >= r1) return;
+        nrows = min(16, r1 - r0);
+    }
     const int D = L + R, DP = D + 8;
     extern __shared__ __align__(128) unsigned char ltc_smem[];
     __nv_bfloat16* Kt = reinterpret_cast<__nv_bfloat16*>(ltc_smem);                               // [BN][DP]
@@ -405,16 +432,24 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
     for (int e = lane + 32 * wsub; e < 16 * D; e += 32 * WPH) {
         const int i = e / D, c = e - i * D;
         float v = 0.f;
-        if (head && i < nrows)
-            v = c < L ? q_lat[(size_t)(r0 + i) * q_ts + (size_t)h * q_hs + c] : q_rot[((size_t)(r0 + i) * H + h) * R + (c - L)];
+        if (head && i < nrows) {
+            const size_t tok = HEADS ? r0 : r0 + i, hd = HEADS ? h + i : h;
+            v = c < L ? q_lat[tok * q_ts + hd * q_hs + c] : q_rot[(tok * H + hd) * R + (c - L)];
+        }
         Q[i * DP + c] = __float2bfloat16_rn(v);
     }
-    const int pos0 = positions[r0], pos_hi = pos0 + nrows - 1;
+    const int pos0 = positions[r0];
+    int pos_hi = HEADS ? pos0 : pos0 + nrows - 1;
     // with a window a row sees only its last `window` keys: the tile's first row bounds the keys from below (pages before
     // that may have been given back and are never addressed), and the walk starts at the tile of BN keys that holds it, so
     // that a row's keys fall into the same tiles however the prompt was cut
     const int key_lo = window > 0 ? max(0, pos0 + 1 - window) : 0;
-    const int k_start = key_lo / BN * BN;
+    int k_start = key_lo / BN * BN;
+    if (HEADS) {                                   // this block's share of the tiles
+        const int tiles = (pos0 - k_start) / BN + 1, per = (tiles + splits - 1) / splits;
+        k_start += (int)blockIdx.z * per * BN;
+        pos_hi = min(pos0, k_start + per * BN - 1);
+    }
     const int* table = block_tables + (size_t)s * max_pages;
     // this warp's latent columns, in groups of 16
     const int col0 = wsub * colsw;
@@ -425,6 +460,7 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
     for (int i = 0; i < NT16 * 2; ++i) { o[i][0] = 0.f; o[i][1] = 0.f; o[i][2] = 0.f; o[i][3] = 0.f; }
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;       // l: this thread's share of the row sums
     const bool row0 = g < nrows, row1 = g + 8 < nrows;
+    const int p0 = HEADS ? pos0 : pos0 + g, p1 = HEADS ? pos0 : pos0 + g + 8;       // these rows' positions
     const int lat_chunks = L / 8, kr_chunks = R / 8;            // 16-byte pieces of a key
     // The key tile as a list of 16-byte pieces, BN keys x (lat_chunks + kr_chunks) pieces: thread t takes pieces
     // t, t + threads, ... The NEXT tile's pieces are fetched into registers while this tile is worked on.
@@ -497,8 +533,8 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = k0 + 8 * j + 2 * t4 + e;
-                const bool in0 = key <= pos0 + g && (window <= 0 || key > pos0 + g - window);
-                const bool in1 = key <= pos0 + g + 8 && (window <= 0 || key > pos0 + g + 8 - window);
+                const bool in0 = key <= p0 && (window <= 0 || key > p0 - window);
+                const bool in1 = key <= p1 && (window <= 0 || key > p1 - window);
                 sc[j][e] = (row0 && in0) ? sc[j][e] * scale : -INFINITY;
                 sc[j][2 + e] = (row1 && in1) ? sc[j][2 + e] * scale : -INFINITY;
                 mx0 = fmaxf(mx0, sc[j][e]);
@@ -557,15 +593,32 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
     l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    if (HEADS && splits > 1) {                     // (maximum, sum, weighted sum) of this share, per head
+        float* pr0 = part + (((size_t)r0 * H + h + g) * splits + blockIdx.z) * (L + 2);
+        float* pr1 = pr0 + (size_t)8 * splits * (L + 2);
+        if (wsub == 0 && t4 == 0) {
+            if (row0) { pr0[0] = m0; pr0[1] = l0; }
+            if (row1) { pr1[0] = m1; pr1[1] = l1; }
+        }
+#pragma unroll
+        for (int n = 0; n < NT16 * 2; ++n) {
+            if (n < 2 * n16) {
+                const int c = 2 + col0 + 8 * n + 2 * t4;          // L + 2 is even: pairs of columns are 8-byte aligned
+                if (row0) *reinterpret_cast<float2*>(pr0 + c) = make_float2(o[n][0], o[n][1]);
+                if (row1) *reinterpret_cast<float2*>(pr1 + c) = make_float2(o[n][2], o[n][3]);
+            }
+        }
+        return;
+    }
     const float inv0 = 1.0f / l0, inv1 = 1.0f / l1;
+    __nv_bfloat16* o0 = out + (size_t)(HEADS ? r0 : r0 + g) * o_ts + (size_t)(HEADS ? h + g : h) * o_hs;
+    __nv_bfloat16* o1 = o0 + (HEADS ? 8 * o_hs : 8 * o_ts);
 #pragma unroll
     for (int n = 0; n < NT16 * 2; ++n) {
         if (n < 2 * n16) {
             const int c = col0 + 8 * n + 2 * t4;
-            if (row0)
-                *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(r0 + g) * o_ts + (size_t)h * o_hs + c) = __floats2bfloat162_rn(o[n][0] * inv0, o[n][1] * inv0);
-            if (row1)
-                *reinterpret_cast<__nv_bfloat162*>(out + (size_t)(r0 + g + 8) * o_ts + (size_t)h * o_hs + c) = __floats2bfloat162_rn(o[n][2] * inv1, o[n][3] * inv1);
+            if (row0) *reinterpret_cast<__nv_bfloat162*>(o0 + c) = __floats2bfloat162_rn(o[n][0] * inv0, o[n][1] * inv0);
+            if (row1) *reinterpret_cast<__nv_bfloat162*>(o1 + c) = __floats2bfloat162_rn(o[n][2] * inv1, o[n][3] * inv1);
         }
     }
 }
@@ -607,14 +660,72 @@ VOB_EXPORT int vob_latent_attend_tc(const float* q_lat, long q_ts, long q_hs, co
     dim3 grid((max_new + 15) / 16, (H + hb - 1) / hb, seqs), block(32 * hb * wph);
 #define VOB_LTC(N)                                                                                                              \
     do {                                                                                                                        \
-        cudaError_t e = cudaFuncSetAttribute(latent_attend_tc_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        cudaError_t e = cudaFuncSetAttribute(latent_attend_tc_kernel<N, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         if (e != cudaSuccess) return (int)e;                                                                                    \
-        return vob_launch(latent_attend_tc_kernel<N>, grid, block, smem, stream, q_lat, q_ts, q_hs, q_rot, (const __nv_bfloat16*)lat, \
+        return vob_launch(latent_attend_tc_kernel<N, false>, grid, block, smem, stream, q_lat, q_ts, q_hs, q_rot, (const __nv_bfloat16*)lat, \
                           (const __nv_bfloat16*)kr, block_tables, max_pages, seq_starts, positions, page_size, H, L, R, scale,  \
-                          (__nv_bfloat16*)out, o_ts, o_hs, wph, colsw, window);                                                 \
+                          (__nv_bfloat16*)out, o_ts, o_hs, wph, colsw, window, nullptr, 1, nullptr);                            \
     } while (0)
     if (colsw <= 64) VOB_LTC(4);
     if (colsw <= 128) VOB_LTC(8);
     VOB_LTC(16);
 #undef VOB_LTC
+}
+
+
+// The shape of a block in steps of single tokens: groups of 16 heads per block, and the warps that share a group's latent columns.
+static int ltc_heads_shape(int H, int L, int R, int* wph, int* colsw) {
+    if (L % 16 || R % 16 || L <= 0 || R <= 0 || L > 1024 || H <= 0) return 0;
+    const size_t DP = (size_t)L + R + 8;
+    const size_t shared = (size_t)VOB_LTC_BN * DP * 2, per_group = 16 * DP * 2;
+    const int least = (L + 255) / 256, groups = (H + 15) / 16;
+    int hb = groups < 4 ? groups : 4;
+    while (hb > 1 && (shared + hb * per_group > 100 * 1024 || hb * least > 8)) --hb;
+    if (shared + hb * per_group > 200 * 1024) return 0;
+    int w = 8 / hb;
+    if (w > L / 16) w = L / 16;
+    *wph = w < least ? least : w;
+    *colsw = ((L / 16 + *wph - 1) / *wph) * 16;
+    return hb;
+}
+
+// Groups of 16 heads a block takes, 0: the sizes do not fit.
+VOB_EXPORT int vob_latent_decode_tc_groups(int H, int L, int R) {
+    int wph, colsw;
+    return ltc_heads_shape(H, L, R, &wph, &colsw);
+}
+
+// Steps of single tokens: row t is one token of request row_seq[t]. Operands as for vob_latent_attend (bfloat16 caches and out
+// only; out's strides even, part 8-byte aligned).
+VOB_EXPORT int vob_latent_decode_tc(const float* q_lat, long q_ts, long q_hs, const float* q_rot, const void* lat, const void* kr,
+                                    const int* block_tables, int max_pages, const int* row_seq, const int* positions, int page_size, int T,
+                                    int H, int L, int R, float scale, void* out, long o_ts, long o_hs, int splits, float* part, int window,
+                                    cudaStream_t stream) {
+    if (T <= 0) return 0;
+    int wph, colsw;
+    const int hb = ltc_heads_shape(H, L, R, &wph, &colsw);
+    if (hb <= 0) return VOB_ERR_UNSUPPORTED;
+    if (window < 0 || page_size <= 0 || max_pages <= 0 || splits < 1 || splits > VOB_LATENT_SPLITS || (splits > 1 && !part) || H > 65535
+        || (o_ts & 1) || (o_hs & 1) || ((uintptr_t)out & 3) || ((uintptr_t)part & 7))
+        return VOB_ERR_BAD_ARG;
+    const size_t DP = (size_t)L + R + 8;
+    const size_t smem = (size_t)VOB_LTC_BN * DP * 2 + (size_t)hb * 16 * DP * 2;
+    dim3 grid(T, ((H + 15) / 16 + hb - 1) / hb, splits), block(32 * hb * wph);
+    int status = VOB_ERR_BAD_ARG;
+#define VOB_LTCH(N)                                                                                                                   \
+    do {                                                                                                                              \
+        cudaError_t e = cudaFuncSetAttribute(latent_attend_tc_kernel<N, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (e != cudaSuccess) return (int)e;                                                                                          \
+        status = vob_launch(latent_attend_tc_kernel<N, true>, grid, block, smem, stream, q_lat, q_ts, q_hs, q_rot, (const __nv_bfloat16*)lat, \
+                            (const __nv_bfloat16*)kr, block_tables, max_pages, nullptr, positions, page_size, H, L, R, scale,          \
+                            (__nv_bfloat16*)out, o_ts, o_hs, wph, colsw, window, row_seq, splits, part);                              \
+    } while (0)
+    if (colsw <= 64) VOB_LTCH(4);
+    else if (colsw <= 128) VOB_LTCH(8);
+    else VOB_LTCH(16);
+#undef VOB_LTCH
+    if (status == 0 && splits > 1)
+        status = vob_launch(latent_merge_kernel<__nv_bfloat16>, dim3(T, H), dim3(128), 0, stream, (const float*)part, positions, H, L, splits,
+                            (__nv_bfloat16*)out, o_ts, o_hs);
+    return status;
 }

@@ -1633,6 +1633,50 @@ def latent_attend_tc(q_lat: torch.Tensor, q_rot: torch.Tensor, lat: torch.Tensor
              out.stride(1), int(window), _stream()), op)
 
 
+LATENT_MAX_SPLITS = 64       # blocks a row's keys are shared over at most
+
+
+def latent_decode_tc_groups(heads: int, rank: int, rot: int) -> int:
+    """Groups of 16 heads a block of the tensor-core kernel for single tokens takes (bfloat16 only); 0: it does not take these sizes."""
+    f = _fn("latent_attention", "vob_latent_decode_tc_groups", [_I, _I, _I])
+    return int(f(int(heads), int(rank), int(rot)))
+
+
+@_timed
+def latent_decode_tc(q_lat: torch.Tensor, q_rot: torch.Tensor, lat: torch.Tensor, kr: torch.Tensor, block_tables: torch.Tensor,
+                     row_seq: torch.Tensor, positions: torch.Tensor, scale: float, out: torch.Tensor, splits: int = 1,
+                     partials: Optional[torch.Tensor] = None, window: int = 0) -> None:
+    """`latent_attend` in bfloat16 on the tensor cores, 16 heads of a row at a time: for steps of single tokens, whose heads all
+    read the same keys. Same operands and result (q_lat is rounded to bfloat16, as for prompt portions)."""
+    op = "latent_decode_tc"
+    _cuda(op, q_lat, q_rot, lat, kr, block_tables, row_seq, positions, out, partials)
+    if q_lat.dim() != 3 or q_lat.dtype != torch.float32 or q_lat.stride(2) != 1:
+        raise ShapeError(op, f"q_lat must be float32 [T, heads, rank] with unit inner stride, got {q_lat.dtype} {list(q_lat.shape)}")
+    T, H, L = q_lat.shape
+    R = kr.shape[3]
+    if lat.dtype != torch.bfloat16 or kr.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or out.shape != (T, H, L) or out.stride(2) != 1:
+        raise ShapeError(op, f"bfloat16 caches and a bfloat16 out of [{T}, {H}, {L}] with unit inner stride are needed, got {out.dtype} {list(out.shape)}")
+    if q_rot.shape != (T, H, R) or q_rot.dtype != torch.float32 or not q_rot.is_contiguous():
+        raise ShapeError(op, f"q_rot must be contiguous float32 [{T}, {H}, {R}], got {q_rot.dtype} {list(q_rot.shape)}")
+    if lat.dim() != 4 or lat.shape[1] != 1 or lat.shape[3] != L or kr.shape[:3] != lat.shape[:3] or not lat.is_contiguous() or not kr.is_contiguous():
+        raise ShapeError(op, f"lat [pages, 1, page, {L}] and kr [pages, 1, page, {R}] are needed, got {list(lat.shape)} and {list(kr.shape)}")
+    if not latent_decode_tc_groups(H, L, R):
+        raise ShapeError(op, f"a latent of {L} with a rotated part of {R} is not supported (multiples of 16 that fit shared memory)")
+    if block_tables.dtype != torch.int32 or block_tables.dim() != 2 or not block_tables.is_contiguous():
+        raise ShapeError(op, "block_tables must be contiguous int32 [requests, max_pages]")
+    _int32_vec(row_seq, T, op, "row_seq")
+    _int32_vec(positions, T, op, "positions")
+    splits = int(splits)
+    if not 1 <= splits <= LATENT_MAX_SPLITS:
+        raise ShapeError(op, f"splits must be 1..{LATENT_MAX_SPLITS}, got {splits}")
+    if splits > 1 and (partials is None or partials.dtype != torch.float32 or not partials.is_contiguous() or partials.numel() < T * H * splits * (L + 2)):
+        raise ShapeError(op, f"{splits} splits need contiguous float32 partials of {T * H * splits * (L + 2)} elements")
+    f = _fn("latent_attention", "vob_latent_decode_tc", [_P, _L, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _L, _L, _I, _P, _I, _P])
+    _check(f(_ptr(q_lat), q_lat.stride(0), q_lat.stride(1), _ptr(q_rot), _ptr(lat), _ptr(kr), _ptr(block_tables), block_tables.shape[1],
+             _ptr(row_seq), _ptr(positions), lat.shape[2], T, H, L, R, float(scale), _ptr(out), out.stride(0), out.stride(1), splits,
+             _ptr(partials) if splits > 1 else _P(0), int(window), _stream()), op, 2 if splits > 1 else 1)
+
+
 # ------------------------------------------------------------------------------------ attention with options
 def _kv_caches(op, kcache, vcache, kv_heads, dim, vdim, dtype):
     for name, c, w in (("kcache", kcache, dim), ("vcache", vcache, vdim)):

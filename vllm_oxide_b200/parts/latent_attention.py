@@ -83,6 +83,7 @@ class LatentAttention(Mixer):
         self.splits = None        # a number forces so many blocks per row's keys (tests)
         self.tensor_cores = True  # False: prompt portions go through the float32 kernel too (tests)
         self._tc_ok = None
+        self._groups = None       # groups of 16 heads a block of the kernel for single tokens takes
 
     def key_splits(self, rows: int) -> int:
         """Blocks that share a row's keys: steps of few rows would leave most of the GPU idle with one
@@ -91,6 +92,18 @@ class LatentAttention(Mixer):
             return int(self.splits)
         blocks = rows * -(-self.H // 8)
         return max(1, min(32, 2 * self.num_sms // blocks)) if blocks < self.num_sms else 1
+
+    def single_splits(self, rows: int) -> int:
+        """The same for the tensor-core kernel of single tokens (0: it does not take this layer's sizes): about two blocks an SM."""
+        if self._groups is None:
+            ok = self.dtype == torch.bfloat16 and self.batched and self.tensor_cores
+            self._groups = kernels.latent_decode_tc_groups(self.H, self.L, self.R) if ok else 0
+        if not self._groups or not self.tensor_cores or not self.batched:
+            return 0
+        if self.splits is not None:
+            return int(self.splits)
+        blocks = rows * -(-self.H // (16 * self._groups))
+        return max(1, min(kernels.LATENT_MAX_SPLITS, 2 * self.num_sms // blocks))
 
     def cache_spec(self) -> Optional[CacheSpec]:
         kind = "window" if self.window else "full"
@@ -106,6 +119,9 @@ class LatentAttention(Mixer):
         if self.splits is None:     # the most any step of at most `rows` rows takes: below one block per SM every row has 32 shares
             few = min(rows, self.num_sms // -(-H // 8))
             parts = max(parts, aligned(few * H * 32 * (self.L + 2) * 4))
+            if self.single_splits(1):         # rows times shares is at most two blocks an SM, and at most the most shares a row can have
+                most = min(rows * kernels.LATENT_MAX_SPLITS, 2 * self.num_sms // -(-H // (16 * self._groups)))
+                parts = max(parts, aligned(most * H * (self.L + 2) * 4))
         low = aligned(rows * self.Q * es) + aligned(rows * H * (self.D + self.R) * es) if self.Q else 0
         return (low + aligned(rows * self.w_in.shape[0] * es) + aligned(rows * H * self.R * 4) + aligned(rows * H * self.L * 4)
                 + aligned(rows * H * self.L * es) + 2 * aligned(rows * H * self.V * es) + parts)
@@ -136,7 +152,8 @@ class LatentAttention(Mixer):
         q_heads = q.view(T, H, D + R)[:, :, :D]                                    # [T, H, D], strided
         gate = proj[:, self.gate_off:self.gate_off + H * V] if self.gated else None
         bt = ctx.block_tables[cache.group]
-        splits = self.key_splits(T)
+        single = ctx.decode_only and self.single_splits(T)
+        splits = self.single_splits(T) if single else self.key_splits(T)
         partials = ctx.alloc((T * H * splits * (L + 2),), torch.float32) if splits > 1 else None
         if self.dtype == torch.bfloat16 and self.batched:
             # head-major buffers, so that each of the two per-head products is one batched product
@@ -149,6 +166,9 @@ class LatentAttention(Mixer):
                 # prompt portions: scores and the weighted sum on the tensor cores, 16 tokens of a request at a time
                 kernels.latent_attend_tc(q_lat.transpose(0, 1), q_rot, lat, kr, bt, ctx.seq_starts, ctx.positions, ctx.seqs,
                                          min(ctx.max_new, T), self.scale, out_lat.transpose(0, 1), self.window)
+            elif single:
+                kernels.latent_decode_tc(q_lat.transpose(0, 1), q_rot, lat, kr, bt, ctx.row_seq, ctx.positions, self.scale,
+                                         out_lat.transpose(0, 1), splits, partials, self.window)
             else:
                 kernels.latent_attend(q_lat.transpose(0, 1), q_rot, lat, kr, bt, ctx.row_seq, ctx.positions, self.scale,
                                       out_lat.transpose(0, 1), splits, partials, self.window)
