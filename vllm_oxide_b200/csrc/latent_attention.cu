@@ -26,7 +26,7 @@ VOB_PDL_SWITCH(latent_attention)
 // Cosine and sine are both multiplied by `mag`. Rows with position < 0 write nothing (their q_rot is zero); a slot < 0 writes
 // no cache. `q` null: no queries here; `slots` null: no cache write; `low` [T, ld_low] (Q columns) null: no query latent, else
 // low_out [T, Q] = low_w * low / sqrt(mean(low^2) + eps), every row.
-// Launch: one block of 128 threads per token.
+// Launch: grid (tokens, blocks that share a token's queries), 128 threads; the first block of a token does the rest.
 template <typename T, typename TC>
 __global__ void __launch_bounds__(128)
 latent_prep_kernel(const T* __restrict__ q, long ld_q, int H, int D, int R, const T* __restrict__ down_p, long ld, int L,
@@ -42,20 +42,23 @@ latent_prep_kernel(const T* __restrict__ q, long ld_q, int H, int D, int R, cons
     if (q) {
         const T* row = q + (size_t)t * ld_q;
         float* qo = q_rot + (size_t)t * H * R;
-        for (int e = tid; e < H * R; e += blockDim.x) {
-            float v = 0.f;
+        // a thread takes a pair of features: its angle's cosine and sine serve both
+        for (int e = blockIdx.y * blockDim.x + tid; e < H * half; e += blockDim.x * gridDim.y) {
+            const int h = e / half, i = e - h * half;
+            float u = 0.f, v = 0.f;
             if (pos >= 0) {
-                const int h = e / R, f = e - h * R;
-                const int i = f < half ? f : f - half;
                 const float ang = (float)pos * inv_freq[i];
                 const float cs = cosf(ang) * mag, sn = sinf(ang) * mag;
                 const T* qh = row + (size_t)h * (D + R) + D;
                 const float a = ld_f(qh + i), b = ld_f(qh + i + half);
-                v = f < half ? a * cs - b * sn : b * cs + a * sn;
+                u = a * cs - b * sn;
+                v = b * cs + a * sn;
             }
-            qo[e] = v;
+            qo[h * R + i] = u;
+            qo[h * R + i + half] = v;
         }
     }
+    if (blockIdx.y > 0) return;
     const int slot = slots ? slots[t] : -1;
     const bool write = pos >= 0 && slot >= 0;
     if (!write && !low) return;
@@ -102,7 +105,8 @@ VOB_EXPORT int vob_latent_prep(const void* q, int code, long ld_q, int H, int D,
     if (T <= 0) return 0;
     if (H <= 0 || D < 0 || R <= 0 || (R & 1) || L <= 0 || code != cache_code) return VOB_ERR_BAD_ARG;
     if ((q && !q_rot) || (slots && (!down || !lat || !kr)) || (low && (Q <= 0 || !low_w || !low_out))) return VOB_ERR_BAD_ARG;
-    VOB_DISPATCH_ELEM(code, return vob_launch(latent_prep_kernel<ElemT, ElemT>, dim3(T), dim3(128), 0, stream, (const ElemT*)q, ld_q, H, D, R,
+    const int pairs = H * (R / 2), by = !q ? 1 : pairs <= 128 ? 1 : pairs >= 1024 ? 8 : (pairs + 127) / 128;
+    VOB_DISPATCH_ELEM(code, return vob_launch(latent_prep_kernel<ElemT, ElemT>, dim3(T, by), dim3(128), 0, stream, (const ElemT*)q, ld_q, H, D, R,
                                               (const ElemT*)down, ld, L, norm_w, eps, positions, slots, inv_freq, mag, (ElemT*)lat,
                                               (ElemT*)kr, q_rot, (const ElemT*)low, ld_low, Q, low_w, (ElemT*)low_out));
     return 0;
@@ -296,15 +300,28 @@ latent_merge_kernel(const float* __restrict__ part, const int* __restrict__ posi
         for (int i = tid; i < L; i += blockDim.x) st_f(orow + i, 0.f);
         return;
     }
-    __shared__ float m[VOB_LATENT_SPLITS], sum[VOB_LATENT_SPLITS], wgt[VOB_LATENT_SPLITS];
-    if (tid < splits) { m[tid] = p[(size_t)tid * (L + 2)]; sum[tid] = p[(size_t)tid * (L + 2) + 1]; }
+    __shared__ float wgt[VOB_LATENT_SPLITS], total;
+    if (tid < 32) {                    // one warp works out the shares' weights, two shares a lane
+        float m[2], sum[2];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int z = tid + 32 * k;
+            m[k] = z < splits ? p[(size_t)z * (L + 2)] : -INFINITY;
+            sum[k] = z < splits ? p[(size_t)z * (L + 2) + 1] : 0.f;
+        }
+        const float M = warp_max(fmaxf(m[0], m[1]));
+        float l = 0.f;
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const float w = sum[k] > 0.f ? expf(m[k] - M) : 0.f;            // 0: a share without keys, nothing of it is read
+            if (tid + 32 * k < splits) wgt[tid + 32 * k] = w;
+            l = fmaf(sum[k], w, l);
+        }
+        l = warp_sum(l);
+        if (tid == 0) total = l;
+    }
     __syncthreads();
-    float M = -INFINITY;
-    for (int z = 0; z < splits; ++z) M = fmaxf(M, m[z]);
-    if (tid < splits) wgt[tid] = sum[tid] > 0.f ? expf(m[tid] - M) : 0.f;      // 0: a share without keys, nothing of it is read
-    __syncthreads();
-    float l = 0.f;
-    for (int z = 0; z < splits; ++z) l = fmaf(sum[z], wgt[z], l);
+    const float l = total;
     const float inv = 1.0f / l;
     for (int i = tid; i < L; i += blockDim.x) {
         float a = 0.f;
@@ -393,7 +410,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 
 // NT16: groups of 16 latent columns a warp owns at most (its O accumulator is NT16 * 8 registers).
 template <int NT16, bool HEADS>
-__global__ void __launch_bounds__(256, 1)
+__global__ void __launch_bounds__(256, HEADS && NT16 <= 4 ? 2 : 1)
 latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, const float* __restrict__ q_rot,
                         const __nv_bfloat16* __restrict__ lat, const __nv_bfloat16* __restrict__ kr, const int* __restrict__ block_tables,
                         int max_pages, const int* __restrict__ seq_starts, const int* __restrict__ positions, int page_size, int H, int L,
@@ -429,14 +446,25 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
     extern __shared__ __align__(128) unsigned char ltc_smem[];
     __nv_bfloat16* Kt = reinterpret_cast<__nv_bfloat16*>(ltc_smem);                               // [BN][DP]
     __nv_bfloat16* Q = Kt + (size_t)BN * DP + (size_t)hh * 16 * DP;                                // [16][DP] per head
-    for (int e = lane + 32 * wsub; e < 16 * D; e += 32 * WPH) {
-        const int i = e / D, c = e - i * D;
-        float v = 0.f;
-        if (head && i < nrows) {
-            const size_t tok = HEADS ? r0 : r0 + i, hd = HEADS ? h + i : h;
-            v = c < L ? q_lat[tok * q_ts + hd * q_hs + c] : q_rot[(tok * H + hd) * R + (c - L)];
+    // the queries, rounded: four features a lane, up to four rows of a warp in flight (L and R are multiples of 16)
+    for (int i0 = wsub; i0 < 16; i0 += 4 * WPH) {
+        for (int c = 4 * lane; c < D; c += 128) {
+            float4 v[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const int i = i0 + k * WPH;
+                v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (head && i < nrows) {
+                    const size_t tok = HEADS ? r0 : r0 + i, hd = HEADS ? h + i : h;
+                    v[k] = *reinterpret_cast<const float4*>(c < L ? q_lat + tok * q_ts + hd * q_hs + c : q_rot + (tok * H + hd) * R + (c - L));
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const int i = i0 + k * WPH;
+                if (i < 16) *reinterpret_cast<uint2*>(Q + i * DP + c) = make_uint2(pack_bf16(v[k].x, v[k].y), pack_bf16(v[k].z, v[k].w));
+            }
         }
-        Q[i * DP + c] = __float2bfloat16_rn(v);
     }
     const int pos0 = positions[r0];
     int pos_hi = HEADS ? pos0 : pos0 + nrows - 1;
@@ -653,7 +681,8 @@ VOB_EXPORT int vob_latent_attend_tc(const float* q_lat, long q_ts, long q_hs, co
     int wph, colsw;
     const int hb = ltc_shape(H, L, R, &wph, &colsw);
     if (hb <= 0) return VOB_ERR_UNSUPPORTED;
-    if (page_size <= 0 || max_pages <= 0 || seqs > 65535 || (H + hb - 1) / hb > 65535 || (o_ts & 1) || (o_hs & 1) || ((uintptr_t)out & 3))
+    if (page_size <= 0 || max_pages <= 0 || seqs > 65535 || (H + hb - 1) / hb > 65535 || (o_ts & 1) || (o_hs & 1) || ((uintptr_t)out & 3)
+        || (q_ts & 3) || (q_hs & 3) || (((uintptr_t)q_lat | (uintptr_t)q_rot) & 15))
         return VOB_ERR_BAD_ARG;
     const size_t DP = (size_t)L + R + 8;
     const size_t smem = (size_t)VOB_LTC_BN * DP * 2 + (size_t)hb * 16 * DP * 2;
@@ -706,7 +735,8 @@ VOB_EXPORT int vob_latent_decode_tc(const float* q_lat, long q_ts, long q_hs, co
     const int hb = ltc_heads_shape(H, L, R, &wph, &colsw);
     if (hb <= 0) return VOB_ERR_UNSUPPORTED;
     if (window < 0 || page_size <= 0 || max_pages <= 0 || splits < 1 || splits > VOB_LATENT_SPLITS || (splits > 1 && !part) || H > 65535
-        || (o_ts & 1) || (o_hs & 1) || ((uintptr_t)out & 3) || ((uintptr_t)part & 7))
+        || (o_ts & 1) || (o_hs & 1) || ((uintptr_t)out & 3) || ((uintptr_t)part & 7)
+        || (q_ts & 3) || (q_hs & 3) || (((uintptr_t)q_lat | (uintptr_t)q_rot) & 15))
         return VOB_ERR_BAD_ARG;
     const size_t DP = (size_t)L + R + 8;
     const size_t smem = (size_t)VOB_LTC_BN * DP * 2 + (size_t)hb * 16 * DP * 2;
