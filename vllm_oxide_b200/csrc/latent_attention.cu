@@ -417,6 +417,7 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
                         int R, float scale, __nv_bfloat16* __restrict__ out, long o_ts, long o_hs, int WPH, int colsw, int window,
                         const int* __restrict__ row_seq, int splits, float* __restrict__ part) {
     constexpr int BN = VOB_LTC_BN;
+    constexpr int PRE = HEADS && NT16 <= 4 ? 5 : VOB_LTC_PRE;       // two blocks an SM leave room for fewer
     pdl_launch_dependents();
     pdl_wait(48);
     const int NW = blockDim.x >> 5, HB = NW / WPH;
@@ -494,46 +495,48 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
     // t, t + threads, ... The NEXT tile's pieces are fetched into registers while this tile is worked on.
     const int pieces = lat_chunks + kr_chunks, tile_pieces = BN * pieces;
     const int dp_pieces = DP / 8;                    // a row of Kt in 16-byte pieces (DP is a multiple of 8)
-    uint4 nxt[VOB_LTC_PRE];
+    uint4 nxt[PRE];
+    // where this thread's pieces lie in a tile, the same in every tile: key << 8 | piece, two to a register
+    unsigned place[(PRE + 1) / 2];
+#pragma unroll
+    for (int i = 0; i < PRE; ++i) {
+        const int x = (int)threadIdx.x + i * (int)blockDim.x;
+        const unsigned kk = x / pieces, pc = (kk << 8) | (unsigned)(x - (int)kk * pieces);
+        if (i & 1) place[i >> 1] |= pc << 16;
+        else place[i >> 1] = pc & 0xffffu;
+    }
+    const int shift = (page_size & (page_size - 1)) == 0 ? 31 - __clz(page_size) : -1;       // pages of a power of two: no division
+    auto piece = [&](int key, int c) {
+        uint4 val = make_uint4(0u, 0u, 0u, 0u);
+        if (key <= pos_hi && key >= key_lo) {
+            const int pg = shift >= 0 ? key >> shift : key / page_size;
+            const size_t slot = (size_t)table[pg] * page_size + (key - pg * page_size);
+            val = c < lat_chunks ? reinterpret_cast<const uint4*>(lat + slot * L)[c] : reinterpret_cast<const uint4*>(kr + slot * R)[c - lat_chunks];
+        }
+        return val;
+    };
     auto fetch = [&](int k0) {
 #pragma unroll
-        for (int i = 0; i < VOB_LTC_PRE; ++i) {
-            const int x = (int)threadIdx.x + i * (int)blockDim.x;
-            uint4 val = make_uint4(0u, 0u, 0u, 0u);
-            if (x < tile_pieces) {
-                const int kk = x / pieces, c = x - kk * pieces;
-                const int key = k0 + kk;
-                if (key <= pos_hi && key >= key_lo) {
-                    const size_t slot = (size_t)table[key / page_size] * page_size + key % page_size;
-                    val = c < lat_chunks ? reinterpret_cast<const uint4*>(lat + slot * L)[c]
-                                         : reinterpret_cast<const uint4*>(kr + slot * R)[c - lat_chunks];
-                }
-            }
-            nxt[i] = val;
+        for (int i = 0; i < PRE; ++i) {
+            const unsigned pc = i & 1 ? place[i >> 1] >> 16 : place[i >> 1] & 0xffffu;
+            if ((int)threadIdx.x + i * (int)blockDim.x < tile_pieces) nxt[i] = piece(k0 + (int)(pc >> 8), (int)(pc & 255u));
         }
     };
     fetch(k_start);
+    const float scale2 = scale * 1.4426950408889634f;        // scores in units of ln 2, for exp2f
+    const int p_min = pos0, p_max = HEADS ? pos0 : pos0 + nrows - 1;             // positions of the tile's first and last row
     for (int k0 = k_start; k0 <= pos_hi; k0 += BN) {
         __syncthreads();
 #pragma unroll
-        for (int i = 0; i < VOB_LTC_PRE; ++i) {
-            const int x = (int)threadIdx.x + i * (int)blockDim.x;
-            if (x < tile_pieces) {
-                const int kk = x / pieces, c = x - kk * pieces;
-                reinterpret_cast<uint4*>(Kt)[(size_t)kk * dp_pieces + c] = nxt[i];
-            }
+        for (int i = 0; i < PRE; ++i) {
+            const unsigned pc = i & 1 ? place[i >> 1] >> 16 : place[i >> 1] & 0xffffu;
+            if ((int)threadIdx.x + i * (int)blockDim.x < tile_pieces)
+                reinterpret_cast<uint4*>(Kt)[(pc >> 8) * (unsigned)dp_pieces + (pc & 255u)] = nxt[i];
         }
         // what of a tile the registers do not hold (small blocks, wide keys) is copied now
-        for (int x = (int)threadIdx.x + VOB_LTC_PRE * (int)blockDim.x; x < tile_pieces; x += (int)blockDim.x) {
+        for (int x = (int)threadIdx.x + PRE * (int)blockDim.x; x < tile_pieces; x += (int)blockDim.x) {
             const int kk = x / pieces, c = x - kk * pieces;
-            const int key = k0 + kk;
-            uint4 val = make_uint4(0u, 0u, 0u, 0u);
-            if (key <= pos_hi && key >= key_lo) {
-                const size_t slot = (size_t)table[key / page_size] * page_size + key % page_size;
-                val = c < lat_chunks ? reinterpret_cast<const uint4*>(lat + slot * L)[c]
-                                     : reinterpret_cast<const uint4*>(kr + slot * R)[c - lat_chunks];
-            }
-            reinterpret_cast<uint4*>(Kt)[(size_t)kk * dp_pieces + c] = val;
+            reinterpret_cast<uint4*>(Kt)[(size_t)kk * dp_pieces + c] = piece(k0 + kk, c);
         }
         if (k0 + BN <= pos_hi) fetch(k0 + BN);
         __syncthreads();
@@ -556,17 +559,30 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
         }
         // the softmax of rows g and g + 8 over this tile's keys
         float mx0 = -INFINITY, mx1 = -INFINITY;
+        if (k0 + BN - 1 <= p_min && (window <= 0 || k0 > p_max - window)) {      // every row sees the whole tile
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+            for (int j = 0; j < 4; ++j) {
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int key = k0 + 8 * j + 2 * t4 + e;
-                const bool in0 = key <= p0 && (window <= 0 || key > p0 - window);
-                const bool in1 = key <= p1 && (window <= 0 || key > p1 - window);
-                sc[j][e] = (row0 && in0) ? sc[j][e] * scale : -INFINITY;
-                sc[j][2 + e] = (row1 && in1) ? sc[j][2 + e] * scale : -INFINITY;
-                mx0 = fmaxf(mx0, sc[j][e]);
-                mx1 = fmaxf(mx1, sc[j][2 + e]);
+                for (int e = 0; e < 2; ++e) {
+                    sc[j][e] *= scale2;
+                    sc[j][2 + e] *= scale2;
+                    mx0 = fmaxf(mx0, sc[j][e]);
+                    mx1 = fmaxf(mx1, sc[j][2 + e]);
+                }
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int key = k0 + 8 * j + 2 * t4 + e;
+                    const bool in0 = key <= p0 && (window <= 0 || key > p0 - window);
+                    const bool in1 = key <= p1 && (window <= 0 || key > p1 - window);
+                    sc[j][e] = (row0 && in0) ? sc[j][e] * scale2 : -INFINITY;
+                    sc[j][2 + e] = (row1 && in1) ? sc[j][2 + e] * scale2 : -INFINITY;
+                    mx0 = fmaxf(mx0, sc[j][e]);
+                    mx1 = fmaxf(mx1, sc[j][2 + e]);
+                }
             }
         }
         mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
@@ -575,14 +591,14 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
         mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
         const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
         const bool none0 = mn0 == -INFINITY, none1 = mn1 == -INFINITY;
-        const float corr0 = none0 ? 1.f : expf(m0 - mn0), corr1 = none1 ? 1.f : expf(m1 - mn1);
+        const float corr0 = none0 ? 1.f : exp2f(m0 - mn0), corr1 = none1 ? 1.f : exp2f(m1 - mn1);
         float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                sc[j][e] = none0 ? 0.f : expf(sc[j][e] - mn0);
-                sc[j][2 + e] = none1 ? 0.f : expf(sc[j][2 + e] - mn1);
+                sc[j][e] = none0 ? 0.f : exp2f(sc[j][e] - mn0);
+                sc[j][2 + e] = none1 ? 0.f : exp2f(sc[j][2 + e] - mn1);
                 sum0 += sc[j][e];
                 sum1 += sc[j][2 + e];
             }
@@ -625,8 +641,8 @@ latent_attend_tc_kernel(const float* __restrict__ q_lat, long q_ts, long q_hs, c
         float* pr0 = part + (((size_t)r0 * H + h + g) * splits + blockIdx.z) * (L + 2);
         float* pr1 = pr0 + (size_t)8 * splits * (L + 2);
         if (wsub == 0 && t4 == 0) {
-            if (row0) { pr0[0] = m0; pr0[1] = l0; }
-            if (row1) { pr1[0] = m1; pr1[1] = l1; }
+            if (row0) { pr0[0] = m0 * 0.6931471805599453f; pr0[1] = l0; }
+            if (row1) { pr1[0] = m1 * 0.6931471805599453f; pr1[1] = l1; }
         }
 #pragma unroll
         for (int n = 0; n < NT16 * 2; ++n) {
