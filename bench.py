@@ -707,7 +707,8 @@ def rotepel_roofline(rs, blocks, n, batch, peaks, prefill, decode):
     out = {}
 
     def add(name, phase, totals, nbytes=None, flops=None):
-        ms = sum(t for op, _, t in totals if op == name or op == name + "_tc")      # the tensor-core form of a kernel counts with it
+        also = {name + "_tc"} | ({"latent_decode_tc"} if name == "latent_attend" else set())     # the tensor-core forms of a kernel count with it
+        ms = sum(t for op, _, t in totals if op == name or op in also)
         if ms <= 0:
             return
         e = {"ms": round(ms, 4)}
@@ -1151,7 +1152,7 @@ def pironex_roofline(ps, blocks, n, batch, peaks, prefill, decode):
             nbytes=2 * blocks * keys * (kd + vd) * 2 if phase == "decode" else None, flops=2 * blocks * keys * at["heads"] * 2 * (at["dim"] + at["vdim"]))
         add(("flex_prep",), "flex_prep", phase, totals, nbytes=blocks * rows * ((2 * qd + 2 * kd + 2 * vd) + 2 * qd) * 2)
         lkeys = sum(min(i + 1, win) for i in range(n)) if phase == "prefill" else batch * min(n + 3, win)
-        add(("latent_attend", "latent_attend_tc"), "latent attention", phase, totals,
+        add(("latent_attend", "latent_attend_tc", "latent_decode_tc"), "latent attention", phase, totals,
             nbytes=blocks * lkeys * (lat["kv_rank"] + lat["rot_dim"]) * 2 if phase == "decode" else None,
             flops=blocks * lkeys * lat["heads"] * 2 * (2 * lat["kv_rank"] + lat["rot_dim"]))
         seqs = 1 if phase == "prefill" else batch
@@ -1414,7 +1415,7 @@ def side_by_side_roofline(arch, rs, n, batch, peaks, prefill, decode):
             nbytes=nA * keys * (kd + vd) * 2 if phase == "decode" else None, flops=nA * keys * at["heads"] * 2 * (at["dim"] + at["vdim"]))
         add(("flex_prep",), "flex_prep", phase, totals, nbytes=nA * rows * 2 * (qd + kd + vd) * 2)
         lkeys = sum(i + 1 for i in range(n)) if phase == "prefill" else batch * (n + 3)
-        add(("latent_attend", "latent_attend_tc"), "latent attention", phase, totals,
+        add(("latent_attend", "latent_attend_tc", "latent_decode_tc"), "latent attention", phase, totals,
             nbytes=nL * lkeys * (lat["kv_rank"] + lat["rot_dim"]) * 2 if phase == "decode" else None,
             flops=nL * lkeys * lat["heads"] * 2 * (2 * lat["kv_rank"] + lat["rot_dim"]))
         # the latent and the rotated key part read and written, the rotated query parts read and written (float32); the query
